@@ -151,7 +151,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
   const uint32_t tmem_O = tmem_base + 32;  // 16 columns
 
   // Single-thread roles: whole warp converged through loops and waits, TMA / tcgen05 instructions predicated on an
-  // elect.sync leader (under `if (lane == 0)` ptxas wraps each of them in a waterfall loop; see gemm.cu).
+  // elect.sync leader (issuing under `if (lane == 0)` measured slower; see gemm.cu).
   if (warp == 0) {
     const bool elected = elect_one_sync();
     {

@@ -235,7 +235,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
   const uint32_t tmem_base = __shfl_sync(0xffffffffu, *tmem_ptr, 0);  // warp-uniform for the compiler too
 
   // Single-thread roles: whole warp converged through loops and waits, TMA / tcgen05 instructions predicated on an
-  // elect.sync leader (under `if (lane == 0)` ptxas wraps each of them in a waterfall loop; see gemm.cu).
+  // elect.sync leader (issuing under `if (lane == 0)` measured slower; see gemm.cu).
   if (warp == 0) {
     const bool elected = elect_one_sync();
     {
