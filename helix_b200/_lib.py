@@ -40,14 +40,15 @@ class LayerDescC(C.Structure):
                 ("weights_of", C.c_int32), ("rope_linear", C.c_float), ("norm_groups", C.c_int32), ("gate_cap", C.c_float),
                 ("side_mixer", C.c_int32), ("side_heads", C.c_int32), ("side_dim", C.c_int32), ("side_vdim", C.c_int32),
                 ("side_gate_cap", C.c_float), ("mix_scale", C.c_float), ("side_scale", C.c_float),
-                ("reserved", C.c_int32 * 5)]
+                ("route_bias", C.c_int32), ("reserved", C.c_int32 * 4)]
 
 
 class StackDescC(C.Structure):
     _fields_ = [("width", C.c_int32), ("vocab", C.c_int32), ("n_layers", C.c_int32), ("compute_f32", C.c_int32),
                 ("norm_eps", C.c_float), ("resid_alpha", C.c_float), ("logit_softcap", C.c_float), ("norm_place", C.c_int32),
                 ("embed_norm", C.c_int32), ("plain_gains", C.c_int32), ("norm_kind", C.c_int32), ("embed_scale", C.c_float),
-                ("logit_scale", C.c_float), ("tie_head", C.c_int32), ("reserved", C.c_int32 * 4)]
+                ("logit_scale", C.c_float), ("tie_head", C.c_int32), ("one_norm", C.c_int32),
+                ("layer_scale", C.c_int32), ("resid_mult", C.c_float), ("reserved", C.c_int32 * 1)]
 
 
 class SeqFeedC(C.Structure):

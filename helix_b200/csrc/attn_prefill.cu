@@ -66,18 +66,24 @@ __device__ int g_attn_trace_n[8];
 #define HB_TRACE(ev) do {} while (0)
 #endif
 
-template <int D>
+// Where K and V rows come from: the packed activation, the paged planes, or (latent attention) expanded rows — per-head key and
+// value parts made from cached latents plus one rotated key part that all heads share.
+enum KvSource : int { KV_PACKED = 0, KV_PAGED = 1, KV_EXPANDED = 2 };
+
+template <int DK, int DV, int SRC>
 struct ACfg {
-  static constexpr int Q_BYTES = BQ * D * 2;    // one q tile
-  static constexpr int KV_BYTES = BKV * D * 2;
-  static constexpr int STAGES = D == 128 ? 3 : 4;  // K ring and V ring depth (16 KB tiles at D = 128)
+  static constexpr int Q_BYTES = BQ * DK * 2;    // one q tile
+  static constexpr int K_BYTES = BKV * DK * 2;
+  static constexpr int V_BYTES = BKV * DV * 2;
+  static constexpr int STAGES = DK * DV >= 128 * 128 && !(SRC == KV_EXPANDED && DK == 128) ? 3 : 4;  // K ring and V ring depth
   // D = 64 (encoder; short sequences, an item's output write-back is a large part of its time) stages O in shared
-  // memory and writes it with TMA: one 32-row x 128 B swizzled box per softmax warp.  At D = 128 the K/V rings leave no room.
-  static constexpr bool STAGE_O = true;
-  static constexpr int O_STAGE_BYTES = 32 * D * 2;  // per softmax warp
+  // memory and writes it with TMA: one 32-row x 128 B swizzled box per softmax warp.  Expanded rows leave no room for it.
+  static constexpr bool STAGE_O = SRC != KV_EXPANDED;
+  static constexpr int O_STAGE_BYTES = 32 * DV * 2;  // per softmax warp
   static constexpr int BAR_BYTES = 1024;            // barriers + TMEM pointer, padded so the staging area stays 1024-aligned
-  static constexpr int SMEM = 2 * Q_BYTES + 2 * STAGES * KV_BYTES + 1024 + BAR_BYTES + (STAGE_O ? 8 * O_STAGE_BYTES : 0);
-  static constexpr int SUB = D / 64;  // 64-column swizzle sub-tiles per row
+  static constexpr int SMEM = 2 * Q_BYTES + STAGES * (K_BYTES + V_BYTES) + 1024 + BAR_BYTES + (STAGE_O ? 8 * O_STAGE_BYTES : 0);
+  static constexpr int SUBK = DK / 64, SUBV = DV / 64;  // 64-column swizzle sub-tiles per row
+  static_assert(SMEM <= 227 * 1024, "shared memory");
 };
 
 // PERSISTENT kernel: one CTA per SM walks a static list of (256-row q pair, sequence, q-head) items, heaviest
@@ -97,11 +103,15 @@ struct ACfg {
 //                   from TMEM (tcgen05.mma A-from-TMEM), V straight from its [kv][d] layout (MN-major B).
 //   warps 2..5 / 6..9 : softmax warpgroup of q tile 0 / 1, one thread per q row; lazy O rescale; O/l -> global.
 //
-// PAGED = false: K/V rows come from the same packed [T, ...] activation as Q (whole-prompt prefill, encoder), kv_len == q_len.
-// PAGED = true : the q rows are the LAST q_len positions of a kv_len-long sequence whose K/V (including the chunk's own,
+// KV_PACKED: K/V rows come from the same packed [T, ...] activation as Q (whole-prompt prefill, encoder), kv_len == q_len.
+// KV_PAGED: the q rows are the LAST q_len positions of a kv_len-long sequence whose K/V (including the chunk's own,
 //                written by the RoPE/KV-write kernel just before) live in the paged pool (chunked prefill, prefix-cache
 //                hits): tile j is page_table[b][j].
-template <int D, bool PAGED, int POLY>
+// KV_EXPANDED: batch entry b is run b of `runs` (q rows [t0, t0 + len) of the packed activation, the last rows of the kv rows
+//                [row0, row0 + kv) of the expanded buffers).  A q / k row has DK / 64 sub-tiles: the head's unrotated part in
+//                all but the last, the rotated part (shared by all heads on the key side) in the last; parts that are no
+//                multiple of 64 wide are zero-filled by the tensor maps.
+template <int DK, int DV, int SRC, int POLY>
 __global__ void __launch_bounds__(kThreads, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_o,
@@ -109,15 +119,18 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     const int32_t* __restrict__ cu_seqlens, int B, int Hq, int group, int causal, float scale_log2,
                     int max_q_pairs, const int32_t* __restrict__ kv_lens, const int32_t* __restrict__ page_table,
                     int max_pages, int Hkv, int chunk, int sink, const float* __restrict__ head_gate, int ldg,
-                    int window, float cap_in, float cap_out, const bf16* __restrict__ sink_w) {
-  using C = ACfg<D>;
+                    int window, float cap_in, float cap_out, const bf16* __restrict__ sink_w,
+                    const __grid_constant__ CUtensorMap map_qr, const __grid_constant__ CUtensorMap map_kr,
+                    const __grid_constant__ AttnRuns runs, int vdim, const float* __restrict__ entry_gate) {
+  using C = ACfg<DK, DV, SRC>;
+  constexpr bool PAGED = SRC == KV_PAGED, EXPANDED = SRC == KV_EXPANDED;
   constexpr int KST = C::STAGES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;                          // [2][Q_BYTES]
-  uint8_t* sK = sQ + 2 * C::Q_BYTES;           // [KST][KV_BYTES]
-  uint8_t* sV = sK + KST * C::KV_BYTES;        // [KST][KV_BYTES]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + KST * C::KV_BYTES);
+  uint8_t* sK = sQ + 2 * C::Q_BYTES;           // [KST][K_BYTES]
+  uint8_t* sV = sK + KST * C::K_BYTES;        // [KST][V_BYTES]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + KST * C::V_BYTES);
   uint64_t* q_full = bars + 0;
   uint64_t* q_empty = bars + 1;
   uint64_t* s_full = bars + 2;    // [q tile][S buffer]
@@ -130,7 +143,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   uint64_t* v_full = k_empty + KST;
   uint64_t* v_empty = v_full + KST;
   uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(v_empty + KST);
-  uint8_t* sO = reinterpret_cast<uint8_t*>(bars) + C::BAR_BYTES;  // [8 softmax warps][32 rows][D] (STAGE_O only)
+  uint8_t* sO = reinterpret_cast<uint8_t*>(bars) + C::BAR_BYTES;  // [8 softmax warps][32 rows][DV] (STAGE_O only)
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int num_items = max_q_pairs * B * Hq;
@@ -148,9 +161,15 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     it.b = rem / Hq;
     it.h = rem % Hq;
     it.kvh = it.h / group;
-    it.seq0 = cu_seqlens[it.b];
-    it.len = cu_seqlens[it.b + 1] - it.seq0;  // q rows of this sequence in the step
-    it.kv_len = PAGED ? kv_lens[it.b] : it.len;
+    if constexpr (EXPANDED) {  // positions below count from the first expanded row of the run
+      it.seq0 = runs.t0[it.b];
+      it.len = runs.len[it.b];
+      it.kv_len = runs.kv[it.b];
+    } else {
+      it.seq0 = cu_seqlens[it.b];
+      it.len = cu_seqlens[it.b + 1] - it.seq0;  // q rows of this sequence in the step
+      it.kv_len = PAGED ? kv_lens[it.b] : it.len;
+    }
     it.q_off = it.kv_len - it.len;  // position of the first q row (0 unless this is a later chunk of a long prompt)
     it.q0 = qp * QPAIR;
     it.valid = it.q0 < it.len;
@@ -162,7 +181,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     // sliding window (window > 0, paged only): a row sees the `window` positions that end with itself; tiles before the
     // window of the pair's first row are skipped
     it.j_lo = (PAGED && chunk > 0) ? ((it.q_off + it.q0) / chunk * chunk) / BKV
-              : (PAGED && window > 0) ? max(0, it.q_off + it.q0 - window + 1) / BKV : 0;
+              : (SRC != KV_PACKED && window > 0) ? max(0, it.q_off + it.q0 - window + 1) / BKV : 0;
     it.n0 = (causal ? min(kv_tiles, (it.q_off + it.q0 + BQ - 1) / BKV + 1) : kv_tiles) - it.j_lo;
     it.n1 = it.act1 ? (causal ? min(kv_tiles, (it.q_off + it.q0 + 2 * BQ - 1) / BKV + 1) : kv_tiles) - it.j_lo : 0;
     it.n = max(it.n0, it.n1);
@@ -174,6 +193,10 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     tma_prefetch_desc(&map_k);
     tma_prefetch_desc(&map_v);
     if constexpr (C::STAGE_O) tma_prefetch_desc(&map_o);
+    if constexpr (EXPANDED) {
+      tma_prefetch_desc(&map_qr);
+      tma_prefetch_desc(&map_kr);
+    }
     mbar_init(q_full, 1);
     mbar_init(q_empty, 2);  // both issuers
     for (int i = 0; i < 4; ++i) {
@@ -214,38 +237,50 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           mbar_arrive_expect_tx(q_full, (it.act1 ? 2 : 1) * C::Q_BYTES);
           for (int t = 0; t < (it.act1 ? 2 : 1); ++t)
 #pragma unroll
-            for (int c = 0; c < C::SUB; ++c)
-              tma_load_2d(sQ + t * C::Q_BYTES + c * (BQ * 128), &map_q, q_full, it.h * D + c * 64,
-                          it.seq0 + it.q0 + t * BQ, kEvictFirst);
+            for (int c = 0; c < C::SUBK; ++c) {
+              uint8_t* dst = sQ + t * C::Q_BYTES + c * (BQ * 128);
+              const int row = it.seq0 + it.q0 + t * BQ;
+              if constexpr (EXPANDED)
+                tma_load_3d(dst, c < C::SUBK - 1 ? &map_q : &map_qr, q_full, c < C::SUBK - 1 ? c * 64 : 0, it.h, row, kEvictFirst);
+              else
+                tma_load_2d(dst, &map_q, q_full, it.h * DK + c * 64, row, kEvictFirst);
+            }
         }
         ++qi;
         for (int j = 0; j < it.n; ++j, ++kt) {
           const int s = kt % KST;
           const uint32_t ph = (kt / KST) & 1;
           int blk = 0;  // PAGED: (page, kv head) block of the tile's page
+          if constexpr (EXPANDED) blk = runs.row0[it.b] + (it.j_lo + j) * BKV;  // first expanded row of the tile
           if constexpr (PAGED) blk = page_table[(size_t)it.b * max_pages + it.j_lo + j] * Hkv + it.kvh;
           mbar_wait(&k_empty[s], ph ^ 1);
           if (leader) {
-            mbar_arrive_expect_tx(&k_full[s], C::KV_BYTES);
+            mbar_arrive_expect_tx(&k_full[s], C::K_BYTES);
 #pragma unroll
-            for (int c = 0; c < C::SUB; ++c) {
-              uint8_t* dst = sK + s * C::KV_BYTES + c * (BKV * 128);
-              if constexpr (PAGED)
+            for (int c = 0; c < C::SUBK; ++c) {
+              uint8_t* dst = sK + s * C::K_BYTES + c * (BKV * 128);
+              if constexpr (EXPANDED) {
+                if (c < C::SUBK - 1) tma_load_3d(dst, &map_k, &k_full[s], c * 64, it.h, blk, kEvictLast);
+                else tma_load_2d(dst, &map_kr, &k_full[s], 0, blk, kEvictLast);
+              } else if constexpr (PAGED) {
                 tma_load_3d(dst, &map_k, &k_full[s], c * 64, 0, blk, kEvictLast);
-              else
-                tma_load_2d(dst, &map_k, &k_full[s], it.kvh * D + c * 64, it.seq0 + j * BKV, kEvictLast);
+              } else {
+                tma_load_2d(dst, &map_k, &k_full[s], it.kvh * DK + c * 64, it.seq0 + j * BKV, kEvictLast);
+              }
             }
           }
           mbar_wait(&v_empty[s], ph ^ 1);
           if (leader) {
-            mbar_arrive_expect_tx(&v_full[s], C::KV_BYTES);
+            mbar_arrive_expect_tx(&v_full[s], C::V_BYTES);
 #pragma unroll
-            for (int c = 0; c < C::SUB; ++c) {
-              uint8_t* dst = sV + s * C::KV_BYTES + c * (BKV * 128);
-              if constexpr (PAGED)
+            for (int c = 0; c < C::SUBV; ++c) {
+              uint8_t* dst = sV + s * C::V_BYTES + c * (BKV * 128);
+              if constexpr (EXPANDED)
+                tma_load_3d(dst, &map_v, &v_full[s], c * 64, it.h, blk, kEvictLast);
+              else if constexpr (PAGED)
                 tma_load_3d(dst, &map_v, &v_full[s], c * 64, 0, blk, kEvictLast);
               else
-                tma_load_2d(dst, &map_v, &v_full[s], it.kvh * D + c * 64, it.seq0 + j * BKV, kEvictLast);
+                tma_load_2d(dst, &map_v, &v_full[s], it.kvh * DV + c * 64, it.seq0 + j * BKV, kEvictLast);
             }
           }
         }
@@ -263,7 +298,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int t = warp - 1;
     const bool leader = elect_one_sync();
     constexpr uint32_t idesc_qk = umma_idesc_bf16(BQ, BKV, 0, 0);
-    constexpr uint32_t idesc_pv = umma_idesc_bf16(BQ, D, 0, 1);  // A = P from TMEM, B = V is MN-major
+    constexpr uint32_t idesc_pv = umma_idesc_bf16(BQ, DV, 0, 1);  // A = P from TMEM, B = V is MN-major
     const uint64_t qdesc = umma_desc_kmajor_sw128(smem_u32(sQ + t * C::Q_BYTES));
     const uint64_t kdesc0 = umma_desc_kmajor_sw128(smem_u32(sK));
     const uint64_t vdesc0 = umma_desc_mnmajor_sw128(smem_u32(sV), BKV * 128, 1024);
@@ -278,9 +313,9 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     // S(tile x) = Q_t · Kᵀ (K in ring slot kslot) into buffer x & 1
     auto mma_s = [&](int x) {
       const uint32_t d_tmem = tmem_s + (x & 1) * BKV;
-      const uint64_t kd = kdesc0 + (uint64_t)(kslot * (C::KV_BYTES >> 4));
+      const uint64_t kd = kdesc0 + (uint64_t)(kslot * (C::K_BYTES >> 4));
 #pragma unroll
-      for (int k = 0; k < D / 16; ++k)
+      for (int k = 0; k < DK / 16; ++k)
         umma_f16_ss(d_tmem, qdesc + (((k >> 2) * (BQ * 128) + (k & 3) * 32) >> 4),
                     kd + (((k >> 2) * (BKV * 128) + (k & 3) * 32) >> 4), idesc_qk, k != 0 ? 1u : 0u);
       umma_commit(&my_s_full[x & 1]);
@@ -289,7 +324,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     // O_t (+)= P(tile x) · V (V in ring slot vslot)
     auto mma_pv = [&](int x, uint32_t acc) {
       const uint32_t p_tmem = tmem_s + (x & 1) * BKV;
-      const uint64_t vd = vdesc0 + (uint64_t)(vslot * (C::KV_BYTES >> 4));
+      const uint64_t vd = vdesc0 + (uint64_t)(vslot * (C::V_BYTES >> 4));
 #pragma unroll
       for (int k = 0; k < BKV / 16; ++k)
         umma_f16_ts(tmem_o, p_tmem + k * 8, vd + ((k * 16 * 128) >> 4), idesc_pv, (acc | k) != 0 ? 1u : 0u);
@@ -426,7 +461,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             m_used = m_new;
             l *= f;
 #pragma unroll
-            for (int c = 0; c < D / 32; ++c) {
+            for (int c = 0; c < DV / 32; ++c) {
               uint32_t o[32];
               tmem_ld_32x32b_x32(tO + c * 32, o);
               tmem_ld_wait();
@@ -496,7 +531,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           if (lane == 0) tma_store_wait_read<0>();  // this warp's previous store has finished reading the buffer
           __syncwarp();
 #pragma unroll
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t o[32];
             tmem_ld_32x32b_x32(tO + c * 32, o);
             tmem_ld_wait();
@@ -516,23 +551,36 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           __syncwarp();
           if (lane == 0) {
 #pragma unroll
-            for (int c = 0; c < C::SUB; ++c)
-              tma_store_2d(&map_o, stage + c * (32 * 128), it.h * D + c * 64, it.seq0 + it.q0 + t * BQ + qd * 32);
+            for (int c = 0; c < C::SUBV; ++c)
+              tma_store_2d(&map_o, stage + c * (32 * 128), it.h * DV + c * 64, it.seq0 + it.q0 + t * BQ + qd * 32);
             tma_store_commit();
             mbar_arrive(&o_free[t]);
           }
         }
       }
       if (!staged) {
-        bf16* orow = out + (size_t)(it.seq0 + qrow) * ldo + it.h * D;
+        const int dv = EXPANDED ? vdim : DV;
+        bf16* orow = out + (size_t)(it.seq0 + qrow) * ldo + it.h * dv;
+        const float* grow = EXPANDED && entry_gate ? entry_gate + (size_t)(it.seq0 + qrow) * ldg + it.h * dv : nullptr;
 #pragma unroll
-        for (int c = 0; c < D / 32; ++c) {
+        for (int c = 0; c < DV / 32; ++c) {
           uint32_t o[32];
           tmem_ld_32x32b_x32(tO + c * 32, o);
           tmem_ld_wait();
           if (qrow < it.len) {
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
+              if (EXPANDED && c * 32 + i * 8 >= dv) break;  // vdim is a multiple of 8
+              if constexpr (EXPANDED) {
+                if (grow != nullptr) {  // one gate per output entry
+                  const float4 ga = *reinterpret_cast<const float4*>(grow + c * 32 + i * 8);
+                  const float4 gb = *reinterpret_cast<const float4*>(grow + c * 32 + i * 8 + 4);
+                  const float gg[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
+#pragma unroll
+                  for (int e = 0; e < 8; ++e)
+                    o[8 * i + e] = __float_as_uint(__fdividef(__uint_as_float(o[8 * i + e]), 1.f + __expf(-gg[e])));
+                }
+              }
               uint4 w;
               w.x = pack_bf16x2(__uint_as_float(o[8 * i + 0]) * inv_l, __uint_as_float(o[8 * i + 1]) * inv_l);
               w.y = pack_bf16x2(__uint_as_float(o[8 * i + 2]) * inv_l, __uint_as_float(o[8 * i + 3]) * inv_l);
@@ -564,7 +612,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 inline int paged_only(int v, bool paged) { return paged ? v : 0; }
 template <int D, bool PAGED, int POLY>
 cudaError_t launch_p(cudaStream_t stream, const AttnPrefillArgs& a) {
-  using C = ACfg<D>;
+  constexpr int SRC = PAGED ? KV_PAGED : KV_PACKED;
+  using C = ACfg<D, D, SRC>;
   CUtensorMap mq, mk, mv, mo;
   if (!make_tmap_2d(&mo, a.out, TM_BF16, (uint64_t)a.Hq * D, (uint64_t)a.T, (uint64_t)a.ldo * 2, 64, 32)) return cudaErrorInvalidValue;
   if (!make_tmap_2d(&mq, a.q, TM_BF16, (uint64_t)a.Hq * D, (uint64_t)a.T, (uint64_t)a.ldq * 2, 64, BQ)) return cudaErrorInvalidValue;
@@ -577,7 +626,7 @@ cudaError_t launch_p(cudaStream_t stream, const AttnPrefillArgs& a) {
     if (!make_tmap_2d(&mk, a.k, TM_BF16, (uint64_t)a.Hkv * D, (uint64_t)a.T, (uint64_t)a.ldk * 2, 64, BKV)) return cudaErrorInvalidValue;
     if (!make_tmap_2d(&mv, a.v, TM_BF16, (uint64_t)a.Hkv * D, (uint64_t)a.T, (uint64_t)a.ldv * 2, 64, BKV)) return cudaErrorInvalidValue;
   }
-  auto kern = attn_prefill_kernel<D, PAGED, POLY>;
+  auto kern = attn_prefill_kernel<D, D, SRC, POLY>;
   static int num_sms = 0;
   if (num_sms == 0) {
     int dev = 0;
@@ -592,7 +641,33 @@ cudaError_t launch_p(cudaStream_t stream, const AttnPrefillArgs& a) {
                                             scale_log2, max_q_pairs, a.kv_lens, a.page_table, a.max_pages, a.Hkv,
                                             paged_only(a.block_mask, PAGED), a.unit_sink, a.head_gate, a.ldg,
                                             paged_only(a.window, PAGED), a.softcap > 0.f ? a.scale / a.softcap : 0.f,
-                                            a.softcap > 0.f ? a.softcap * 1.4426950408889634f : 0.f, a.sink);
+                                            a.softcap > 0.f ? a.softcap * 1.4426950408889634f : 0.f, a.sink, mq, mk, AttnRuns{}, D, nullptr);
+  return cudaGetLastError();
+}
+
+// latent attention over expanded rows
+template <int DK, int DV>
+cudaError_t launch_expanded(cudaStream_t stream, const AttnExpandedArgs& a) {
+  using C = ACfg<DK, DV, KV_EXPANDED>;
+  CUtensorMap mq, mqr, mk, mkr, mv;
+  const uint64_t hd = (uint64_t)(a.nope + a.rot) * 2, H = a.H, T = a.T, rows = a.rows;
+  if (!make_tmap_3d(&mq, a.q, TM_BF16, a.nope, H, T, hd, (uint64_t)a.ldq * 2, 64, 1, BQ)) return cudaErrorInvalidValue;
+  if (!make_tmap_3d(&mqr, a.q + a.nope, TM_BF16, a.rot, H, T, hd, (uint64_t)a.ldq * 2, 64, 1, BQ)) return cudaErrorInvalidValue;
+  if (!make_tmap_3d(&mk, a.k, TM_BF16, a.nope, H, rows, (uint64_t)a.nope * 2, (uint64_t)a.ldkv * 2, 64, 1, BKV)) return cudaErrorInvalidValue;
+  if (!make_tmap_3d(&mv, a.v, TM_BF16, a.vdim, H, rows, (uint64_t)a.vdim * 2, (uint64_t)a.ldkv * 2, 64, 1, BKV)) return cudaErrorInvalidValue;
+  if (!make_tmap_2d(&mkr, a.k_rot, TM_BF16, a.rot, rows, (uint64_t)a.ldkr * 2, 64, BKV)) return cudaErrorInvalidValue;
+  auto kern = attn_prefill_kernel<DK, DV, KV_EXPANDED, 2>;
+  int longest = 0;
+  for (int i = 0; i < a.runs.n; ++i) longest = std::max(longest, a.runs.len[i]);
+  const int max_q_pairs = (longest + QPAIR - 1) / QPAIR;
+  const long long items = (long long)max_q_pairs * a.runs.n * a.H;
+  int dev = 0, num_sms = 0;
+  cudaGetDevice(&dev);
+  cudaDeviceGetAttribute(&num_sms, cudaDevAttrMultiProcessorCount, dev);
+  const int grid = (int)std::min<long long>(items, effective_sms(num_sms));
+  kern<<<grid, kThreads, C::SMEM, stream>>>(mq, mk, mv, mq, a.out, a.ldo, nullptr, a.runs.n, a.H, 1, 1, a.scale * 1.4426950408889634f,
+                                            max_q_pairs, nullptr, nullptr, 0, a.H, 0, 0, a.head_gate, a.ldg, a.window, 0.f, 0.f, a.sink,
+                                            mqr, mkr, a.runs, a.vdim, a.entry_gate);
   return cudaGetLastError();
 }
 
@@ -649,13 +724,19 @@ cudaError_t launch(cudaStream_t stream, const AttnPrefillArgs& a) {
 cudaError_t attn_prefill_init() {
   cudaError_t e;
 #define HB_ATTR1(D_, P_, Y_)                                                                                         \
-  if ((e = cudaFuncSetAttribute(attn_prefill_kernel<D_, P_, Y_>, cudaFuncAttributeMaxDynamicSharedMemorySize,         \
-                                ACfg<D_>::SMEM)) != cudaSuccess)                                                     \
+  if ((e = cudaFuncSetAttribute(attn_prefill_kernel<D_, D_, P_, Y_>, cudaFuncAttributeMaxDynamicSharedMemorySize,     \
+                                ACfg<D_, D_, P_>::SMEM)) != cudaSuccess)                                             \
     return e;
 #define HB_ATTR(D_, P_) HB_ATTR1(D_, P_, 0) HB_ATTR1(D_, P_, 2) HB_ATTR1(D_, P_, 4)
-  HB_ATTR(128, false) HB_ATTR(128, true) HB_ATTR(64, false) HB_ATTR(64, true)
+  HB_ATTR(128, KV_PACKED) HB_ATTR(128, KV_PAGED) HB_ATTR(64, KV_PACKED) HB_ATTR(64, KV_PAGED)
 #undef HB_ATTR
 #undef HB_ATTR1
+#define HB_ATTRX(K_, V_)                                                                                                  \
+  if ((e = cudaFuncSetAttribute(attn_prefill_kernel<K_, V_, KV_EXPANDED, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                ACfg<K_, V_, KV_EXPANDED>::SMEM)) != cudaSuccess)                                        \
+    return e;
+  HB_ATTRX(128, 64) HB_ATTRX(128, 128) HB_ATTRX(192, 64) HB_ATTRX(192, 128)
+#undef HB_ATTRX
   return cudaSuccess;
 }
 
@@ -675,6 +756,19 @@ cudaError_t attn_prefill(cudaStream_t stream, const AttnPrefillArgs& a) {
   if (a.D == 128) return launch<128, false>(stream, a);
   if (a.D == 64) return launch<64, false>(stream, a);
   return cudaErrorInvalidValue;
+}
+
+bool attn_expanded_ok(int nope, int rot, int vdim) {
+  return nope > 0 && rot > 0 && vdim > 0 && nope % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && nope <= 128 && rot <= 64 && vdim <= 128;
+}
+cudaError_t attn_expanded(cudaStream_t stream, const AttnExpandedArgs& a) {
+  if (a.runs.n <= 0) return cudaSuccess;
+  if (!attn_expanded_ok(a.nope, a.rot, a.vdim) || a.H <= 0 || a.T <= 0 || a.rows <= 0 || a.runs.n > AttnRuns::kMax || a.window < 0) return cudaErrorInvalidValue;
+  if (a.ldq % 8 || a.ldkv % 8 || a.ldkr % 8 || a.ldo % 8) return cudaErrorInvalidValue;
+  if (a.entry_gate && (a.ldg % 4 || ((uintptr_t)a.entry_gate & 15))) return cudaErrorInvalidValue;
+  const bool wide = a.nope > 64;
+  if (a.vdim <= 64) return wide ? launch_expanded<192, 64>(stream, a) : launch_expanded<128, 64>(stream, a);
+  return wide ? launch_expanded<192, 128>(stream, a) : launch_expanded<128, 128>(stream, a);
 }
 
 #ifdef HB_ATTN_TRACE

@@ -120,6 +120,8 @@ class Engine {
   // one step over T packed tokens of B entries; logits of the entries' last rows -> logits_ (+ sampling when `sample`);
   // n_extra > 0: logits of rows extra_rows[0..n_extra) (device indices; null = rows 0..n_extra-1) -> extra_out
   bool stack_tc(int N, int K, int lda, int ldc) const;  // stack_gemm takes a tensor-core path for this shape at any M
+  int latent_attention_tc(int T, const StepLayout& L, const hb_layer_desc& l, const StackLayerW& w,
+                          const std::vector<std::pair<int, int>>& runs);
   int forward_stack(int T, int B, const StepLayout& L, const int32_t* extra_rows, int n_extra, float* extra_out, bool sample);
   // C[M, N] (fp32, row stride ldc) = A . W^T: tcgen05 GEMM when the mode and the strides allow it (A_b16 = bf16 copy of A),
   // CUDA-core fp32 GEMM otherwise
@@ -203,6 +205,12 @@ class Engine {
     bf16 *q16 = nullptr, *ctx16 = nullptr;  // bf16 copies of the per-head queries / weighted latents (per-head tcgen05 products)
     bf16 *qabs16 = nullptr, *kbuf = nullptr, *ct = nullptr, *P = nullptr;
     float* S = nullptr;
+    // latent attention on the tensor cores (bf16 mode).  Blocks of up to 128 tokens, head-major: unrotated query parts, queries in
+    // the latent space, weighted latents, values [H][128][..]; expanded rows: gathered latents, rotated parts, per-head keys | values
+    bf16 *lat_qh = nullptr, *lat_q = nullptr, *lat_ctx = nullptr, *lat_c = nullptr, *lat_kr = nullptr, *lat_kv = nullptr;
+    float *lat_ov = nullptr, *lat_ws = nullptr;
+    int32_t* lat_heads = nullptr;  // 0, 1, 2, ...: the weights of m tile h of a per-head product
+    size_t lat_rows = 0;           // capacity in expanded rows
     int att_qb = 0;       // tokens per query block
     size_t att_rows = 0, att_keys = 0;  // capacity: score rows (tokens x heads) and key columns of one block
     // mixture of experts: router logits [T][ldz], chosen outputs and their weights [T][top_k], expert outputs [(T, top_k)][W]
@@ -218,7 +226,7 @@ class Engine {
     bf16 *moe_a16 = nullptr, *moe_h16 = nullptr, *moe_y16 = nullptr;
     int32_t* moe_scratch = nullptr;
     bf16* gu16 = nullptr;  // [gate | up] products of a gated unit as bf16 (tensor-core path of steps of > 256 tokens, experts)
-    // rotation of grouped-query layers: distinct frequency sets (device, fp64; layers with equal rotation share one), the
+    // rotation of attention layers: distinct frequency sets (device, fp64; layers with equal rotation share one), the
     // step's cos / sin table of every set, and each layer's set (-1: none)
     std::vector<const double*> freq_sets;
     std::vector<int> freq_half;

@@ -1,11 +1,14 @@
-// Layer-list decoders (HB_ARCH_STACK: the Risepel, Lurepel, Latanex and Funudra designs) inside hb::Engine: model load, the page pool's planes and recurrent state slots,
+// Layer-list decoders (HB_ARCH_STACK: the Risepel, Lurepel, Latanex, Funudra and Kamivik designs) inside hb::Engine: model load, the page pool's planes and recurrent state slots,
 // the step's forward pass and the driven-sequence entry points.  Scheduling, page bookkeeping, the step block, sampling
 // and request records are the engine's own (engine.cu); this file adds what differs from the Llama path:
 //   * the residual stream is fp32 and post-normed; every sublayer reads the stream itself;
 //   * ONE forward serves every step shape: each batch entry is a run of tokens [first, first + n) of a sequence whose
 //     earlier tokens live in the latent pool (attention) and in its state slot (recurrence), so a prompt, a portion of a
 //     prompt and a single decoded token are the same code with different n;
-//   * attention layers cache one latent row per token ([c | k_rot]); a layer may read the rows of an earlier layer;
+//   * latent-attention layers cache one row per token ([c | k_rot]); a layer may read the rows of an earlier layer.  bf16 mode: long
+//     portions expand the rows they see into per-head keys and values and run on the fused tcgen05 attention kernel, single
+//     tokens and short portions carry their queries into the latent space and attend over the cached rows themselves
+//     (attn_latent.cu); the exact mode and other shapes take the per-token kernel;
 //   * recurrent layers keep one fp32 matrix per head in a state slot; an entry that starts at position 0 starts from zero,
 //     so a slot needs no clearing when it changes hands.
 //   * grouped-query layers keep two planes of the pool (rotated unit-norm keys, raw values) in the Llama path's
@@ -27,7 +30,9 @@
 //     forms both normed inputs of the next layer from one row statistic; state-space layers and matrix memories (scalar-decay
 //     recurrences on one kernel, state and convolution inputs in the slot); a second mixer beside a grouped-query one, their
 //     output projections as one product over the concatenated inputs; layers that use an earlier layer's tensors with planes
-//     and state of their own; logits from the embedding table.
+//     and state of their own; logits from the embedding table;
+//   * parallel sublayers behind ONE norm, with gains on both outputs and a factor of their sum; a mixture's weighted rows join the
+//     same launch.
 #include "engine.h"
 #include "launch.h"
 
@@ -86,7 +91,7 @@ int Engine::load_begin_stack(const hb_stack_desc& sd, const hb_layer_desc* layer
   // no position reaches max_ctx, so a longer window sees what a window of max_ctx sees: size the kernels for the shorter one
   std::vector<hb_layer_desc> lv(layers, layers + sd.n_layers);
   for (hb_layer_desc& l : lv) {
-    if (l.mixer == HB_MIXER_LATENT && l.window > cfg_.max_ctx) l.window = cfg_.max_ctx;
+    if (l.mixer == HB_MIXER_LATENT && (l.mask == HB_MASK_CAUSAL || l.window > cfg_.max_ctx)) { l.mask = HB_MASK_WINDOW; l.window = cfg_.max_ctx; }
     if (l.mixer == HB_MIXER_GQA) {  // a block or window that no sequence outgrows is the causal mask
       if (l.mask == HB_MASK_CAUSAL || l.window >= cfg_.max_ctx) { l.mask = HB_MASK_WINDOW; l.window = cfg_.max_ctx; }
     }
@@ -165,7 +170,7 @@ static size_t stack_skinny_floats(const Model& m) {
     shape(m.sw[i].n_in, W);
     shape(W, m.sw[i].o_cols ? (size_t)m.sw[i].o_cols : (size_t)l.heads * l.vdim);
     if (l.ff > 0 && l.ff_kind == HB_FF_RELU2) shape(l.ff, W);
-    if (l.mixer == HB_MIXER_LATENT) shape((size_t)l.heads * (l.dim + l.rot_dim), l.q_rank);
+    if (l.mixer == HB_MIXER_LATENT && l.q_rank > 0) shape((size_t)l.heads * (l.dim + l.rot_dim), l.q_rank);
     if (l.ff > 0) {
       shape(2 * (size_t)l.ff, W);
       shape(W, l.ff);
@@ -182,12 +187,19 @@ static size_t stack_skinny_floats(const Model& m) {
 // Dense-product attention (bf16 mode, prompt portions of >= kAttDenseMin tokens): capacity of one query block over all
 // latent layers.  Returns false when no layer qualifies (row sizes that are not 16-byte multiples).
 constexpr int kAttDenseMin = 64;
+// Latent layers on the tensor cores: bf16 mode and head / latent sizes that both kernels take (attn_expanded, latent_decode)
+static bool latent_tc_ok(const Model& m, const hb_layer_desc& l) {
+  static const bool off = [] { const char* e = getenv("HB_STACK_LATENT_TC"); return e && atoi(e) == 0; }();
+  const int W = m.sd.width, o = l.heads * l.vdim;
+  return !off && !m.sd.compute_f32 && l.mixer == HB_MIXER_LATENT && attn_expanded_ok(l.dim, l.rot_dim, l.vdim) &&
+         latent_decode_ok(l.dim, l.kv_rank, l.rot_dim) && W % 4 == 0 && W >= 64 && o % 8 == 0 && o >= 64 && l.window > 0;
+}
 static bool stack_att_caps(const Model& m, int* qb, size_t* rows, size_t* keys, size_t* rmax, size_t* dmax, size_t* qa16) {
   *qb = 512; *rows = *keys = *rmax = *dmax = *qa16 = 0;
   if (m.sd.compute_f32) return false;
   bool any = false;
   for (const hb_layer_desc& l : m.sl) {
-    if (l.mixer != HB_MIXER_LATENT || (l.kv_rank + l.rot_dim) % 8 || l.kv_rank % 8) continue;
+    if (l.mixer != HB_MIXER_LATENT || latent_tc_ok(m, l) || (l.kv_rank + l.rot_dim) % 8 || l.kv_rank % 8) continue;
     any = true;
     int q = 512;
     while (q > 64 && (size_t)q * l.heads * (l.window + q) * 4 > (size_t(64) << 20)) q /= 2;  // scores of a block <= 64 MB
@@ -195,7 +207,7 @@ static bool stack_att_caps(const Model& m, int* qb, size_t* rows, size_t* keys, 
   }
   if (!any) return false;
   for (const hb_layer_desc& l : m.sl) {
-    if (l.mixer != HB_MIXER_LATENT || (l.kv_rank + l.rot_dim) % 8 || l.kv_rank % 8) continue;
+    if (l.mixer != HB_MIXER_LATENT || latent_tc_ok(m, l) || (l.kv_rank + l.rot_dim) % 8 || l.kv_rank % 8) continue;
     *rows = std::max(*rows, (size_t)*qb * l.heads);
     *keys = std::max(*keys, (size_t)(l.window + *qb + 7) / 8 * 8);
     *rmax = std::max(*rmax, (size_t)l.kv_rank);
@@ -216,6 +228,8 @@ struct StackDims {
   int vf = 0;                // layers that blend values: kv_heads * vdim
   bool shared = false;       // some mixture has a unit every token uses
   int cv = 0;                // widest convolved row (state-space layers, grouped-query layers with convolved projections)
+  size_t lat_qh = 0, lat_r = 0, lat_v = 0, lat_ws = 0;  // latent layers on the tensor cores: elements per head-major block / split partials
+  int lat_rank = 0, lat_rot = 0, lat_kv = 0, lat_heads = 0;  // ... and widest latent, rotated part, expanded row, most heads
   int ab = 0;                // most heads of a scalar-decay recurrence (decay, input weight, exp(-m), n . q per head and token)
 };
 // Grouped-query layers whose prompt portions run on the fused tcgen05 attention kernel (the one the Llama path uses, with
@@ -275,8 +289,21 @@ static StackDims stack_dims(const Model& m, int max_ctx) {
     } else {
       d.n2 = std::max(d.n2, l.heads * (l.dim + l.rot_dim));
       d.q = std::max(d.q, l.q_rank);
-      d.qa = std::max(d.qa, l.heads * (l.kv_rank + l.rot_dim));
-      d.cx = std::max(d.cx, std::max(l.heads * l.kv_rank, l.heads * l.vdim));
+      d.rope_half += l.rope_dims / 2;
+      if (latent_tc_ok(m, l)) {
+        const size_t rows = (size_t)l.heads * kLatentTokRows;
+        d.lat_qh = std::max(d.lat_qh, rows * l.dim);
+        d.lat_r = std::max(d.lat_r, rows * l.kv_rank);
+        d.lat_v = std::max(d.lat_v, rows * l.vdim);
+        d.lat_ws = std::max(d.lat_ws, (size_t)148 * 32 * (l.kv_rank + 2));
+        d.lat_rank = std::max(d.lat_rank, l.kv_rank);
+        d.lat_rot = std::max(d.lat_rot, l.rot_dim);
+        d.lat_kv = std::max(d.lat_kv, l.heads * (l.dim + l.vdim));
+        d.lat_heads = std::max(d.lat_heads, l.heads);
+      } else {
+        d.qa = std::max(d.qa, l.heads * (l.kv_rank + l.rot_dim));
+        d.cx = std::max(d.cx, std::max(l.heads * l.kv_rank, l.heads * l.vdim));
+      }
     }
     if (l.ff > 0 && (l.ff_kind == HB_FF_GELU_TANH || l.ff_kind == HB_FF_SILU)) d.gu = std::max(d.gu, 2 * l.ff);
     if (l.ff > 0 && l.ff_kind == HB_FF_MOE) {
@@ -310,6 +337,11 @@ size_t Engine::workspace_bytes_stack() const {
     const size_t rows = dm.moe_e > 0 ? (size_t)moe_group_max_rows((int)T * dm.moe_top, dm.moe_e) : 0;
     b += al256(std::max(T * (size_t)up8(dm.gu), rows * 2 * (size_t)dm.moe_f) * 2 + 256);
   }
+  if (dm.lat_kv > 0) {
+    const size_t rows = std::max<size_t>(T, cfg_.max_ctx);
+    b += al256(dm.lat_qh * 2) + 2 * al256(dm.lat_r * 2) + al256(dm.lat_v * 4) + al256(dm.lat_ws * 4) + al256((size_t)dm.lat_heads * 4) +
+         al256(rows * dm.lat_rank * 2) + al256(rows * dm.lat_rot * 2) + al256(rows * dm.lat_kv * 2);
+  }
   b += 2 * al256(T * W * 4) + al256(T * W * 2);                       // x, y, x16
   if (sd.norm_place == HB_NORM_BOTH_SIDES || sd.norm_place == HB_NORM_PARALLEL) b += al256(T * W * 4);     // hn
   if (sd.norm_place == HB_NORM_PARALLEL) b += al256(T * W * 4) + al256(T * W * 2);  // hn2, x16b
@@ -341,6 +373,7 @@ int Engine::alloc_runtime_stack() {
   CU(stack_moe_init());
   CU(stack_delta_init());
   CU(stack_ssm_init());
+  CU(attn_latent_init());
   if (!sd.compute_f32) {  // stream-K plans allocate on first use of a shape: make them now, not inside a graph capture
     SmLimitScope sm_scope(cfg_.sm_budget);
     SkinnyPlan pl{};
@@ -349,7 +382,7 @@ int Engine::alloc_runtime_stack() {
       CU(gemm_skinny_plan(model_.sw[i].n_in, sd.width, &pl));
       CU(gemm_skinny_plan(sd.width, model_.sw[i].o_cols ? model_.sw[i].o_cols : l.heads * l.vdim, &pl));
       if (l.ff > 0 && l.ff_kind == HB_FF_RELU2) CU(gemm_skinny_plan(l.ff, sd.width, &pl));
-      if (l.mixer == HB_MIXER_LATENT) CU(gemm_skinny_plan(l.heads * (l.dim + l.rot_dim), l.q_rank, &pl));
+      if (l.mixer == HB_MIXER_LATENT && l.q_rank > 0) CU(gemm_skinny_plan(l.heads * (l.dim + l.rot_dim), l.q_rank, &pl));
       if (l.ff > 0) {
         CU(gemm_skinny_plan(2 * l.ff, sd.width, &pl));
         CU(gemm_skinny_plan(sd.width, l.ff, &pl));
@@ -375,7 +408,7 @@ int Engine::alloc_runtime_stack() {
   const size_t T = t_cap_, W = sd.width;
   const StackDims dm = stack_dims(model_, cfg_.max_ctx);
   const int n1 = dm.n1, n2 = dm.n2, q = dm.q, qa = dm.qa, cx = dm.cx, mo = dm.mo;
-  {  // rotation frequencies of the grouped-query layers (double precision, formed on the host)
+  {  // rotation frequencies of the attention layers (double precision, formed on the host)
     double* fq = (double*)take((size_t)std::max(dm.rope_half, 1) * 8);
     float* cs = (float*)take(T * 2 * (size_t)std::max(dm.rope_half, 1) * 4);
     sk_.layer_set.assign(sd.n_layers, -1);
@@ -384,7 +417,7 @@ int Engine::alloc_runtime_stack() {
     size_t at = 0;
     for (int i = 0; i < sd.n_layers; ++i) {
       const hb_layer_desc& l = model_.sl[i];
-      if (l.mixer != HB_MIXER_GQA || l.rope_dims <= 0) continue;
+      if ((l.mixer != HB_MIXER_GQA && l.mixer != HB_MIXER_LATENT) || l.rope_dims <= 0) continue;
       const std::vector<double> f = stack_rope_freqs(l);
       size_t sidx = 0;
       while (sidx < sets.size() && sets[sidx] != f) ++sidx;
@@ -425,6 +458,23 @@ int Engine::alloc_runtime_stack() {
   if (!sd.compute_f32) {
     const size_t rows = dm.moe_e > 0 ? (size_t)moe_group_max_rows((int)T * dm.moe_top, dm.moe_e) : 0;
     sk_.gu16 = (bf16*)take(std::max(T * (size_t)up8(dm.gu), rows * 2 * (size_t)dm.moe_f) * 2 + 256);
+  }
+  if (dm.lat_kv > 0) {
+    sk_.lat_rows = std::max<size_t>(T, cfg_.max_ctx);
+    sk_.lat_qh = (bf16*)take(dm.lat_qh * 2);
+    sk_.lat_q = (bf16*)take(dm.lat_r * 2);
+    sk_.lat_ctx = (bf16*)take(dm.lat_r * 2);
+    sk_.lat_ov = (float*)take(dm.lat_v * 4);
+    sk_.lat_ws = (float*)take(dm.lat_ws * 4);
+    sk_.lat_heads = (int32_t*)take((size_t)dm.lat_heads * 4);
+    sk_.lat_c = (bf16*)take(sk_.lat_rows * dm.lat_rank * 2);
+    sk_.lat_kr = (bf16*)take(sk_.lat_rows * dm.lat_rot * 2);
+    sk_.lat_kv = (bf16*)take(sk_.lat_rows * dm.lat_kv * 2);
+    CU(cudaMemset(sk_.lat_qh, 0, dm.lat_qh * 2));  // rows of a block that a step does not fill stay finite
+    CU(cudaMemset(sk_.lat_ctx, 0, dm.lat_r * 2));
+    std::vector<int32_t> ids(dm.lat_heads);
+    for (int i = 0; i < dm.lat_heads; ++i) ids[i] = i;
+    CU(cudaMemcpy(sk_.lat_heads, ids.data(), ids.size() * 4, cudaMemcpyHostToDevice));
   }
   sk_.ld1 = up8(n1); sk_.ld2 = up8(n2); sk_.ldcq = up8(q); sk_.ldqa = up8(qa); sk_.ldctx = up8(cx); sk_.ldmo = up8(mo);
   sk_.x = (float*)take(T * W * 4);
@@ -567,6 +617,89 @@ int Engine::stack_gemm(const float* A, const bf16* A16, int lda, const void* Wt,
   return HB_OK;
 }
 
+// Latent attention of one layer on the tensor cores: k.q16 holds the rotated query heads, the step's rows are in the cache; the
+// gated heads go to k.mo16 [T][H Dv].  runs: the tokens of short entries (single tokens, portions below kAttDenseMin); the first
+// block of the first run is in k.lat_qh already.
+int Engine::latent_attention_tc(int T, const StepLayout& L, const hb_layer_desc& l, const StackLayerW& w, const std::vector<std::pair<int, int>>& runs) {
+  const int32_t* positions = (const int32_t*)(d_step_ + L.positions);
+  const int32_t* pt = (const int32_t*)(d_step_ + L.pt);
+  const int32_t* seqof = (const int32_t*)(d_step_ + L.seqof);
+  StackWs& k = sk_;
+  const int H = l.heads, Dk = l.dim, Dv = l.vdim, R = l.kv_rank, Dr = l.rot_dim, Dq = Dk + Dr;
+  const int window = l.window < cfg_.max_ctx ? l.window : 0;
+  const bool head_gate = (l.attn_flags & HB_ATTN_HEAD_GATE) != 0;
+  const bf16* cache = (const bf16*)((uint8_t*)kv_ + plane_off_[w.cache_plane]);
+  // ---- long portions: the rows each of them sees are expanded, then one attention launch per group of portions
+  LatentRuns lr{};
+  AttnRuns ar{};
+  int rows = 0;
+  double pairs = 0;
+  auto launch_group = [&]() -> int {
+    if (lr.n == 0) return HB_OK;
+    SPAN(3, 4.0 * rows * (R + Dr), latent_rows(stream_, cache, pt, max_pages_per_seq_, R, Dr, k.lat_c, k.lat_kr, lr, rows));
+    const int ldkv = H * (Dk + Dv);
+    GemmArgs g{k.lat_c, R, (const bf16*)w.uk, R, k.lat_kv, ldkv, nullptr, 0, nullptr, rows, ldkv, R, EPI_NONE, 0};
+    SPAN(0, 2.0 * rows * ldkv * R, gemm_bf16_tn(stream_, g));
+    AttnExpandedArgs ea{};
+    ea.q = k.q16; ea.ldq = H * Dq;
+    ea.k = k.lat_kv; ea.v = k.lat_kv + (size_t)H * Dk; ea.ldkv = ldkv;
+    ea.k_rot = k.lat_kr; ea.ldkr = Dr;
+    ea.out = k.mo16; ea.ldo = H * Dv;
+    ea.T = T; ea.rows = rows; ea.H = H; ea.nope = Dk; ea.rot = Dr; ea.vdim = Dv; ea.window = window; ea.scale = l.scale;
+    if (head_gate) ea.head_gate = k.p1 + w.off_g; else ea.entry_gate = k.p1 + w.off_g;
+    ea.ldg = k.ld1; ea.sink = (const bf16*)w.sink;
+    ar.n = lr.n;
+    ea.runs = ar;
+    SPAN(1, 2.0 * pairs * H * (Dq + Dv), attn_expanded(stream_, ea));
+    lr.n = 0; rows = 0; pairs = 0;
+    return HB_OK;
+  };
+  for (size_t b = 0; b < step_entries_.size(); ++b) {
+    const StepEntry& en = step_entries_[b];
+    if (en.n < kAttDenseMin) continue;
+    const int pos0 = window > 0 ? std::max(0, en.first - window + 1) : 0, kv = en.first + en.n - pos0;
+    if (lr.n == AttnRuns::kMax || (lr.n > 0 && (size_t)rows + kv > k.lat_rows)) {
+      int rc = launch_group();
+      if (rc != HB_OK) return rc;
+    }
+    lr.row0[lr.n] = ar.row0[lr.n] = rows; lr.pos0[lr.n] = pos0; lr.seq[lr.n] = (int)b;
+    ar.t0[lr.n] = en.t0; ar.len[lr.n] = en.n; ar.kv[lr.n] = kv;
+    lr.n++;
+    rows += kv;
+    pairs += window > 0 ? (double)en.n * std::min(kv, window) : (double)en.n * (en.first + 0.5 * en.n);
+  }
+  int rc = launch_group();
+  if (rc != HB_OK) return rc;
+  // ---- single tokens and short portions, in blocks of up to 128 tokens: q_h^T W_uk,h per head as one grouped product (the head's
+  // weights per 128-row m tile), attention over the cached rows, values out of the weighted latents, gate
+  bool first = true;
+  const int sms = cfg_.sm_budget > 0 ? cfg_.sm_budget : 148;
+  for (const auto& run : runs)
+    for (int t0 = run.first; t0 < run.second; t0 += kLatentTokRows) {
+      const int n = std::min(kLatentTokRows, run.second - t0), M = H * kLatentTokRows;
+      if (!first) SPAN(3, 4.0 * n * H * Dk, latent_q_heads(stream_, k.q16 + (size_t)t0 * H * Dq, H * Dq, k.lat_qh, n, H, Dk, Dr));
+      first = false;
+      GemmArgs g1{k.lat_qh, Dk, (const bf16*)w.ukT, Dk, k.lat_q, R, nullptr, 0, nullptr, M, R, Dk, EPI_NONE, 0};
+      g1.m_tile_group = k.lat_heads; g1.groups = H;
+      SPAN(0, 2.0 * M * R * Dk, gemm_bf16_tn(stream_, g1));
+      LatentDecodeArgs da{};
+      da.q_lat = k.lat_q; da.q = k.q16 + (size_t)t0 * H * Dq; da.ldq = H * Dq;
+      da.cache = cache; da.page_table = pt; da.max_pages = max_pages_per_seq_; da.page_size = page_; da.num_pages = num_pages_;
+      da.positions = positions + t0; da.seq_of = seqof + t0;
+      da.ctx = k.lat_ctx; da.workspace = k.lat_ws; da.sink = (const bf16*)w.sink;
+      da.T = n; da.H = H; da.Dk = Dk; da.R = R; da.Dr = Dr; da.window = window; da.scale = l.scale;
+      da.num_splits = latent_decode_splits(n, H, std::min(l.window, cfg_.max_ctx), sms);
+      SPAN(2, 2.0 * n * (double)std::min(l.window, cfg_.max_ctx) * (R + Dr), latent_decode(stream_, da));
+      if (da.num_splits > 1) launches_.fetch_add(1, std::memory_order_relaxed);  // combine kernel
+      GemmArgs g2{k.lat_ctx, R, (const bf16*)w.uv, R, k.lat_ov, Dv, nullptr, 0, nullptr, M, Dv, R, EPI_F32, 0};
+      g2.m_tile_group = k.lat_heads; g2.groups = H;
+      SPAN(0, 2.0 * M * Dv * R, gemm_bf16_tn(stream_, g2));
+      SPAN(3, 12.0 * n * H * Dv, latent_out_gate(stream_, k.lat_ov, Dv, (long)kLatentTokRows * Dv, k.p1 + (size_t)t0 * k.ld1 + w.off_g, k.ld1,
+                                                 head_gate, nullptr, k.mo16 + (size_t)t0 * H * Dv, n, H, Dv));
+    }
+  return HB_OK;
+}
+
 int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extra_rows, int n_extra, float* extra_out, bool sample) {
   const hb_stack_desc& sd = model_.sd;
   const bool f32 = sd.compute_f32 != 0;
@@ -592,22 +725,27 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
   // what a sublayer reads: the stream itself, or (norms on both sides, parallel sublayers) its normed copy; x16 is the bf16
   // copy of that.  With parallel sublayers the feed-forward has a normed copy of its own (hn2 / x16b).
   const float* xin = (both || par) ? k.hn : k.x;
-  const float* ff_in = par ? k.hn2 : xin;
-  const bf16* ff_in16 = par ? (f32 ? nullptr : k.x16b) : x16;
+  const bool two_norms = par && !sd.one_norm;
+  const float* ff_in = two_norms ? k.hn2 : xin;
+  const bf16* ff_in16 = two_norms ? (f32 ? nullptr : k.x16b) : x16;
+  // a mixture's router product on the tensor cores (its rows padded with zero rows to one MMA tile)
+  auto router_tc = [&](const hb_layer_desc& l) { return T > 256 && l.experts + l.identity_experts <= 64 && stack_tc(64, W, W, k.ldz) && k.ldz >= 64; };
   // parallel sublayers: x += mixer + feed-forward (+ bias), and the two normed inputs of the layer `next` (none behind the last)
-  auto par_step = [&](const float* y, const float* y2, const void* bias, float bias_scale, int next) -> cudaError_t {
+  auto par_step = [&](const float* y, const float* y2, const void* bias, float bias_scale, int next, const ParScale* scale) -> cudaError_t {
     const void* w1 = next < sd.n_layers ? model_.sw[next].norm1 : nullptr;
-    const void* w2 = next < sd.n_layers && model_.sl[next].ff > 0 ? model_.sw[next].norm2 : nullptr;
+    const void* w2 = two_norms && next < sd.n_layers && model_.sl[next].ff > 0 ? model_.sw[next].norm2 : nullptr;
     // the fp32 copies are written only where a product of the next layer reads them (shapes the tensor-core GEMMs do not take)
     bool h1_f32 = true, h2_f32 = true;
     if (next < sd.n_layers) {
       const hb_layer_desc& nl = model_.sl[next];
       const int n_in = model_.sw[next].n_in;
       h1_f32 = !stack_tc(n_in, W, W, nl.mixer == HB_MIXER_GQA ? up8(n_in) : k.ld1);
-      h2_f32 = !stack_tc(nl.ff_kind == HB_FF_RELU2 ? nl.ff : 2 * nl.ff, W, W, k.ld1);
+      if (nl.ff_kind == HB_FF_MOE) h2_f32 = f32 || nl.identity_experts > 0 || !router_tc(nl);
+      else h2_f32 = !stack_tc(nl.ff_kind == HB_FF_RELU2 ? nl.ff : 2 * nl.ff, W, W, k.ld1);
+      if (!two_norms && nl.ff > 0) h1_f32 |= h2_f32;
     }
     return parallel_step(stream_, k.x, nullptr, y, y2, bias, bias_scale, w1, w2, f32, sd.norm_eps, y ? k.x : nullptr, h1_f32 ? k.hn : nullptr, x16,
-                         h2_f32 ? k.hn2 : nullptr, f32 ? nullptr : k.x16b, T, W);
+                         h2_f32 ? k.hn2 : nullptr, f32 ? nullptr : k.x16b, T, W, scale);
   };
   // the residual step: the norm covers the sum (post-norm stream) or the sublayer's output alone; with norms on both sides
   // the same launch also norms the input of the sublayer that follows (`pre`, null behind the last one)
@@ -666,6 +804,73 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     }
     return stack_gemm(k.mo, mo16, F, w_down, W, F, out, W, T);
   };
+  // mixture of experts: out = weighted sum of the chosen experts' outputs.  fuse (parallel sublayers): where the experts ran as
+  // grouped products, their rows and weights are handed to the residual step instead and `out` is left alone
+  auto moe_ff = [&](const hb_layer_desc& l, const StackLayerW& w, float* out, ParScale* fuse) -> int {
+    // router in fp32 on the sublayer's input; experts per (token, choice); identity outputs and weights in the combination
+    const int E = l.experts, R = l.experts + l.identity_experts, F = l.ff;
+    RouteOpts ro;
+    ro.sigmoid = l.router_kind == HB_ROUTER_SIGMOID; ro.groups = l.route_groups; ro.keep = l.route_keep; ro.renorm = l.route_renorm;
+    ro.chosen = l.router_kind == HB_ROUTER_CHOSEN; ro.bias = l.route_bias;
+    ro.scale = l.route_scale != 0.f ? l.route_scale : 1.f;
+    const int eact = l.expert_kind == HB_EXPERT_CLAMPED ? GLU_CLAMPED : l.expert_kind == HB_EXPERT_GELU ? GLU_NONE_GELU : GLU_SILU;
+    const float* add = nullptr;
+    if (l.shared_ff > 0) {  // the unit every token uses; the combination below starts from its output
+      int rc = gated_ff(w.w_gu_sh, w.w_down_sh, l.shared_ff, eact, l.shared_limit, w.sh_packed, k.y2);
+      if (rc != HB_OK) return rc;
+      add = k.y2;
+    }
+    if (router_tc(l)) {
+      // steps of many tokens: logits on the tensor cores from the bf16 copy of the stream (fp32 accumulation; the router's
+      // rows are padded with zero rows to one MMA tile), then the choice in fp32
+      GemmArgs g{ff_in16, W, (const bf16*)w.router, W, k.moe_z, k.ldz, nullptr, 0, nullptr, T, 64, W, EPI_F32, 0};
+      SPAN(0, 2.0 * T * 64 * W, gemm_bf16_tn(stream_, g));
+      SPAN(3, 8.0 * T * R, moe_route(stream_, k.moe_z, k.ldz, w.correction, f32, R, l.top_k, k.moe_ids, k.moe_w, T, ro));
+    } else if (moe_router_smem(R, W, f32) <= 200 * 1024) {
+      SPAN(3, 4.0 * T * W, moe_router(stream_, ff_in, w.router, w.correction, f32, R, W, l.top_k, k.moe_ids, k.moe_w, T,
+                                      cfg_.sm_budget > 0 ? cfg_.sm_budget : 148, ro));
+    } else {  // a router too large for shared memory: product, then choice
+      GemmRtArgs g{ff_in, W, 0, w.router, W, 1, 0, k.moe_z, k.ldz, 0, nullptr, T, R, W, 1, f32};
+      SPAN(5, 2.0 * T * R * W, gemm_rt(stream_, g));
+      SPAN(3, 8.0 * T * R, moe_route(stream_, k.moe_z, k.ldz, w.correction, f32, R, l.top_k, k.moe_ids, k.moe_w, T, ro));
+    }
+    const int items = T * l.top_k;
+    if (moe_grouped_ok(model_, l) && k.moe_a16 && items >= 2 * E) {
+      // items sorted by expert into 128-row segments; both products of every expert in two grouped tcgen05 launches
+      const int rows = moe_group_max_rows(items, E);
+      SPAN(3, 12.0 * items, moe_group_rows(stream_, k.moe_ids, items, l.top_k, E, k.moe_row_of, k.moe_src, k.moe_tiles, k.moe_scratch));
+      if (items > 4096) launches_.fetch_add(2, std::memory_order_relaxed);  // three kernels behind one call
+      SPAN(3, 4.0 * rows * W, moe_gather_rows(stream_, ff_in16, W, k.moe_src, k.moe_a16, rows));
+      if (eact == GLU_NONE_GELU) {  // ungated units: gelu on the accumulators' way out
+        GemmArgs g1{k.moe_a16, W, (const bf16*)w.w_gu, W, k.moe_h16, F, nullptr, 0, nullptr, rows, F, W, EPI_GELU, 0};
+        g1.m_tile_group = k.moe_tiles; g1.groups = E;
+        SPAN(0, 2.0 * rows * F * W, gemm_bf16_tn(stream_, g1));
+      } else if (w.gu_packed) {  // silu(gate) * up on the accumulators' way out
+        GemmArgs g1{k.moe_a16, W, (const bf16*)w.w_gu, W, k.moe_h16, F, nullptr, 0, nullptr, rows, 2 * F, W,
+                    eact == GLU_CLAMPED ? EPI_CLAMPGLU : EPI_SWIGLU, 0};
+        g1.m_tile_group = k.moe_tiles; g1.groups = E; g1.glu_limit = l.ff_limit;
+        SPAN(0, 4.0 * rows * F * W, gemm_bf16_tn(stream_, g1));
+      } else {
+        GemmArgs g1{k.moe_a16, W, (const bf16*)w.w_gu, W, k.gu16, 2 * F, nullptr, 0, nullptr, rows, 2 * F, W, EPI_NONE, 0};
+        g1.m_tile_group = k.moe_tiles; g1.groups = E;
+        SPAN(0, 4.0 * rows * F * W, gemm_bf16_tn(stream_, g1));
+        SPAN(3, 6.0 * rows * F, gated_unit_b16(stream_, k.gu16, 2 * F, eact, k.moe_h16, rows, F, l.ff_limit));
+      }
+      GemmArgs g2{k.moe_h16, F, (const bf16*)w.w_down, F, k.moe_y16, W, nullptr, 0, nullptr, rows, W, F, EPI_NONE, 0};
+      g2.m_tile_group = k.moe_tiles; g2.groups = E;
+      SPAN(0, 2.0 * rows * F * W, gemm_bf16_tn(stream_, g2));
+      if (fuse && l.identity_experts == 0 && !add) {  // the residual step sums the rows itself
+        fuse->rows = k.moe_y16; fuse->row_of = k.moe_row_of; fuse->wts = k.moe_w; fuse->top_k = l.top_k;
+      } else {
+        SPAN(3, 2.0 * T * (l.top_k + 4) * W, moe_combine_rows(stream_, ff_in, k.moe_y16, k.moe_row_of, k.moe_w, l.top_k, out, T, W, add));
+      }
+    } else {
+      SPAN(5, 6.0 * items * F * W, moe_expert_rows(stream_, ff_in, ff_in16, w.w_gu, w.w_down, f32, k.moe_ids, l.top_k, E, F, W, k.moe_y, T, w.gu_packed,
+                                                   eact, l.ff_limit));
+      SPAN(3, 4.0 * T * (l.top_k + 2) * W, moe_combine(stream_, ff_in, k.moe_y, k.moe_ids, k.moe_w, l.top_k, E, out, T, W, add));
+    }
+    return HB_OK;
+  };
   // a matrix memory over the columns of the layer's fused projection (row stride ldin): gates and their running maximum,
   // the recurrence, then normalisation, per-head unit RMS, gain, sigmoid gate and `scale` into columns col0.. of the output
   // projection's input (row stride ldout)
@@ -696,7 +901,7 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
   SPAN(3, rowb, embed_rows_f32(stream_, tokens, model_.s_embed, f32, k.x, x16, T, W, sd.embed_scale != 0.f ? sd.embed_scale : 1.f));
   if (sd.embed_norm) SPAN(3, 2 * rowb, norm_rows(k.x, nullptr, model_.s_embed_norm, k.x, both ? nullptr : x16, T));
   if (both) SPAN(3, 2 * rowb, norm_rows(k.x, nullptr, model_.sw[0].norm1, k.hn, x16, T));
-  if (par) SPAN(3, 3 * rowb, par_step(nullptr, nullptr, nullptr, 0.f, 0));
+  if (par) SPAN(3, 3 * rowb, par_step(nullptr, nullptr, nullptr, 0.f, 0, nullptr));
   for (size_t si = 0; si < k.freq_sets.size(); ++si)  // cos / sin of the step's positions, once per distinct rotation
     SPAN(3, 8.0 * T * k.freq_half[si], stack_rope_table(stream_, positions, k.freq_sets[si], k.freq_half[si], k.rope_cs[si], T));
   for (int i = 0; i < sd.n_layers; ++i) {
@@ -894,15 +1099,46 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     } else {
       const int R = l.kv_rank, Dr = l.rot_dim, Q = l.q_rank;
       uint8_t* plane = (uint8_t*)kv_ + plane_off_[w.cache_plane];
+      const bool head_gate = (l.attn_flags & HB_ATTN_HEAD_GATE) != 0;
+      const bool tc = latent_tc_ok(model_, l) && k.lat_kv && page_ == 64 && stack_tc(W, H * Dv, H * Dv, W);
+      // tokens that attend over the latent rows themselves: runs of neighbouring entries below kAttDenseMin tokens
+      std::vector<std::pair<int, int>> runs;
+      if (tc)
+        for (const StepEntry& en : step_entries_) {
+          if (en.n >= kAttDenseMin) continue;
+          if (!runs.empty() && runs.back().second == en.t0) runs.back().second = en.t0 + en.n;
+          else runs.emplace_back(en.t0, en.t0 + en.n);
+        }
       LatentPrepArgs pa{};
       pa.p = k.p1; pa.ldp = k.ld1; pa.q_off = w.off_dq; pa.kv_off = w.off_dkv;
       pa.wq = w.dq_norm; pa.wkv = w.dkv_norm; pa.f32 = f32; pa.eps = sd.norm_eps;
       pa.cq = k.cq; pa.cq_b16 = cq16; pa.Q = Q;
-      pa.cache = plane; pa.slots = slots; pa.positions = positions;
-      pa.R = R; pa.Dr = Dr; pa.rope_dims = l.rope_dims; pa.rope_base = l.rope_base; pa.T = T;
-      SPAN(3, 8.0 * T * (Q + R + Dr), latent_prep(stream_, pa));
-      rc = stack_gemm(k.cq, cq16, Q, w.uq, H * (Dk + Dr), Q, k.p2, k.ld2, T);
-      if (rc != HB_OK) return rc;
+      pa.cache = plane; pa.slots = slots;
+      pa.cs = k.layer_set[i] >= 0 ? k.rope_cs[k.layer_set[i]] : nullptr; pa.rope_dims = l.rope_dims; pa.pairing = l.rope_pairing;
+      pa.R = R; pa.Dr = Dr; pa.T = T; pa.H = H; pa.Dk = Dk;
+      auto q_rows = [&](LatentPrepArgs& q) {  // query heads as bf16, those of the first run's first block also head by head
+        q.q16 = k.q16;
+        if (!runs.empty()) { q.qh = k.lat_qh; q.qh_t0 = runs[0].first; }
+      };
+      if (tc && Q == 0) q_rows(pa);
+      SPAN(3, 8.0 * T * (Q + R + Dr) + (pa.q16 ? 6.0 * T * H * (Dk + Dr) : 0.0), latent_prep(stream_, pa));
+      const float* qsrc = k.p1 + w.off_q;  // the queries [T][H (Dk + Dr)]
+      int ldqs = k.ld1;
+      if (Q > 0) {
+        rc = stack_gemm(k.cq, cq16, Q, w.uq, H * (Dk + Dr), Q, k.p2, k.ld2, T);
+        if (rc != HB_OK) return rc;
+        qsrc = k.p2; ldqs = k.ld2;
+        if (tc) {
+          LatentPrepArgs pq = pa;
+          pq.p = k.p2; pq.ldp = k.ld2; pq.q_off = 0; pq.kv_off = -1; pq.Q = 0;
+          q_rows(pq);
+          SPAN(3, 6.0 * T * H * (Dk + Dr), latent_prep(stream_, pq));
+        }
+      }
+      if (tc) {
+        rc = latent_attention_tc(T, L, l, w, runs);
+        if (rc != HB_OK) return rc;
+      } else {
       const int D = R + Dr, ldqa = H * D, ldcx = H * R;  // (token, head) rows are contiguous: row stride D / R
       // keys are never expanded: q_h is carried into the latent space instead (q_h^T W_uk,h), one product per head —
       // on the tensor cores for steps of many tokens (bf16 copy of q, W_uk transposed per head at load), else one batched
@@ -910,17 +1146,17 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
       const bool head_tc = !f32 && T > 256 && w.ukT && k.q16 && (Dk + Dr) % 8 == 0 && Dk % 8 == 0 && Dk >= 64 && R % 8 == 0 &&
                            R >= 64 && D % 4 == 0 && Dv % 4 == 0 && Dv >= 64 && !getenv("HB_STACK_SIMT");
       if (head_tc) {
-        SPAN(3, 6.0 * T * H * (Dk + Dr), to_bf16_rows(stream_, k.p2, k.ld2, k.q16, k.ld2, T, H * (Dk + Dr)));
+        SPAN(3, 6.0 * T * H * (Dk + Dr), to_bf16_rows(stream_, qsrc, ldqs, k.q16, k.ld2, T, H * (Dk + Dr)));
         for (int h = 0; h < H; ++h) {
           GemmArgs g{k.q16 + (size_t)h * (Dk + Dr), k.ld2, (const bf16*)w.ukT + (size_t)h * R * Dk, Dk, k.qabs + (size_t)h * D, ldqa,
                      nullptr, 0, nullptr, T, R, Dk, EPI_F32, 0};
           SPAN(0, 2.0 * T * R * Dk, gemm_bf16_tn(stream_, g));
         }
       } else {
-        GemmRtArgs g{k.p2, k.ld2, (long)(Dk + Dr), w.uk, 1, (long)R, (long)Dk * R, k.qabs, ldqa, (long)D, nullptr, T, R, Dk, H, f32};
+        GemmRtArgs g{qsrc, ldqs, (long)(Dk + Dr), w.uk, 1, (long)R, (long)Dk * R, k.qabs, ldqa, (long)D, nullptr, T, R, Dk, H, f32};
         SPAN(5, 2.0 * T * H * Dk * R, gemm_rt(stream_, g));
       }
-      SPAN(3, 8.0 * T * H * Dr, latent_q_rope(stream_, k.p2, k.ld2, k.qabs, ldqa, positions, T, H, Dk, Dr, R, l.rope_dims, l.rope_base));
+      SPAN(3, 8.0 * T * H * Dr, latent_q_rope(stream_, qsrc, ldqs, k.qabs, ldqa, pa.cs, T, H, Dk, Dr, R, l.rope_dims, l.rope_pairing));
       // Long prompt portions (bf16 mode): scores and weighted latents as two tcgen05 products per block of att_qb tokens over
       // the block's gathered keys, softmax (mask, sink) between them.  Everything else — single tokens, short portions, the
       // exact mode — goes through the per-token kernel.  Both read the same cache rows, written by latent_prep above.
@@ -982,7 +1218,8 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
         GemmRtArgs g{k.ctx, ldcx, (long)R, w.uv, (long)R, 1, (long)Dv * R, ov, ldov, (long)Dv, nullptr, T, Dv, R, H, f32};
         SPAN(5, 2.0 * T * H * Dv * R, gemm_rt(stream_, g));
       }
-      SPAN(3, 12.0 * T * H * Dv, sigmoid_gate(stream_, ov, ldov, k.p1 + w.off_g, k.ld1, k.mo, mo16, T, H * Dv));
+      SPAN(3, 12.0 * T * H * Dv, latent_out_gate(stream_, ov, ldov, Dv, k.p1 + w.off_g, k.ld1, head_gate, k.mo, mo16, T, H, Dv));
+      }
     }
     rc = stack_gemm(k.mo, mo16, ocols, w.wo, W, ocols, k.y, W, T);
     if (rc != HB_OK) return rc;
@@ -990,13 +1227,16 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
       // both sublayers read the same stream: the feed-forward runs on its own normed copy, one launch adds both outputs
       // (and the first mixer's output bias, times that mixer's weight) and norms the next layer's inputs
       const float* y2 = nullptr;
+      ParScale scale;
+      scale.s1 = w.ls1; scale.s2 = w.ls2; scale.m = sd.resid_mult != 0.f ? sd.resid_mult : 1.f;
       if (l.ff > 0) {
-        if (l.ff_kind == HB_FF_RELU2) rc = relu2_ff(w.w_gu, w.w_down, l.ff, k.y2);
+        if (l.ff_kind == HB_FF_MOE) rc = moe_ff(l, w, k.y2, &scale);
+        else if (l.ff_kind == HB_FF_RELU2) rc = relu2_ff(w.w_gu, w.w_down, l.ff, k.y2);
         else rc = gated_ff(w.w_gu, w.w_down, l.ff, l.ff_kind == HB_FF_SILU ? GLU_SILU : GLU_GELU_TANH, 0.f, w.gu_packed, k.y2);
         if (rc != HB_OK) return rc;
-        y2 = k.y2;
+        y2 = scale.top_k > 0 ? nullptr : k.y2;
       }
-      SPAN(3, 5 * rowb, par_step(k.y, y2, w.o_bias, l.mix_scale != 0.f ? l.mix_scale : 1.f, i + 1));
+      SPAN(3, 5 * rowb, par_step(k.y, y2, w.o_bias, l.mix_scale != 0.f ? l.mix_scale : 1.f, i + 1, &scale));
       continue;
     }
     SPAN(3, 3 * rowb, resid(w.o_bias, both ? w.norm1b : w.norm1, l.ff > 0 ? w.norm2 : pre_next));
@@ -1005,59 +1245,8 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
       if (rc != HB_OK) return rc;
       SPAN(3, 3 * rowb, resid(nullptr, both ? w.norm2b : w.norm2, pre_next));
     } else if (l.ff > 0 && l.ff_kind == HB_FF_MOE) {
-      // router in fp32 on the stream itself; experts per (token, choice); identity outputs and weights in the combination
-      const int E = l.experts, R = l.experts + l.identity_experts, F = l.ff;
-      RouteOpts ro;
-      ro.sigmoid = l.router_kind == HB_ROUTER_SIGMOID; ro.groups = l.route_groups; ro.keep = l.route_keep; ro.renorm = l.route_renorm;
-      ro.scale = l.route_scale != 0.f ? l.route_scale : 1.f;
-      const int eact = l.expert_kind == HB_EXPERT_CLAMPED ? GLU_CLAMPED : GLU_SILU;
-      const float* add = nullptr;
-      if (l.shared_ff > 0) {  // the unit every token uses; the combination below starts from its output
-        rc = gated_ff(w.w_gu_sh, w.w_down_sh, l.shared_ff, eact, l.shared_limit, w.sh_packed, k.y2);
-        if (rc != HB_OK) return rc;
-        add = k.y2;
-      }
-      if (T > 256 && R <= 64 && stack_tc(64, W, W, k.ldz) && k.ldz >= 64) {
-        // steps of many tokens: logits on the tensor cores from the bf16 copy of the stream (fp32 accumulation; the router's
-        // rows are padded with zero rows to one MMA tile), then the choice in fp32
-        GemmArgs g{x16, W, (const bf16*)w.router, W, k.moe_z, k.ldz, nullptr, 0, nullptr, T, 64, W, EPI_F32, 0};
-        SPAN(0, 2.0 * T * 64 * W, gemm_bf16_tn(stream_, g));
-        SPAN(3, 8.0 * T * R, moe_route(stream_, k.moe_z, k.ldz, w.correction, f32, R, l.top_k, k.moe_ids, k.moe_w, T, ro));
-      } else if (moe_router_smem(R, W, f32) <= 200 * 1024) {
-        SPAN(3, 4.0 * T * W, moe_router(stream_, xin, w.router, w.correction, f32, R, W, l.top_k, k.moe_ids, k.moe_w, T,
-                                        cfg_.sm_budget > 0 ? cfg_.sm_budget : 148, ro));
-      } else {  // a router too large for shared memory: product, then choice
-        GemmRtArgs g{xin, W, 0, w.router, W, 1, 0, k.moe_z, k.ldz, 0, nullptr, T, R, W, 1, f32};
-        SPAN(5, 2.0 * T * R * W, gemm_rt(stream_, g));
-        SPAN(3, 8.0 * T * R, moe_route(stream_, k.moe_z, k.ldz, w.correction, f32, R, l.top_k, k.moe_ids, k.moe_w, T, ro));
-      }
-      const int items = T * l.top_k;
-      if (moe_grouped_ok(model_, l) && k.moe_a16 && items >= 2 * E) {
-        // items sorted by expert into 128-row segments; both products of every expert in two grouped tcgen05 launches
-        const int rows = moe_group_max_rows(items, E);
-        SPAN(3, 12.0 * items, moe_group_rows(stream_, k.moe_ids, items, l.top_k, E, k.moe_row_of, k.moe_src, k.moe_tiles, k.moe_scratch));
-        if (items > 4096) launches_.fetch_add(2, std::memory_order_relaxed);  // three kernels behind one call
-        SPAN(3, 4.0 * rows * W, moe_gather_rows(stream_, x16, W, k.moe_src, k.moe_a16, rows));
-        if (w.gu_packed) {  // silu(gate) * up on the accumulators' way out
-          GemmArgs g1{k.moe_a16, W, (const bf16*)w.w_gu, W, k.moe_h16, F, nullptr, 0, nullptr, rows, 2 * F, W,
-                      eact == GLU_CLAMPED ? EPI_CLAMPGLU : EPI_SWIGLU, 0};
-          g1.m_tile_group = k.moe_tiles; g1.groups = E; g1.glu_limit = l.ff_limit;
-          SPAN(0, 4.0 * rows * F * W, gemm_bf16_tn(stream_, g1));
-        } else {
-          GemmArgs g1{k.moe_a16, W, (const bf16*)w.w_gu, W, k.gu16, 2 * F, nullptr, 0, nullptr, rows, 2 * F, W, EPI_NONE, 0};
-          g1.m_tile_group = k.moe_tiles; g1.groups = E;
-          SPAN(0, 4.0 * rows * F * W, gemm_bf16_tn(stream_, g1));
-          SPAN(3, 6.0 * rows * F, gated_unit_b16(stream_, k.gu16, 2 * F, eact, k.moe_h16, rows, F, l.ff_limit));
-        }
-        GemmArgs g2{k.moe_h16, F, (const bf16*)w.w_down, F, k.moe_y16, W, nullptr, 0, nullptr, rows, W, F, EPI_NONE, 0};
-        g2.m_tile_group = k.moe_tiles; g2.groups = E;
-        SPAN(0, 2.0 * rows * F * W, gemm_bf16_tn(stream_, g2));
-        SPAN(3, 2.0 * T * (l.top_k + 4) * W, moe_combine_rows(stream_, xin, k.moe_y16, k.moe_row_of, k.moe_w, l.top_k, k.y, T, W, add));
-      } else {
-        SPAN(5, 6.0 * items * F * W, moe_expert_rows(stream_, xin, x16, w.w_gu, w.w_down, f32, k.moe_ids, l.top_k, E, F, W, k.moe_y, T, w.gu_packed,
-                                                     eact, l.ff_limit));
-        SPAN(3, 4.0 * T * (l.top_k + 2) * W, moe_combine(stream_, xin, k.moe_y, k.moe_ids, k.moe_w, l.top_k, E, k.y, T, W, add));
-      }
+      rc = moe_ff(l, w, k.y, nullptr);
+      if (rc != HB_OK) return rc;
       SPAN(3, 3 * rowb, resid(nullptr, both ? w.norm2b : w.norm2, pre_next));
     } else if (l.ff > 0 && (l.ff_kind == HB_FF_GELU_TANH || l.ff_kind == HB_FF_SILU)) {
       rc = gated_ff(w.w_gu, w.w_down, l.ff, l.ff_kind == HB_FF_SILU ? GLU_SILU : GLU_GELU_TANH, 0.f, w.gu_packed, k.y);

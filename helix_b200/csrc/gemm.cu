@@ -423,7 +423,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 }
               }
             }
-            if constexpr (EPI == EPI_BIAS_GELU) {
+            if constexpr (EPI == EPI_BIAS_GELU || EPI == EPI_GELU) {
 #pragma unroll
               for (int j = 0; j < 32; j += 2) gelu_erf2(f[j], f[j + 1]);
             }
@@ -604,6 +604,7 @@ cudaError_t gemm_init() {
   if ((e = set_attr_epi<EPI_GEGLU>()) != cudaSuccess) return e;
   if ((e = set_attr_epi<EPI_CLAMPGLU>()) != cudaSuccess) return e;
   if ((e = set_attr_epi<EPI_RELU2>()) != cudaSuccess) return e;
+  if ((e = set_attr_epi<EPI_GELU>()) != cudaSuccess) return e;
   return set_attr_epi<EPI_SWIGLU>();
 }
 
@@ -651,6 +652,7 @@ cudaError_t gemm_bf16_tn(cudaStream_t stream, const GemmArgs& g) {
     }
     case EPI_F32: return launch_epi<EPI_F32>(stream, g, sms);
     case EPI_RELU2: return launch_epi<EPI_RELU2>(stream, g, sms);
+    case EPI_GELU: return launch_epi<EPI_GELU>(stream, g, sms);
     case EPI_ROPE: {
       const RopeEpi& r = g.rope;
       if ((g.N % 256) || !r.out || !r.cs || (r.D != 64 && r.D != 128) || g.N != (r.Hq + 2 * r.Hkv) * r.D || (r.ldc % 8)) return cudaErrorInvalidValue;

@@ -30,6 +30,7 @@ enum Epi : int {
   EPI_CLAMPGLU = 9,    // as EPI_SWIGLU with g = min(gate_j, limit), u = clamp(up_j, -limit, limit): g sigmoid(1.702 g) (u + 1)
                        // (limit = GemmArgs::glu_limit)
   EPI_RELU2 = 10,      // C = relu(acc)^2                      (bf16)
+  EPI_GELU = 11,       // C = gelu_erf(acc)                    (bf16)
   EPI_ROPE = 7,        // fused QKV projection of a decoder: C = bf16(acc [+ bias]) with the q and k heads rotated
                        // (RopeEpi) and the k / v rows also scattered into the paged KV cache
 };
@@ -138,6 +139,29 @@ struct AttnPrefillArgs {
   const bf16* sink = nullptr;
 };
 cudaError_t attn_prefill(cudaStream_t stream, const AttnPrefillArgs& a);
+// The same kernel for latent attention over EXPANDED rows (long prompt portions): per cached position a row [k_0 .. k_(H-1) |
+// v_0 .. v_(H-1)] made from its latent, and one rotated key part shared by all heads.  Run b: q rows [t0, t0 + len) of the packed
+// activation are the last `len` of the kv rows [row0, row0 + kv); causal, optionally the last `window` positions only.
+struct AttnRuns {
+  static constexpr int kMax = 32;
+  int n;
+  int t0[kMax], len[kMax], kv[kMax], row0[kMax];
+};
+struct AttnExpandedArgs {
+  const bf16* q; int ldq;            // [T, H * (nope + rot)], rotated part last in every head
+  const bf16* k; const bf16* v; int ldkv;  // [rows, >= H * nope], [rows, >= H * vdim] (row stride shared)
+  const bf16* k_rot; int ldkr;       // [rows, rot]
+  bf16* out; int ldo;                // [T, H * vdim]
+  int T, rows, H, nope, rot, vdim, window;  // window 0: causal
+  float scale;
+  const float* head_gate = nullptr;  // optional sigmoid gates, row stride ldg: one per head, or one per output entry
+  const float* entry_gate = nullptr;
+  int ldg = 0;
+  const bf16* sink = nullptr;        // [H] learned logits whose exponential joins the denominator
+  AttnRuns runs;
+};
+bool attn_expanded_ok(int nope, int rot, int vdim);  // shapes it takes (multiples of 8 up to 128 / 64 / 128)
+cudaError_t attn_expanded(cudaStream_t stream, const AttnExpandedArgs& a);
 // test-only CUDA-core checker, fp32 output [T, ldo]
 cudaError_t attn_naive_check(cudaStream_t stream, const AttnPrefillArgs& a, float* out_f32);
 
@@ -330,28 +354,42 @@ cudaError_t headnorm_silu_gate(cudaStream_t s, const float* o, long ldo, const f
 
 // ---- latent attention: the cache keeps, per token, the normed latent c [R] and one rotated key part [Dr] shared by all
 //      heads (row = [c | k_rot], R + Dr elements, page-major: row index = page * page_size + offset).
-// From the fused down-projection p[t] = [dq (Q) | dkv (R + Dr) | ...]: cq = rmsnorm(dq) * wq; c = rmsnorm(dkv[:R]) * wkv and
-// k_rot = rotate(dkv[R:], pos) written to cache row slots[t].  kv_off < 0: the layer reads another layer's cache (no write).
+// From the fused projection p[t] = [dq (Q) or the queries | dkv (R + Dr) | ...]:
+//   Q > 0: cq = rmsnorm(dq) * wq (fp32 + bf16 copy);
+//   kv_off >= 0: c = rmsnorm(dkv[:R]) * wkv and k_rot = rotate(dkv[R:]) written to cache row slots[t] (kv_off < 0: the layer reads
+//   another layer's cache);
+//   q16: query rows [H][Dk + Dr] starting at column q_off (Q == 0), rotated parts turned, as bf16 rows [T][H * (Dk + Dr)]; qh: the
+//   unrotated parts of tokens qh_t0 .. qh_t0 + kLatentTokRows - 1 also head by head, [H][kLatentTokRows][Dk].
+// cs: the step's rotation table (stack_rope_table; pairing as in GqaPrepArgs), null when nothing rotates.
+constexpr int kLatentTokRows = 128;  // tokens per block of head-major rows (one m tile of the grouped per-head products)
 struct LatentPrepArgs {
   const float* p; long ldp; int q_off, kv_off;
   const void* wq; const void* wkv; bool f32;
   float eps;
   float* cq; bf16* cq_b16; int Q;
-  void* cache; const int32_t* slots; const int32_t* positions;
-  int R, Dr, rope_dims; float rope_base;
+  void* cache; const int32_t* slots;
+  int R, Dr; const float* cs; int rope_dims, pairing;
   int T;
+  bf16* q16 = nullptr; int H = 0, Dk = 0;
+  bf16* qh = nullptr; int qh_t0 = 0;
 };
 cudaError_t latent_prep(cudaStream_t s, const LatentPrepArgs& a);
-// qabs[t, h, R:R+Dr] = rotate(q[t, h, Dk:Dk+Dr], pos)   (the absorbed part qabs[t, h, :R] comes from a batched GEMM with W_uk)
-cudaError_t latent_q_rope(cudaStream_t s, const float* q, long ldq, float* qabs, long ldqa, const int32_t* positions, int T, int H,
-                          int Dk, int Dr, int R, int rope_dims, float rope_base);
-// Sliding-window attention of every head over the shared latent rows, softmax with a per-head sink in the denominator:
-// ctx[t, h, :] = sum_j p_j c_j,  p_j = exp(s_j - m) / (sum_i exp(s_i - m) + exp(sink_h - m)),
+// qabs[t, h, R:R+Dr] = rotate(q[t, h, Dk:Dk+Dr])   (the absorbed part qabs[t, h, :R] comes from a batched GEMM with W_uk)
+cudaError_t latent_q_rope(cudaStream_t s, const float* q, long ldq, float* qabs, long ldqa, const float* cs, int T, int H, int Dk, int Dr,
+                          int R, int rope_dims, int pairing);
+// Attention of every head over the latent rows a position sees (the last `window` ones), softmax with an optional per-head sink
+// in the denominator, keys in blocks of kLatentKeyBlock with a running maximum:
+// ctx[t, h, :] = sum_j p_j c_j,  p_j = exp(s_j - m) / (sum_i exp(s_i - m) (+ exp(sink_h - m))),
 // s_j = scale * qabs[t, h] . [c_j | k_rot_j] over 0 <= pos_t - j < window.
+constexpr int kLatentKeyBlock = 4096;
+inline size_t latent_attn_smem(int R, int Dr, int window) {
+  const size_t keys = window < kLatentKeyBlock ? window : kLatentKeyBlock;
+  return (4 * (size_t)((R + Dr + 3) / 4 * 4) + 4 * (size_t)R + 5 * keys + 8 * 1024 + 32 * 4) * 4;
+}
 struct LatentAttnArgs {
   const float* qabs; long ldqa;     // [T, H*(R+Dr)]
   const void* cache; bool f32;      // [rows][R+Dr]
-  const void* sink;                 // [H] weight type
+  const void* sink;                 // [H] weight type, or null
   const int32_t* page_table; int max_pages, page_size;
   const int32_t* positions;         // [T]
   const int32_t* seq_of;            // [T] batch entry of each token
@@ -360,6 +398,36 @@ struct LatentAttnArgs {
   float scale;
 };
 cudaError_t latent_attn(cudaStream_t s, const LatentAttnArgs& a);
+// The same for up to kLatentTokRows tokens on the tensor cores (attn_latent.cu; bf16 rows): q_lat [H][kLatentTokRows][R] = queries
+// carried into the latent space, q [T, H * (Dk + Dr)] for their rotated parts; ctx [H][kLatentTokRows][R].  window 0: causal.
+struct LatentDecodeArgs {
+  const bf16* q_lat; const bf16* q; int ldq;
+  const bf16* cache;
+  const int32_t* page_table; int max_pages, page_size, num_pages;
+  const int32_t* positions; const int32_t* seq_of;
+  bf16* ctx;
+  float* workspace;                 // latent_decode_ws_floats(T, H, R, num_splits)
+  const bf16* sink;                 // [H] or null
+  int T, H, Dk, R, Dr, window, num_splits;
+  float scale;
+};
+bool latent_decode_ok(int Dk, int R, int Dr);
+int latent_decode_splits(int T, int H, int max_keys, int sms);
+size_t latent_decode_ws_floats(int T, int H, int R, int splits);
+cudaError_t attn_latent_init();
+cudaError_t latent_decode(cudaStream_t s, const LatentDecodeArgs& a);
+// Rows to expand: run b covers positions pos0 .. of batch entry seq, its rows start at row0 (ascending, dense).
+struct LatentRuns {
+  int n;
+  int row0[32], pos0[32], seq[32];
+};
+cudaError_t latent_rows(cudaStream_t s, const bf16* cache, const int32_t* page_table, int max_pages, int R, int Dr, bf16* c, bf16* k_rot,
+                        const LatentRuns& runs, int rows);
+// qh[h][t][:] = the unrotated part of q[t]'s head h (t < T <= kLatentTokRows)
+cudaError_t latent_q_heads(cudaStream_t s, const bf16* q, int ldq, bf16* qh, int T, int H, int Dk, int Dr);
+// out[t, h Dv + i] = o[t * o_ts + h * o_hs + i] * sigmoid(g[t, per_head ? h : h Dv + i])   (fp32 in, fp32 + bf16 copy out)
+cudaError_t latent_out_gate(cudaStream_t s, const float* o, long o_ts, long o_hs, const float* g, long ldg, bool per_head, float* out,
+                            bf16* out_b16, int T, int H, int Dv);
 // The same attention as three dense products for a block of consecutive tokens of ONE sequence (long prompt portions in the
 // bf16 mode; the two products run on the tcgen05 GEMM):
 //   latent_gather:  kbuf[jj] = cache row of position k0 + jj (jj < nk), ct[r][jj] = its latent entry r (columns nk..ldk zero)
@@ -373,8 +441,6 @@ cudaError_t latent_softmax(cudaStream_t s, const float* S, bf16* P, int ld, int 
                            float scale, const bf16* sink);
 // dst[h][r][d] = src[h][d][r] (bf16): the key up-projection per head, transposed once at load time
 cudaError_t transpose_heads_bf16(cudaStream_t s, const bf16* src, bf16* dst, int H, int Dk, int R);
-// out = o * sigmoid(g)
-cudaError_t sigmoid_gate(cudaStream_t s, const float* o, long ldo, const float* g, long ldg, float* out, bf16* out_b16, int T, int N);
 // f32 -> bf16 copy of a [T, N] block (row strides lds / ldd)
 cudaError_t to_bf16_rows(cudaStream_t s, const float* src, long lds, bf16* dst, long ldd, int T, int N);
 
@@ -530,10 +596,17 @@ cudaError_t gate_scale_rows(cudaStream_t s, const float* in, const bf16* in_b16,
                             float* out, bf16* out_b16, long ldout, int col0, int T, int n);
 // Sublayers that read the same stream and are added in one step:
 //   v = x[row_index ? row_index[r] : r] (+ y[r]) (+ y2[r]) (+ bias_scale * bias);  x_out[r] = v (when given; may be x);
+//   with ParScale: v = x + m (s1 * y[r] + s2 * y2[r]), gains s1 / s2 [W] of the weight type (null: ones) and the factor m; y2 may
+//   then come as a mixture's rows instead: y2[r] = sum_k wts[r, k] * rows[row_of[r, k]] (bf16 expert outputs, summed in order of k);
 //   h1[r] = v / rms(v) * w1, h2[r] = v / rms(v) * w2 as fp32 and / or bf16 (each optional): one statistic serves both norms
+struct ParScale {
+  const void* s1 = nullptr; const void* s2 = nullptr;
+  float m = 1.f;
+  const bf16* rows = nullptr; const int32_t* row_of = nullptr; const float* wts = nullptr; int top_k = 0;
+};
 cudaError_t parallel_step(cudaStream_t s, const float* x, const int32_t* row_index, const float* y, const float* y2, const void* bias,
                           float bias_scale, const void* w1, const void* w2, bool f32, float eps, float* x_out, float* h1, bf16* h1_b16,
-                          float* h2, bf16* h2_b16, int rows, int W);
+                          float* h2, bf16* h2_b16, int rows, int W, const ParScale* sc = nullptr);
 // out = relu(in)^2 (fp32 in, row stride ldi; fp32 and / or bf16 out, dense rows of n)
 cudaError_t relu2_rows(cudaStream_t s, const float* in, long ldi, float* out, bf16* out_b16, int T, int n);
 // the same on bf16 rows (tensor-core path)
@@ -541,14 +614,16 @@ cudaError_t relu2_rows_b16(cudaStream_t s, const bf16* in, long ldi, bf16* out, 
 
 // ---- gated feed-forward units and mixtures of experts (stack_moe.cu).
 cudaError_t stack_moe_init();
-enum GluAct : int { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED = 2 };
+enum GluAct : int { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED = 2, GLU_NONE_GELU = 3 };  // GLU_NONE_GELU: ungated, gelu_erf(up)
 // GLU_CLAMPED: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1); the others act(gate) * up.
 // How a router turns logits into a choice.  softmax or sigmoid scores; the top_k largest of (score + correction) among the
 // eligible outputs are chosen, lowest index first among equals: with groups > 1 the outputs form that many equal groups of
 // neighbours, a group scores the sum of its two largest corrected scores and only the `keep` best groups are eligible.
-// The weights are the chosen outputs' uncorrected scores, divided by their sum (+ 1e-20) when renorm, times scale.
+// The weights are the chosen outputs' uncorrected scores, divided by their sum (+ 1e-20) when renorm, times scale.  bias: the
+// correction row is added to the logits instead of the scores.  chosen: the largest (biased) logits are chosen and the weights
+// are the softmax over the chosen ones.
 struct RouteOpts {
-  int sigmoid = 0, groups = 0, keep = 0, renorm = 0;
+  int sigmoid = 0, groups = 0, keep = 0, renorm = 0, chosen = 0, bias = 0;
   float scale = 1.f;
 };
 // out[t, j] = act(gu[t, j]) * gu[t, F + j]   (row stride ldg; out may be null when only the bf16 copy is wanted)

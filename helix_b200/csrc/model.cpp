@@ -177,10 +177,14 @@ std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
       if (l.dim > 256) return "GLA key channels per head > 256 unsupported (one warp per 16 channels, 512 threads per block)" + at;
       if (!(l.tau > 0.f) || l.decay_rank <= 0) return "GLA needs tau > 0 and a decay rank" + at;
     } else if (l.mixer == HB_MIXER_LATENT) {
-      if (l.q_rank <= 0 || l.kv_rank <= 0 || l.rot_dim < 0 || l.window <= 0) return "latent attention sizes" + at;
+      if (l.q_rank < 0 || l.kv_rank <= 0 || l.rot_dim < 0) return "latent attention sizes" + at;
+      if (l.mask != HB_MASK_WINDOW && l.mask != HB_MASK_CAUSAL) return "latent attention masks: window or causal" + at;
+      if (l.mask == HB_MASK_WINDOW && l.window <= 0) return "window size must be positive" + at;
+      if (l.rope_pairing != 0 && l.rope_pairing != 1) return "unknown rope_pairing" + at;
+      if (l.attn_flags & ~(HB_ATTN_NO_SINK | HB_ATTN_HEAD_GATE)) return "unsupported latent attention option" + at;
       if (l.rope_dims < 0 || l.rope_dims % 2 || l.rope_dims > l.rot_dim) return "rope_dims must be even and <= rot_dim" + at;
       if (l.rope_dims > 0 && !(l.rope_base > 0.f)) return "rope_base must be positive" + at;
-      if ((size_t)(4 * (l.kv_rank + l.rot_dim + 4) + 5 * l.window + 8 * 1024 + 136) * 4 > 200 * 1024) return "window + latent row exceed the attention kernel's shared memory" + at;
+      if (latent_attn_smem(l.kv_rank, l.rot_dim, l.mask == HB_MASK_CAUSAL ? 1 << 30 : l.window) > 200 * 1024) return "latent row exceeds the attention kernel's shared memory" + at;
       if (l.kv_from >= 0) {
         if (l.kv_from >= i) return "kv_from must name an earlier layer" + at;
         const hb_layer_desc& s = L[l.kv_from];
@@ -249,8 +253,9 @@ std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
       if (l.ff_kind == HB_FF_MOE) {
         if (l.experts <= 0 || l.identity_experts < 0 || l.top_k <= 0 || l.top_k > l.experts + l.identity_experts) return "mixture-of-experts sizes" + at;
         if (l.experts + l.identity_experts > 1024 || l.top_k > 32) return "more than 1024 router outputs or top_k > 32 unsupported" + at;
-        if (l.router_kind != HB_ROUTER_SOFTMAX && l.router_kind != HB_ROUTER_SIGMOID) return "unknown router kind" + at;
-        if (l.expert_kind != HB_EXPERT_SILU && l.expert_kind != HB_EXPERT_CLAMPED) return "unknown expert kind" + at;
+        if (l.router_kind != HB_ROUTER_SOFTMAX && l.router_kind != HB_ROUTER_SIGMOID && l.router_kind != HB_ROUTER_CHOSEN) return "unknown router kind" + at;
+        if (l.expert_kind != HB_EXPERT_SILU && l.expert_kind != HB_EXPERT_CLAMPED && l.expert_kind != HB_EXPERT_GELU) return "unknown expert kind" + at;
+        if (l.expert_kind == HB_EXPERT_GELU && l.shared_ff > 0) return "ungated experts with a shared unit are unsupported" + at;
         if (l.route_groups > 1) {
           const int R = l.experts + l.identity_experts;
           if (R % l.route_groups) return "router outputs must divide into the groups" + at;
@@ -269,7 +274,10 @@ std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
   if (d.norm_place == HB_NORM_PARALLEL) {
     if (d.norm_kind != HB_NORM_RMS) return "parallel sublayers need RMS norms";
     for (int i = 0; i < d.n_layers; ++i)
-      if (L[i].ff > 0 && (L[i].ff_kind == HB_FF_MOE || L[i].ff_kind == HB_FF_CLAMPED)) return "parallel sublayers with a mixture or a biased feed-forward are unsupported";
+      if (L[i].ff > 0 && (L[i].ff_kind == HB_FF_CLAMPED || (L[i].ff_kind == HB_FF_MOE && L[i].shared_ff > 0)))
+        return "parallel sublayers with a biased feed-forward or a shared expert are unsupported";
+  } else if (d.one_norm || d.layer_scale || (d.resid_mult != 0.f && d.resid_mult != 1.f)) {
+    return "one_norm, layer_scale and resid_mult need parallel sublayers";
   }
   if (d.norm_kind != HB_NORM_RMS && d.norm_kind != HB_NORM_TANH) return "unknown norm_kind";
   for (int i = 0; i < d.n_layers; ++i) {
@@ -371,6 +379,16 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
     muted = shared_w;
     w.norm1 = norm_block(p + "norm1");
     if (both) w.norm1b = norm_block(p + "norm1b");
+    if (d.layer_scale) {
+      uint8_t* s1 = take(W);
+      put(p + "ls1", s1, 0, W, 1, true, 1.f);
+      w.ls1 = s1;
+      if (l.ff > 0) {
+        uint8_t* s2 = take(W);
+        put(p + "ls2", s2, 0, W, 1, true, 1.f);
+        w.ls2 = s2;
+      }
+    }
     // a matrix memory: rows [q | k | v | g | i | f] from row `row0` of the fused projection `in`, gate biases in `bias`
     auto carve_mlstm = [&](const std::string& pm, uint8_t* in, uint8_t* bias, size_t row0, size_t Hm, size_t Dm, size_t Dvm, float cap) {
       MlstmW& q = w.ml;
@@ -591,30 +609,35 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
     } else {
       const size_t Q = l.q_rank, R = l.kv_rank, Dr = l.rot_dim;
       const bool own = l.kv_from < 0;
-      w.off_dq = 0;
-      w.off_dkv = own ? (int)Q : -1;
-      w.off_g = (int)(Q + (own ? R + Dr : 0));
-      w.n_in = (int)(w.off_g + H * Dv);
+      const size_t q_rows = Q > 0 ? Q : H * (Dk + Dr);  // the query latent, or the queries themselves
+      const size_t g_rows = (l.attn_flags & HB_ATTN_HEAD_GATE) ? H : H * Dv;
+      w.off_dq = w.off_q = 0;
+      w.off_dkv = own ? (int)q_rows : -1;
+      w.off_g = (int)(q_rows + (own ? R + Dr : 0));
+      w.n_in = (int)(w.off_g + g_rows);
       uint8_t* in = take((size_t)w.n_in * W);
       w.w_in = in;
-      put(p + "mix.dq", in, 0, Q, W);
-      if (own) put(p + "mix.dkv", in, Q, R + Dr, W);
-      put(p + "mix.g", in, w.off_g, H * Dv, W);
-      uint8_t* dqn = take(Q);
-      uint8_t* uq = take(H * (Dk + Dr) * Q);
+      put(p + (Q > 0 ? "mix.dq" : "mix.q"), in, 0, q_rows, W);
+      if (own) put(p + "mix.dkv", in, q_rows, R + Dr, W);
+      put(p + "mix.g", in, w.off_g, g_rows, W);
+      uint8_t* dqn = Q > 0 ? take(Q) : nullptr;
+      uint8_t* uq = Q > 0 ? take(H * (Dk + Dr) * Q) : nullptr;
       uint8_t* dkvn = own ? take(R) : nullptr;
-      uint8_t* uk = take(H * Dk * R);
-      uint8_t* uv = take(H * Dv * R);
+      uint8_t* uk = take(H * (Dk + Dv) * R);  // key rows, then value rows: one product expands both
+      uint8_t* uv = uk ? uk + H * Dk * R * es : nullptr;
       uint8_t* ukT = d.compute_f32 ? nullptr : take(H * Dk * R);
       w.ukT = ukT;
-      uint8_t* sink = take(H);
+      const bool has_sink = !(l.attn_flags & HB_ATTN_NO_SINK);
+      uint8_t* sink = has_sink ? take(H) : nullptr;
       uint8_t* o = take(W * H * Dv);
-      put(p + "mix.dq.norm", dqn, 0, Q, 1, true, 1.f);
-      put(p + "mix.uq", uq, 0, H * (Dk + Dr), Q);
+      if (Q > 0) {
+        put(p + "mix.dq.norm", dqn, 0, Q, 1, true, 1.f);
+        put(p + "mix.uq", uq, 0, H * (Dk + Dr), Q);
+      }
       if (own) put(p + "mix.dkv.norm", dkvn, 0, R, 1, true, 1.f);
       put(p + "mix.uk", uk, 0, H * Dk, R);
       put(p + "mix.uv", uv, 0, H * Dv, R);
-      put(p + "mix.sink", sink, 0, H, 1, false, 1.f, true);
+      if (has_sink) put(p + "mix.sink", sink, 0, H, 1, false, 1.f, true);
       put(p + "mix.o", o, 0, W, H * Dv);
       w.dq_norm = dqn; w.uq = uq; w.dkv_norm = dkvn; w.uk = uk; w.uv = uv; w.sink = sink; w.wo = o;
       if (own) {
@@ -627,14 +650,15 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
     }
     if (l.ff > 0 && l.ff_kind == HB_FF_MOE) {
       const size_t Fn = l.ff, E = l.experts, R = (size_t)l.experts + l.identity_experts;
-      uint8_t* n2 = norm_block(p + "norm2");
+      const bool gated = l.expert_kind != HB_EXPERT_GELU;
+      uint8_t* n2 = d.one_norm ? nullptr : norm_block(p + "norm2");
       if (both) w.norm2b = norm_block(p + "norm2b");
       uint8_t* router = take(std::max<size_t>(R, 64) * W);  // at least one MMA tile of rows; the arena is zeroed at load
       uint8_t* corr = take(R);
-      uint8_t* gu = take(E * 2 * Fn * W);
+      uint8_t* gu = take(E * (gated ? 2 : 1) * Fn * W);
       uint8_t* dn = take(E * W * Fn);
       put(p + "mlp.router", router, 0, R, W);
-      put(p + "mlp.correction", corr, 0, R, 1, false, 1.f, true);
+      put(p + (l.route_bias ? "mlp.router.b" : "mlp.correction"), corr, 0, R, 1, false, 1.f, true);
       if (l.shared_ff > 0) {
         const size_t Fs = l.shared_ff;
         uint8_t* sg = take(2 * Fs * W);
@@ -645,18 +669,19 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
         put(p + "mlp.shared.down", sd, 0, W, Fs);
         w.w_gu_sh = sg; w.w_down_sh = sd; w.sh_packed = spk;
       }
-      const bool packed = !d.compute_f32 && Fn % 128 == 0;
+      const bool packed = gated && !d.compute_f32 && Fn % 128 == 0;
       for (size_t e = 0; e < E; ++e) {
         const std::string pe = p + "mlp.e" + std::to_string(e) + ".";
-        put(pe + "gate", gu, e * 2 * Fn, Fn, W, false, 1.f, false, packed ? 1 : 0);
-        put(pe + "up", gu, e * 2 * Fn + (packed ? 0 : Fn), Fn, W, false, 1.f, false, packed ? 2 : 0);
+        if (gated) put(pe + "gate", gu, e * 2 * Fn, Fn, W, false, 1.f, false, packed ? 1 : 0);
+        if (gated) put(pe + "up", gu, e * 2 * Fn + (packed ? 0 : Fn), Fn, W, false, 1.f, false, packed ? 2 : 0);
+        else put(pe + "up", gu, e * Fn, Fn, W);
         put(pe + "down", dn, e * W, W, Fn);
       }
       w.gu_packed = packed;
       w.norm2 = n2; w.router = router; w.correction = corr; w.w_gu = gu; w.w_down = dn;
     } else if (l.ff > 0 && (l.ff_kind == HB_FF_GELU_TANH || l.ff_kind == HB_FF_SILU)) {
       const size_t Fn = l.ff;
-      uint8_t* n2 = norm_block(p + "norm2");
+      uint8_t* n2 = d.one_norm ? nullptr : norm_block(p + "norm2");
       if (both) w.norm2b = norm_block(p + "norm2b");
       uint8_t* gu = take(2 * Fn * W);
       uint8_t* dn = take(W * Fn);
@@ -668,7 +693,7 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
       w.norm2 = n2; w.w_gu = gu; w.w_down = dn;
     } else if (l.ff > 0 && l.ff_kind == HB_FF_RELU2) {
       const size_t Fn = l.ff;
-      uint8_t* n2 = norm_block(p + "norm2");
+      uint8_t* n2 = d.one_norm ? nullptr : norm_block(p + "norm2");
       if (both) w.norm2b = norm_block(p + "norm2b");
       uint8_t* up_w = take(Fn * W);
       uint8_t* dn = take(W * Fn);
@@ -677,7 +702,7 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
       w.norm2 = n2; w.w_gu = up_w; w.w_down = dn;
     } else if (l.ff > 0) {
       const size_t Fn = l.ff;
-      uint8_t* n2 = norm_block(p + "norm2");
+      uint8_t* n2 = d.one_norm ? nullptr : norm_block(p + "norm2");
       if (both) w.norm2b = norm_block(p + "norm2b");
       uint8_t* gu = take(2 * Fn * W);
       uint8_t* bgu = take(2 * Fn);

@@ -23,7 +23,7 @@ struct BertLayerW {
 
 // One layer of a layer-list decoder (HB_ARCH_RISEPEL).  Pointers are arena addresses of elements of Model::elem bytes.
 // Projections that read the same input are stacked into one weight (w_in) so one GEMM produces all of them:
-//   GLA:    rows [q | k | v | g | a1]            LATENT: rows [dq | dkv (own cache only) | g]
+//   GLA:    rows [q | k | v | g | a1]            LATENT: rows [dq, or q when there is no query latent | dkv (own cache only) | g]
 //   GQA:    rows [q | k | v (unless the values are the keys) | g (one row per head, when gated)]
 //   DELTA:  rows [q | k | v | g | b (one row per head) | a (one row per head)]
 // Norms of kind HB_NORM_TANH are blocks [gain (width) | offset (width) | alpha (1)] behind one pointer.
@@ -45,6 +45,7 @@ struct StackLayerW {
   int off_q = 0, off_k = 0, off_v = 0, off_g = 0, off_a1 = 0, off_dq = 0, off_dkv = -1;  // columns of the fused projection
   void *a2 = nullptr, *a2b = nullptr, *hnorm = nullptr;                                          // GLA
   void *dq_norm = nullptr, *uq = nullptr, *dkv_norm = nullptr, *uk = nullptr, *uv = nullptr, *sink = nullptr;  // LATENT
+  void *ls1 = nullptr, *ls2 = nullptr;  // layer_scale: gains of the sublayers' outputs [width]
   void* ukT = nullptr;  // LATENT, bf16 mode: [heads][kv_rank][dim] copy of uk (built after load; no checkpoint tensor)
   void* b_in = nullptr;     // GQA with biases: [n_in] in the order of w_in's rows
   void* qk_gain = nullptr;  // GQA with whole-projection norms: [heads * dim | kv_heads * dim]
@@ -66,8 +67,9 @@ struct StackLayerW {
   size_t state_off = 0;  // GLA: float offset of this layer's [heads][dim][vdim] block inside a state slot
   int cache_plane = -1;  // LATENT: plane of the latent pool this layer reads (its own, or the kv_from layer's); GQA: its key plane
   int cache_plane_v = -1;  // GQA: its value plane.  Both are [page][kv_head][page_size][dim | vdim]
-  // mixture of experts: router rows and choice corrections for experts + identity outputs; expert e's [gate | up] rows at
-  // w_gu + e * 2 ff * width, its down-projection at w_down + e * width * ff
+  // mixture of experts: router rows and choice corrections (or logit biases) for experts + identity outputs; expert e's
+  // [gate | up] rows at w_gu + e * 2 ff * width (ungated experts: its up rows at w_gu + e * ff * width), its down-projection at
+  // w_down + e * width * ff
   void *router = nullptr, *correction = nullptr;
   // bf16 mode, ff a multiple of 128 (tanh-GELU unit, experts): [gate | up] rows stored per 256-row tile as [128 gate | 128 up],
   // the layout the gated epilogue of the tcgen05 GEMM reads; every other consumer indexes through it

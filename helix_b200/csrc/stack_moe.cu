@@ -60,7 +60,7 @@ template <typename WT>
 __device__ __forceinline__ void route_one(const float* zr, const WT* __restrict__ corr, int R, int top_k, float* pick,
                                           int32_t* __restrict__ ids, float* __restrict__ wts, int l, const RouteOpts& ro) {
   float mx = 0.f, inv = 1.f;
-  if (!ro.sigmoid) {
+  if (!ro.sigmoid && !ro.chosen) {
     mx = -INFINITY;
     for (int i = l; i < R; i += 32) mx = fmaxf(mx, zr[i]);
     mx = warp_max(mx);
@@ -69,8 +69,12 @@ __device__ __forceinline__ void route_one(const float* zr, const WT* __restrict_
     sum = warp_sum(sum);
     inv = 1.f / sum;
   }
-  auto score = [&](int i) { return ro.sigmoid ? sigmoidf_(zr[i]) : expf(zr[i] - mx) * inv; };
-  for (int i = l; i < R; i += 32) pick[i] = score(i) + ldf<WT>(corr, i);
+  // (chosen: the choice and the weights both come from the biased logits, the softmax covers the chosen outputs only)
+  auto score = [&](int i) {
+    if (ro.chosen) return zr[i] + (ro.bias ? ldf<WT>(corr, i) : 0.f);
+    return ro.sigmoid ? sigmoidf_(zr[i]) : expf(zr[i] - mx) * inv;
+  };
+  for (int i = l; i < R; i += 32) pick[i] = ro.bias ? score(i) : score(i) + ldf<WT>(corr, i);
   __syncwarp();
   if (ro.groups > 1 && ro.keep < ro.groups) {
     float* gs = pick + R;
@@ -120,7 +124,11 @@ __device__ __forceinline__ void route_one(const float* zr, const WT* __restrict_
     }
     if (l == 0) {
       if (bi >= R) bi = 0;  // fewer eligible outputs than top_k (excluded at load): stay inside the tables
-      const float sc = score(bi);  // the score itself, without the correction
+      float sc = score(bi);  // the score itself, without the correction
+      if (ro.chosen) {
+        if (k == 0) mx = sc;  // the largest chosen logit
+        sc = expf(sc - mx);
+      }
       ids[k] = bi;
       wts[k] = sc;
       wsum += sc;
@@ -129,7 +137,7 @@ __device__ __forceinline__ void route_one(const float* zr, const WT* __restrict_
     __syncwarp();
   }
   if (l == 0) {
-    const float f = (ro.renorm ? 1.f / (wsum + 1e-20f) : 1.f) * ro.scale;
+    const float f = (ro.chosen ? 1.f / wsum : ro.renorm ? 1.f / (wsum + 1e-20f) : 1.f) * ro.scale;
     if (f != 1.f)
       for (int k = 0; k < top_k; ++k) wts[k] *= f;
   }
@@ -280,7 +288,9 @@ __device__ __forceinline__ float warp_dot(const WT* __restrict__ wrow, const flo
   return warp_sum(s);
 }
 
-// block per (token, choice).  dynamic smem: x [Wp] + inner activation [F]
+__device__ __forceinline__ float gelu_erf_(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
+
+// block per (token, choice).  act GLU_NONE_GELU: ungated units (w_gu: [E][F][W] up rows).  dynamic smem: x [Wp] + inner activation [F]
 template <typename WT>
 __global__ void __launch_bounds__(256) moe_expert_rows_kernel(const float* __restrict__ x, const bf16* __restrict__ xb,
                                                               const WT* __restrict__ w_gu, const WT* __restrict__ w_down,
@@ -296,8 +306,17 @@ __global__ void __launch_bounds__(256) moe_expert_rows_kernel(const float* __res
   for (int i = threadIdx.x; i < W; i += blockDim.x) xs[i] = xb ? __bfloat162float(xb[(size_t)t * W + i]) : x[(size_t)t * W + i];
   __syncthreads();
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const WT* gu = w_gu + (size_t)e * 2 * F * W;
+  const bool gated = act != GLU_NONE_GELU;
+  const WT* gu = w_gu + (size_t)e * (gated ? 2 : 1) * F * W;
   for (int f = w; f < F; f += nw) {
+    if (!gated) {
+      const float u = warp_dot<WT>(gu + (size_t)f * W, xs, W, l);
+      if (l == 0) {
+        const float v = gelu_erf_(u);
+        hs[f] = xb ? __bfloat162float(__float2bfloat16(v)) : v;
+      }
+      continue;
+    }
     const size_t gr = packed ? (size_t)(f >> 7) * 256 + (f & 127) : (size_t)f, ur = packed ? gr + 128 : (size_t)F + f;
     const float g = warp_dot<WT>(gu + gr * W, xs, W, l);
     const float u = warp_dot<WT>(gu + ur * W, xs, W, l);

@@ -259,14 +259,38 @@ __global__ void clamped_glu_kernel(const float* __restrict__ gu, long ldg, const
   }
 }
 
-__global__ void sigmoid_gate_kernel(const float* __restrict__ o, long ldo, const float* __restrict__ g, long ldg,
-                                    float* __restrict__ out, bf16* __restrict__ outb, int N) {
-  const int t = blockIdx.y;
-  const int j = blockIdx.x * blockDim.x + threadIdx.x;
+// VEC = 4: Dv, the strides and the offsets are multiples of four (16-byte loads, 8-byte stores)
+template <int VEC>
+__global__ void latent_gate_kernel(const float* __restrict__ o, long o_ts, long o_hs, const float* __restrict__ g, long ldg, int per_head,
+                                   float* __restrict__ out, bf16* __restrict__ outb, int H, int Dv) {
+  const int t = blockIdx.y, N = H * Dv;
+  const int j = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
   if (j >= N) return;
-  const float v = o[(size_t)t * ldo + j] * sigmoidf_(g[(size_t)t * ldg + j]);
-  out[(size_t)t * N + j] = v;
-  if (outb) outb[(size_t)t * N + j] = __float2bfloat16(v);
+  const int h = j / Dv, i = j - h * Dv;
+  const float* src = o + (size_t)t * o_ts + (size_t)h * o_hs + i;
+  const float* gs = g + (size_t)t * ldg + (per_head ? h : j);
+  float v[VEC];
+  if (VEC == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(src);
+    v[0] = x.x; v[1 % VEC] = x.y; v[2 % VEC] = x.z; v[VEC - 1] = x.w;
+  } else {
+    v[0] = src[0];
+  }
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) v[e] *= sigmoidf_(gs[per_head ? 0 : e]);
+  if (VEC == 4) {
+    if (out) *reinterpret_cast<float4*>(out + (size_t)t * N + j) = make_float4(v[0], v[1 % VEC], v[2 % VEC], v[VEC - 1]);
+    if (outb) {
+      __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1 % VEC]), hi = __floats2bfloat162_rn(v[2 % VEC], v[VEC - 1]);
+      uint2 pk;
+      pk.x = *reinterpret_cast<unsigned*>(&lo);
+      pk.y = *reinterpret_cast<unsigned*>(&hi);
+      *reinterpret_cast<uint2*>(outb + (size_t)t * N + j) = pk;
+    }
+  } else {
+    if (out) out[(size_t)t * N + j] = v[0];
+    if (outb) outb[(size_t)t * N + j] = __float2bfloat16(v[0]);
+  }
 }
 
 // VEC = 4: N, both strides and both bases are multiples of four elements (16-byte loads, 8-byte stores)
@@ -418,21 +442,24 @@ __global__ void headnorm_gate_kernel(const float* __restrict__ o, long ldo, cons
 }
 
 // ------------------------------------------------------------------ latent attention
-// angle of pair i at position p: p * base^(-2i/dims), in fp32
-__device__ __forceinline__ void rope_pair(float u, float v, int pos, int i, int dims, float base, float* ou, float* ov) {
-  const float f = powf(base, -2.f * (float)i / (float)dims);
-  float s, c;
-  sincosf((float)pos * f, &s, &c);
-  *ou = u * c - v * s;
-  *ov = v * c + u * s;
+// entry i < rope_dims of a rotated vector src (cs: cos / sin pairs of the token); pairing 1: entries 2e and 2e + 1 form pair e,
+// pairing 0: entries e and e + rope_dims / 2
+__device__ __forceinline__ float rope_entry(const float* __restrict__ src, int i, const float* __restrict__ cs, int rope_dims, int pairing) {
+  const int half = rope_dims >> 1;
+  const int e = pairing ? i >> 1 : (i < half ? i : i - half);
+  const bool first = pairing ? (i & 1) == 0 : i < half;
+  const float c = cs[2 * e], s = cs[2 * e + 1];
+  const float u = src[pairing ? 2 * e : e], v = src[pairing ? 2 * e + 1 : e + half];
+  return first ? u * c - v * s : v * c + u * s;
 }
 
 template <typename WT, typename CT>
-__global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
+__global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
   __shared__ float red[32];
   const int t = blockIdx.x;
   const float* p = a.p + (size_t)t * a.ldp;
-  {
+  const float* cs = a.rope_dims > 0 ? a.cs + (size_t)t * a.rope_dims : nullptr;
+  if (a.Q > 0) {
     float ss = 0.f;
     for (int i = threadIdx.x; i < a.Q; i += blockDim.x) ss += p[a.q_off + i] * p[a.q_off + i];
     ss = block_sum(ss, red);
@@ -441,6 +468,29 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
       const float v = p[a.q_off + i] * rs * ldf<WT>((const WT*)a.wq, i);
       a.cq[(size_t)t * a.Q + i] = v;
       if (a.cq_b16) a.cq_b16[(size_t)t * a.Q + i] = __float2bfloat16(v);
+    }
+  }
+  if (a.q16) {  // query heads as bf16, eight entries per thread (head parts are multiples of eight)
+    const int Dq = a.Dk + a.Dr, n8 = a.H * Dq / 8;
+    const int tq = t - a.qh_t0;
+    for (int i8 = threadIdx.x; i8 < n8; i8 += blockDim.x) {
+      const int h = i8 * 8 / Dq, e = i8 * 8 - h * Dq;
+      const float* src = p + a.q_off + (size_t)h * Dq;
+      float v[8];
+      if (e < a.Dk || e - a.Dk >= a.rope_dims) {
+        const float4 x = *reinterpret_cast<const float4*>(src + e), y = *reinterpret_cast<const float4*>(src + e + 4);
+        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+      } else {
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          v[k] = e - a.Dk + k < a.rope_dims ? rope_entry(src + a.Dk, e - a.Dk + k, cs, a.rope_dims, a.pairing) : src[e + k];
+      }
+      __nv_bfloat162 b[4] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3]), __floats2bfloat162_rn(v[4], v[5]),
+                             __floats2bfloat162_rn(v[6], v[7])};
+      const uint4 u = *reinterpret_cast<uint4*>(b);
+      *reinterpret_cast<uint4*>(a.q16 + (size_t)t * a.H * Dq + i8 * 8) = u;
+      if (a.qh && e < a.Dk && tq >= 0 && tq < kLatentTokRows)
+        *reinterpret_cast<uint4*>(a.qh + ((size_t)h * kLatentTokRows + tq) * a.Dk + e) = u;
     }
   }
   if (a.kv_off < 0) return;
@@ -453,37 +503,25 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
   ss = block_sum(ss, red);
   const float rs = 1.f / sqrtf(ss / (float)a.R + a.eps);
   for (int i = threadIdx.x; i < a.R; i += blockDim.x) stf<CT>(row, i, kv[i] * rs * ldf<WT>((const WT*)a.wkv, i));
-  const int half = a.rope_dims / 2, pos = a.positions[t];
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    float u, v;
-    rope_pair(kv[a.R + i], kv[a.R + half + i], pos, i, a.rope_dims, a.rope_base, &u, &v);
-    stf<CT>(row, a.R + i, u);
-    stf<CT>(row, a.R + half + i, v);
-  }
-  for (int i = a.rope_dims + threadIdx.x; i < a.Dr; i += blockDim.x) stf<CT>(row, a.R + i, kv[a.R + i]);
+  for (int i = threadIdx.x; i < a.Dr; i += blockDim.x)
+    stf<CT>(row, a.R + i, i < a.rope_dims ? rope_entry(kv + a.R, i, cs, a.rope_dims, a.pairing) : kv[a.R + i]);
 }
 
-__global__ void latent_q_rope_kernel(const float* __restrict__ q, long ldq, float* __restrict__ qabs, long ldqa,
-                                     const int32_t* __restrict__ positions, int H, int Dk, int Dr, int R, int rope_dims, float base) {
-  const int t = blockIdx.x, pos = positions[t], half = rope_dims / 2;
+__global__ void latent_q_rope_kernel(const float* __restrict__ q, long ldq, float* __restrict__ qabs, long ldqa, const float* __restrict__ cs,
+                                     int H, int Dk, int Dr, int R, int rope_dims, int pairing) {
+  const int t = blockIdx.x;
+  const float* ct = cs + (size_t)t * rope_dims;
   for (int e = threadIdx.x; e < H * Dr; e += blockDim.x) {
     const int h = e / Dr, i = e % Dr;
     const float* src = q + (size_t)t * ldq + (size_t)h * (Dk + Dr) + Dk;
-    float* dst = qabs + (size_t)t * ldqa + (size_t)h * (R + Dr) + R;
-    if (i < half) {
-      float u, v;
-      rope_pair(src[i], src[half + i], pos, i, rope_dims, base, &u, &v);
-      dst[i] = u;
-      dst[half + i] = v;
-    } else if (i >= rope_dims) {
-      dst[i] = src[i];
-    }
+    qabs[(size_t)t * ldqa + (size_t)h * (R + Dr) + R + i] = i < rope_dims ? rope_entry(src, i, ct, rope_dims, pairing) : src[i];
   }
 }
 
 // One block per (token, group of kLatHG heads), kLatThreads threads.  Every head of a token reads the same cache rows, so a
-// block serves several heads from one pass over them.  dynamic smem: q [HG][D] + scores [window][HG] + page-resolved row
-// index [window] + group partials [threads][HG] + 32.
+// block serves several heads from one pass over them.  Keys are taken in blocks of up to kLatentKeyBlock with a running maximum
+// and sum (one block unless a position sees more).  dynamic smem: q [HG][D] + weighted sums [HG][R] + scores [keys][HG] +
+// page-resolved row index [keys] + group partials [8 threads] + 32 HG.
 // Scores: one warp per key (16-byte loads of bf16 rows when the row length allows), HG dot products per loaded row.
 // Weighted sum: thread (g, r) adds the keys jj = g mod G of latent entry r for all HG heads; groups are then summed in group
 // order — fixed per (R, threads), independent of the batch.
@@ -495,26 +533,40 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(LatentAttnArgs
   extern __shared__ float sm[];
   const int D = a.R + a.Dr, Dp = (D + 3) / 4 * 4;
   float* qs = sm;                       // [HG][Dp]
-  float* sc = qs + HG * Dp;             // [window][HG]
-  float* part = sc + HG * a.window;     // [8 * threads]: group partials of the weighted sum
+  const int KB = min(a.window, kLatentKeyBlock);
+  float* acc_s = qs + HG * Dp;          // [HG][R] weighted sums of the blocks so far
+  float* sc = acc_s + HG * a.R;         // [keys][HG]
+  float* part = sc + HG * KB;           // [8 * threads]: group partials of the weighted sum
   float* red = part + 8 * blockDim.x;   // [32 * HG]
-  int* rowoff = reinterpret_cast<int*>(red + 32 * HG);  // [window] cache row of every visible key (page lookup done once)
+  int* rowoff = reinterpret_cast<int*>(red + 32 * HG);  // [keys] cache row of every visible key (page lookup done once)
   const int t = blockIdx.x, h0 = blockIdx.y * HG;
   const int nh = min(HG, a.H - h0);
   const int pos = a.positions[t];
-  const int n = min(pos + 1, a.window), j0 = pos - n + 1;  // keys j0 .. pos
+  const int n_all = min(pos + 1, a.window), first = pos - n_all + 1;  // keys first .. pos
   const int32_t* pt = a.page_table + (size_t)a.seq_of[t] * a.max_pages;
   const CT* cache = (const CT*)a.cache;
   for (int e = threadIdx.x; e < HG * Dp; e += blockDim.x) {
     const int hh = e / Dp, i = e % Dp;
     qs[e] = (hh < nh && i < D) ? a.qabs[(size_t)t * a.ldqa + (size_t)(h0 + hh) * D + i] : 0.f;
   }
+  for (int e = threadIdx.x; e < HG * a.R; e += blockDim.x) acc_s[e] = 0.f;
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
+  float m_run[HG], l_run[HG];
+#pragma unroll
+  for (int hh = 0; hh < HG; ++hh) {  // the sink is a key without a value: it opens the running maximum and sum
+    m_run[hh] = a.sink && hh < nh ? ldf<WT>((const WT*)a.sink, h0 + hh) : -INFINITY;
+    l_run[hh] = a.sink ? 1.f : 0.f;
+  }
+  for (int kb = 0; kb < n_all; kb += KB) {
+  const int n = min(KB, n_all - kb), j0 = first + kb;
+  const bool last_block = kb + KB >= n_all;
+  float inv[HG], fac[HG];
+  __syncthreads();  // the previous block's scores and rows have been read
   for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
     const int j = j0 + jj;
     rowoff[jj] = pt[j / a.page_size] * a.page_size + j % a.page_size;
   }
   __syncthreads();
-  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
   if (sizeof(CT) == 2 && (D & 7) == 0) {
     // bf16 rows that start on 16-byte boundaries: two keys per iteration, their loads issued together
     for (int jj = w; jj < n; jj += 2 * nw) {
@@ -568,10 +620,10 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(LatentAttnArgs
     }
   }
   __syncthreads();
-  // fp32 softmax with the sink in the denominator; the HG heads share each block reduction
-  float inv[HG], mx[HG], sink[HG];
+  // fp32 softmax; the HG heads share each block reduction
+  float mx[HG];
 #pragma unroll
-  for (int hh = 0; hh < HG; ++hh) mx[hh] = sink[hh] = hh < nh ? ldf<WT>((const WT*)a.sink, h0 + hh) : 0.f;
+  for (int hh = 0; hh < HG; ++hh) mx[hh] = m_run[hh];
   for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
     const float4 v = *reinterpret_cast<const float4*>(sc + jj * HG);
     mx[0] = fmaxf(mx[0], v.x); mx[1] = fmaxf(mx[1], v.y); mx[2] = fmaxf(mx[2], v.z); mx[3] = fmaxf(mx[3], v.w);
@@ -602,7 +654,18 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(LatentAttnArgs
   }
   __syncthreads();  // also publishes the exponentials in sc[]
 #pragma unroll
-  for (int hh = 0; hh < HG; ++hh) inv[hh] = 1.f / (warp_sum(l < nw ? red[l * HG + hh] : 0.f) + expf(sink[hh] - mx[hh]));
+  for (int hh = 0; hh < HG; ++hh) {
+    fac[hh] = m_run[hh] == -INFINITY ? 0.f : expf(m_run[hh] - mx[hh]);
+    l_run[hh] = l_run[hh] * fac[hh] + warp_sum(l < nw ? red[l * HG + hh] : 0.f);
+    m_run[hh] = mx[hh];
+    inv[hh] = last_block ? 1.f / l_run[hh] : 1.f;
+  }
+  // entry r of head hh: this block's weighted sum joins the earlier ones; the last block leaves
+  auto put = [&](int hh, int r, float tot) {
+    const float v = acc_s[hh * a.R + r] * fac[hh] + tot;
+    if (!last_block) acc_s[hh * a.R + r] = v;
+    else if (hh < nh) a.ctx[(size_t)t * a.ldc + (size_t)(h0 + hh) * a.R + r] = v * inv[hh];
+  };
   if (sizeof(CT) == 2 && (D & 7) == 0 && (a.R & 7) == 0 && a.R / 8 <= (int)blockDim.x) {
     // bf16 rows: a thread owns 8 consecutive latent entries (one 16-byte load per key), the block's threads form G groups
     // that take every G-th key, so many loads are in flight per SM; groups are summed in group order, one head at a time
@@ -644,10 +707,10 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(LatentAttnArgs
         for (int r = threadIdx.x; r < a.R; r += blockDim.x) {
           float tot = 0.f;
           for (int gg = 0; gg < G; ++gg) tot += part[gg * a.R + r];
-          a.ctx[(size_t)t * a.ldc + (size_t)(h0 + hh) * a.R + r] = tot * inv[hh];
+          put(hh, r, tot);
         }
     }
-    return;
+    continue;
   }
   const int Rp = (a.R + 31) / 32 * 32;
   const int G = max(1, (int)blockDim.x / Rp);
@@ -679,14 +742,15 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(LatentAttnArgs
         for (int hh = 0; hh < HG; ++hh) {
           float tot = 0.f;
           for (int gg = 0; gg < G; ++gg) tot += part[(gg * Rp + threadIdx.x) * HG + hh];
-          if (hh < nh) a.ctx[(size_t)t * a.ldc + (size_t)(h0 + hh) * a.R + threadIdx.x] = tot * inv[hh];
+          put(hh, threadIdx.x, tot);
         }
       }
     } else if (r < a.R) {
 #pragma unroll
       for (int hh = 0; hh < HG; ++hh)
-        if (hh < nh) a.ctx[(size_t)t * a.ldc + (size_t)(h0 + hh) * a.R + r] = acc[hh] * inv[hh];
+        put(hh, r, acc[hh]);
     }
+  }
   }
 }
 
@@ -735,7 +799,7 @@ __global__ void __launch_bounds__(128) latent_softmax_kernel(const float* __rest
   const int lo = max(pos - window + 1, k0) - k0, hi = min(pos, k0 + nk - 1) - k0;  // visible columns [lo, hi]
   const float* s = S + (size_t)row * ld;
   bf16* p = P + (size_t)row * ld;
-  const float snk = __bfloat162float(sink[h]);
+  const float snk = sink ? __bfloat162float(sink[h]) : -INFINITY;
   float m = snk;
   for (int j = lo + l; j <= hi; j += 32) m = fmaxf(m, s[j] * scale);
   m = warp_max(m);
@@ -874,9 +938,14 @@ cudaError_t clamped_glu(cudaStream_t s, const float* gu, long ldg, const void* b
   return KERR();
 }
 
-cudaError_t sigmoid_gate(cudaStream_t s, const float* o, long ldo, const float* g, long ldg, float* out, bf16* outb, int T, int N) {
+cudaError_t latent_out_gate(cudaStream_t s, const float* o, long o_ts, long o_hs, const float* g, long ldg, bool per_head, float* out,
+                            bf16* outb, int T, int H, int Dv) {
   if (T <= 0) return cudaSuccess;
-  sigmoid_gate_kernel<<<dim3((N + 255) / 256, T), 256, 0, s>>>(o, ldo, g, ldg, out, outb, N);
+  const int N = H * Dv;
+  const bool vec = Dv % 4 == 0 && o_ts % 4 == 0 && o_hs % 4 == 0 && ((uintptr_t)o & 15) == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)outb & 7) == 0;
+  dim3 grid(((vec ? N / 4 : N) + 255) / 256, T);
+  if (vec) latent_gate_kernel<4><<<grid, 256, 0, s>>>(o, o_ts, o_hs, g, ldg, per_head ? 1 : 0, out, outb, H, Dv);
+  else latent_gate_kernel<1><<<grid, 256, 0, s>>>(o, o_ts, o_hs, g, ldg, per_head ? 1 : 0, out, outb, H, Dv);
   return KERR();
 }
 cudaError_t to_bf16_rows(cudaStream_t s, const float* src, long lds, bf16* dst, long ldd, int T, int N) {
@@ -925,22 +994,25 @@ cudaError_t headnorm_silu_gate(cudaStream_t s, const float* o, long ldo, const f
 
 cudaError_t latent_prep(cudaStream_t s, const LatentPrepArgs& a) {
   if (a.T <= 0) return cudaSuccess;
-  if (a.rope_dims % 2 || a.rope_dims > a.Dr) return cudaErrorInvalidValue;
-  if (a.f32) latent_prep_kernel<float, float><<<a.T, 128, 0, s>>>(a);
-  else latent_prep_kernel<bf16, bf16><<<a.T, 128, 0, s>>>(a);
+  if (a.rope_dims % 2 || a.rope_dims > a.Dr || (a.rope_dims > 0 && !a.cs)) return cudaErrorInvalidValue;
+  if (a.q16 && (a.Dk % 8 || a.Dr % 8 || a.ldp % 4 || a.q_off % 4 || ((uintptr_t)a.p & 15))) return cudaErrorInvalidValue;
+  if (a.f32) latent_prep_kernel<float, float><<<a.T, 256, 0, s>>>(a);
+  else latent_prep_kernel<bf16, bf16><<<a.T, 256, 0, s>>>(a);
   return KERR();
 }
 
-cudaError_t latent_q_rope(cudaStream_t s, const float* q, long ldq, float* qabs, long ldqa, const int32_t* positions, int T, int H,
-                          int Dk, int Dr, int R, int rope_dims, float base) {
-  if (T <= 0) return cudaSuccess;
-  latent_q_rope_kernel<<<T, 128, 0, s>>>(q, ldq, qabs, ldqa, positions, H, Dk, Dr, R, rope_dims, base);
+cudaError_t latent_q_rope(cudaStream_t s, const float* q, long ldq, float* qabs, long ldqa, const float* cs, int T, int H, int Dk, int Dr,
+                          int R, int rope_dims, int pairing) {
+  if (T <= 0 || Dr <= 0) return cudaSuccess;
+  if (rope_dims > 0 && !cs) return cudaErrorInvalidValue;
+  latent_q_rope_kernel<<<T, 128, 0, s>>>(q, ldq, qabs, ldqa, cs, H, Dk, Dr, R, rope_dims, pairing);
   return KERR();
 }
 
 cudaError_t latent_attn(cudaStream_t s, const LatentAttnArgs& a) {
   if (a.T <= 0) return cudaSuccess;
-  const size_t smem = (size_t)(kLatHG * ((a.R + a.Dr + 3) / 4 * 4) + (kLatHG + 1) * a.window + 8 * kLatThreads + 32 * kLatHG) * 4;
+  if (a.window <= 0) return cudaErrorInvalidValue;
+  const size_t smem = latent_attn_smem(a.R, a.Dr, a.window);
   if (smem > 200 * 1024) return cudaErrorInvalidValue;
   dim3 grid(a.T, (a.H + kLatHG - 1) / kLatHG);
   if (a.f32) latent_attn_kernel<float, float><<<grid, kLatThreads, smem, s>>>(a);

@@ -462,7 +462,7 @@ __global__ void __launch_bounds__(256) parallel_step_kernel(const float* x, cons
                                                             const WT* __restrict__ bias, float bias_scale, const WT* __restrict__ w1,
                                                             const WT* __restrict__ w2, float eps, float* x_out,
                                                             float* __restrict__ h1, bf16* __restrict__ h1b, float* __restrict__ h2,
-                                                            bf16* __restrict__ h2b, int W) {
+                                                            bf16* __restrict__ h2b, int W, const ParScale sc) {
   extern __shared__ __align__(16) float row[];
   __shared__ float red[32];
   const size_t r = blockIdx.x;
@@ -470,7 +470,13 @@ __global__ void __launch_bounds__(256) parallel_step_kernel(const float* x, cons
   float ss = 0.f;
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     float v = xs[i];
-    if (y) v += y2 ? y[r * W + i] + y2[r * W + i] : y[r * W + i];
+    if (y) {
+      float u = y[r * W + i], u2 = y2 ? y2[r * W + i] : 0.f;
+      for (int k = 0; k < sc.top_k; ++k) u2 = fmaf(sc.wts[r * sc.top_k + k], __bfloat162float(sc.rows[(size_t)sc.row_of[r * sc.top_k + k] * W + i]), u2);
+      if (sc.s1) u *= ldf<WT>((const WT*)sc.s1, i);
+      if (sc.s2) u2 *= ldf<WT>((const WT*)sc.s2, i);
+      v = fmaf(sc.m, u + u2, v);
+    }
     if (bias) v = fmaf(bias_scale, ldf<WT>(bias, i), v);
     row[i] = v;
     if (x_out) x_out[r * W + i] = v;
@@ -491,6 +497,81 @@ __global__ void __launch_bounds__(256) parallel_step_kernel(const float* x, cons
       if (h2) h2[r * W + i] = v;
       if (h2b) h2b[r * W + i] = __float2bfloat16(v);
     }
+  }
+}
+
+// The same step with the row in registers as float4 (W a multiple of 4, W <= 4 * 256 * kParChunks)
+constexpr int kParChunks = 8;
+constexpr int kParTop = 8;  // expert rows per token that the in-register form takes
+template <typename WT>
+__device__ __forceinline__ float4 ldf4(const WT* p) {
+  if constexpr (sizeof(WT) == 4) return *reinterpret_cast<const float4*>(p);
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ float4 fma4(float a, float4 b, float4 c) {
+  return make_float4(fmaf(a, b.x, c.x), fmaf(a, b.y, c.y), fmaf(a, b.z, c.z), fmaf(a, b.w, c.w));
+}
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ void st_pair(float* f, bf16* b, float4 v) {
+  if (f) *reinterpret_cast<float4*>(f) = v;
+  if (b) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 pk;
+    pk.x = *reinterpret_cast<unsigned*>(&lo);
+    pk.y = *reinterpret_cast<unsigned*>(&hi);
+    *reinterpret_cast<uint2*>(b) = pk;
+  }
+}
+template <typename WT, int CH>
+__global__ void __launch_bounds__(256) parallel_step_vec_kernel(const float* x, const int32_t* __restrict__ row_index, const float* __restrict__ y,
+                                                                const float* __restrict__ y2, const WT* __restrict__ bias, float bias_scale,
+                                                                const WT* __restrict__ w1, const WT* __restrict__ w2, float eps, float* x_out,
+                                                                float* __restrict__ h1, bf16* __restrict__ h1b, float* __restrict__ h2,
+                                                                bf16* __restrict__ h2b, int W, const ParScale sc) {
+  __shared__ float red[32];
+  const size_t r = blockIdx.x;
+  const float* xs = x + (row_index ? (size_t)row_index[r] : r) * W;
+  float4 v[CH];
+  float wk[kParTop];
+  size_t rk[kParTop];
+#pragma unroll
+  for (int k = 0; k < kParTop; ++k) {
+    wk[k] = k < sc.top_k ? sc.wts[r * sc.top_k + k] : 0.f;
+    rk[k] = k < sc.top_k ? (size_t)sc.row_of[r * sc.top_k + k] * W : 0;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = (threadIdx.x + c * 256) * 4;
+    if (i >= W) continue;
+    float4 a = *reinterpret_cast<const float4*>(xs + i);
+    if (y) {
+      float4 u = *reinterpret_cast<const float4*>(y + r * W + i);
+      float4 u2 = y2 ? *reinterpret_cast<const float4*>(y2 + r * W + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int k = 0; k < kParTop; ++k)
+        if (k < sc.top_k) u2 = fma4(wk[k], ldf4<bf16>(sc.rows + rk[k] + i), u2);
+      if (sc.s1) u = mul4(u, ldf4<WT>((const WT*)sc.s1 + i));
+      if (sc.s2) u2 = mul4(u2, ldf4<WT>((const WT*)sc.s2 + i));
+      a = fma4(sc.m, make_float4(u.x + u2.x, u.y + u2.y, u.z + u2.z, u.w + u2.w), a);
+    }
+    if (bias) a = fma4(bias_scale, ldf4<WT>(bias + i), a);
+    if (x_out) *reinterpret_cast<float4*>(x_out + r * W + i) = a;
+    v[c] = a;
+    ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+  }
+  if (!w1 && !w2) return;
+  ss = block_sum(ss, red);
+  const float rs = 1.f / sqrtf(ss / (float)W + eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = (threadIdx.x + c * 256) * 4;
+    if (i >= W) continue;
+    const float4 u = make_float4(v[c].x * rs, v[c].y * rs, v[c].z * rs, v[c].w * rs);
+    if (w1) st_pair(h1 ? h1 + r * W + i : nullptr, h1b ? h1b + r * W + i : nullptr, mul4(u, ldf4<WT>(w1 + i)));
+    if (w2) st_pair(h2 ? h2 + r * W + i : nullptr, h2b ? h2b + r * W + i : nullptr, mul4(u, ldf4<WT>(w2 + i)));
   }
 }
 
@@ -624,16 +705,31 @@ cudaError_t gate_scale_rows(cudaStream_t s, const float* in, const bf16* inb, lo
 
 cudaError_t parallel_step(cudaStream_t s, const float* x, const int32_t* row_index, const float* y, const float* y2, const void* bias,
                           float bias_scale, const void* w1, const void* w2, bool f32, float eps, float* x_out, float* h1, bf16* h1b, float* h2,
-                          bf16* h2b, int rows, int W) {
+                          bf16* h2b, int rows, int W, const ParScale* scale) {
   if (rows <= 0) return cudaSuccess;
-  if ((y2 && !y) || (size_t)W * 4 > 200 * 1024) return cudaErrorInvalidValue;
+  const ParScale sc = scale ? *scale : ParScale();
+  if (((y2 || sc.top_k > 0) && !y) || (sc.top_k > 0 && (y2 || !sc.rows || !sc.row_of || !sc.wts))) return cudaErrorInvalidValue;
+  const uintptr_t al = (uintptr_t)x | (uintptr_t)y | (uintptr_t)y2 | (uintptr_t)bias | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)x_out | (uintptr_t)h1 |
+                       (uintptr_t)h1b | (uintptr_t)h2 | (uintptr_t)h2b | (uintptr_t)sc.s1 | (uintptr_t)sc.s2 | (uintptr_t)sc.rows;
+  if (W % 4 == 0 && W <= 4 * 256 * kParChunks && (al & 15) == 0 && sc.top_k <= kParTop) {
+#define HB_PAR(WT, CH)                                                                                                                      \
+  parallel_step_vec_kernel<WT, CH><<<rows, 256, 0, s>>>(x, row_index, y, y2, (const WT*)bias, bias_scale, (const WT*)w1, (const WT*)w2, eps, \
+                                                        x_out, h1, h1b, h2, h2b, W, sc)
+    if (W <= 1024) { if (f32) HB_PAR(float, 1); else HB_PAR(bf16, 1); }
+    else if (W <= 2048) { if (f32) HB_PAR(float, 2); else HB_PAR(bf16, 2); }
+    else if (W <= 4096) { if (f32) HB_PAR(float, 4); else HB_PAR(bf16, 4); }
+    else { if (f32) HB_PAR(float, 8); else HB_PAR(bf16, 8); }
+#undef HB_PAR
+    return cudaGetLastError();
+  }
+  if ((size_t)W * 4 > 200 * 1024) return cudaErrorInvalidValue;
   const size_t smem = (size_t)W * 4;
   if (f32)
     parallel_step_kernel<float><<<rows, 256, smem, s>>>(x, row_index, y, y2, (const float*)bias, bias_scale, (const float*)w1, (const float*)w2,
-                                                        eps, x_out, h1, h1b, h2, h2b, W);
+                                                        eps, x_out, h1, h1b, h2, h2b, W, sc);
   else
     parallel_step_kernel<bf16><<<rows, 256, smem, s>>>(x, row_index, y, y2, (const bf16*)bias, bias_scale, (const bf16*)w1, (const bf16*)w2, eps,
-                                                       x_out, h1, h1b, h2, h2b, W);
+                                                       x_out, h1, h1b, h2, h2b, W, sc);
   return cudaGetLastError();
 }
 

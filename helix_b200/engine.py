@@ -85,11 +85,11 @@ MASK_WINDOW, MASK_CHUNK, MASK_CAUSAL = 0, 1, 2
 FF_CLAMPED, FF_GELU_TANH, FF_MOE, FF_SILU, FF_RELU2 = 0, 1, 2, 3, 4
 NORM_OF_SUM, NORM_OF_OUTPUT, NORM_BOTH_SIDES, NORM_PARALLEL = 0, 1, 2, 3
 NORM_RMS, NORM_TANH = 0, 1
-ROUTER_SOFTMAX, ROUTER_SIGMOID = 0, 1
-EXPERT_SILU, EXPERT_CLAMPED = 0, 1
+ROUTER_SOFTMAX, ROUTER_SIGMOID, ROUTER_CHOSEN = 0, 1, 2
+EXPERT_SILU, EXPERT_CLAMPED, EXPERT_GELU = 0, 1, 2
 ATTN_QK_UNIT_NORM, ATTN_V_IS_K, ATTN_UNIT_SINK, ATTN_HEAD_GATE = 1, 2, 4, 8
 ATTN_QKV_BIAS, ATTN_QK_PROJ_NORM, ATTN_LEARNED_SINK, ATTN_V_BLEND = 16, 32, 64, 128
-ATTN_QKV_CONV, ATTN_OUT_GATE, ATTN_OUT_BIAS = 256, 512, 1024
+ATTN_QKV_CONV, ATTN_OUT_GATE, ATTN_OUT_BIAS, ATTN_NO_SINK = 256, 512, 1024, 2048
 
 
 @dataclass
@@ -144,6 +144,7 @@ class LayerDesc:
     side_gate_cap: float = 0.0
     mix_scale: float = 0.0     # weights of the two mixers' outputs; 0 = 1
     side_scale: float = 0.0
+    route_bias: int = 0        # FF_MOE: 1: mlp.router.b joins the logits (no correction tensor)
 
     def to_c(self):
         return LayerDescC(self.mixer, self.heads, self.dim, self.vdim, self.tau, self.decay_rank, self.q_rank, self.kv_rank,
@@ -153,7 +154,7 @@ class LayerDesc:
                           self.score_cap, self.conv_taps, self.router_kind, self.route_groups, self.route_keep, self.route_renorm,
                           self.route_scale, self.expert_kind, self.shared_ff, self.shared_limit, self.weights_of, self.rope_linear,
                           self.norm_groups, self.gate_cap, self.side_mixer, self.side_heads, self.side_dim, self.side_vdim,
-                          self.side_gate_cap, self.mix_scale, self.side_scale)
+                          self.side_gate_cap, self.mix_scale, self.side_scale, self.route_bias)
 
 
 @dataclass
@@ -173,6 +174,9 @@ class StackDesc:
     embed_scale: float = 0.0   # 0 = 1
     logit_scale: float = 0.0   # 0 = 1
     tie_head: int = 0          # 1: logits from the embedding table
+    one_norm: int = 0          # NORM_PARALLEL: both sublayers read norm1(x)
+    layer_scale: int = 0       # NORM_PARALLEL: per-entry gains ls1 / ls2 on the sublayers' outputs
+    resid_mult: float = 0.0    # NORM_PARALLEL: factor of the sublayers' sum; 0 = 1
     arch: int = 2
     unused_tensors: frozenset = frozenset()  # checkpoint tensors the design names but this stack has no use for (skipped at load)
 
@@ -188,7 +192,7 @@ class StackDesc:
         arr = (LayerDescC * len(self.layers))(*[l.to_c() for l in self.layers])
         return StackDescC(self.width, self.vocab, len(self.layers), self.compute_f32, self.norm_eps, self.resid_alpha,
                           self.logit_softcap, self.norm_place, self.embed_norm, self.plain_gains, self.norm_kind, self.embed_scale,
-                          self.logit_scale, self.tie_head), arr
+                          self.logit_scale, self.tie_head, self.one_norm, self.layer_scale, self.resid_mult), arr
 
 
 @dataclass

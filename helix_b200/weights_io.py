@@ -280,8 +280,47 @@ def funudra_desc(cfg, shapes=None, compute_f32=False):
                      embed_norm=1, plain_gains=1, tie_head=1)
 
 
+def kamivik_desc(cfg, shapes=None, compute_f32=False):
+    """config.json of a Kamivik checkpoint -> StackDesc: layers whose two sublayers read one normed copy of the stream and are
+    added through per-entry gains and a common factor; latent attention with directly projected queries, interleaved rotation
+    and an ordinary softmax ("latent_attention": causal, one output gate per head; "latent_attention_2": sliding window, a
+    gate per output entry); mixtures of ungated erf-GELU experts (biased router logits, softmax over the chosen ones).  Every
+    size and every constant that may differ between checkpoints comes from the configuration."""
+    layers = []
+    for i, ly in enumerate(cfg["layers"]):
+        m = ly["mixer"]
+        d = LayerDesc(mixer=MIXER_LATENT, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                      rot_dim=int(m["rot_dim"]), scale=float(m["scale"]), attn_flags=_e.ATTN_NO_SINK, rope_pairing=1)
+        rot = m.get("rot")
+        if rot and rot.get("dims"):
+            d.rope_dims, d.rope_base = int(rot["dims"]), float(rot["base"])
+        if ly["type"] == "latent_attention":
+            d.mask, d.attn_flags = _e.MASK_CAUSAL, d.attn_flags | _e.ATTN_HEAD_GATE
+        elif ly["type"] == "latent_attention_2":
+            d.mask, d.window = _e.MASK_WINDOW, int(m["mask"]["size"])
+        else:
+            raise ValueError(f"layer {i}: unknown layer type {ly['type']!r}")
+        mlp = ly.get("mlp")
+        if mlp is not None:
+            if mlp.get("kind") != "moe":
+                raise ValueError(f"layer {i}: unsupported feed-forward kind {mlp.get('kind')!r}")
+            r = mlp["router"]
+            d.ff_kind, d.ff, d.experts, d.top_k = _e.FF_MOE, int(mlp["expert"]["ff"]), int(r["experts"]), int(r["top"])
+            d.router_kind, d.expert_kind, d.route_bias = _e.ROUTER_CHOSEN, _e.EXPERT_GELU, 1
+        layers.append(d)
+    mult = float(cfg.get("residual_mult", 1.0))
+    if mult == 0.0:
+        raise ValueError("a residual factor of zero is not representable (0 means 1)")
+    # a checkpoint may carry the second gain of a layer that has no feed-forward to scale
+    unused = frozenset(f"l{i}.ls2" for i, d in enumerate(layers) if d.ff == 0)
+    return StackDesc(unused_tensors=unused, width=int(cfg["width"]), vocab=int(cfg["vocab"]), layers=layers, compute_f32=int(bool(compute_f32)),
+                     norm_eps=float(cfg["norm"]["eps"]), resid_alpha=1.0, logit_softcap=0.0, norm_place=_e.NORM_PARALLEL,
+                     plain_gains=1, one_norm=1, layer_scale=1, resid_mult=mult)
+
+
 # layer-list decoders by config.json "architecture"
-STACK_READERS = {"Risepel": risepel_desc, "Lurepel": lurepel_desc, "Latanex": latanex_desc, "Funudra": funudra_desc}
+STACK_READERS = {"Risepel": risepel_desc, "Lurepel": lurepel_desc, "Latanex": latanex_desc, "Funudra": funudra_desc,
+                 "Kamivik": kamivik_desc}
 
 
 def desc_from_hf_config(cfg, shapes=None, compute_f32=False):

@@ -46,7 +46,7 @@
 extern "C" {
 #endif
 
-#define HB_ABI_VERSION 6
+#define HB_ABI_VERSION 7
 
 typedef enum hb_status {
   HB_OK = 0,
@@ -63,7 +63,7 @@ typedef enum hb_arch {
   HB_ARCH_BERT = 1,
   HB_ARCH_RISEPEL = 2, /* layer-list decoders (hb_stack_desc + hb_layer_desc[]): recurrent, latent-attention and grouped-query
                           mixers, gated / clamped / mixture-of-experts feed-forwards on a 32-bit residual stream (the Risepel,
-                          Lurepel and Latanex designs are settings of it); loaded with hb_model_load_begin_stack */
+                          Lurepel, Latanex, Funudra and Kamivik designs are settings of it); loaded with hb_model_load_begin_stack */
   HB_ARCH_STACK = 2
 } hb_arch;
 
@@ -126,6 +126,10 @@ typedef struct hb_model_desc {
  *                         expanded from a shared latent (kv_rank) plus one rotary key part (rot_dim) shared by all heads;
  *                         sliding window, learned per-head sink in the softmax denominator, sigmoid output gate.  kv_from >= 0:
  *                         the layer has no down-projection of its own and reads the cache rows of that earlier layer.
+ *                         Options: q_rank == 0: queries are projected straight from the layer input (mix.q, no query latent);
+ *                         mask HB_MASK_CAUSAL: every earlier position is seen; rope_pairing; attn_flags HB_ATTN_NO_SINK (an
+ *                         ordinary softmax, no mix.sink) and HB_ATTN_HEAD_GATE (mix.g has one row per head, head h's output
+ *                         times sigmoid of row h, instead of one row per output entry).
  *        HB_MIXER_GQA     grouped-query attention over cached per-head keys and values (kv_heads of them; query head h reads
  *                         head h / (heads / kv_heads)).  rope_dims leading entries of q and k rotate (rope_pairing, optional
  *                         wavelength-dependent frequency scaling rope_factor / rope_low / rope_high / rope_original); the
@@ -170,7 +174,9 @@ typedef struct hb_model_desc {
  *      Residual step (hb_stack_desc.norm_place): HB_NORM_OF_SUM x <- norm(alpha x + f(x)), HB_NORM_OF_OUTPUT
  *      x <- x + norm(f(x)), HB_NORM_BOTH_SIDES x <- x + norm_b(f(norm_a(x))) (norm1 / norm1b around the mixer, norm2 /
  *      norm2b around the feed-forward), or HB_NORM_PARALLEL x <- x + mixer(norm1(x)) + ff(norm2(x)): both sublayers read
- *      the same x (RMS norms; HB_FF_RELU2 and the gated units).  norm_kind: HB_NORM_RMS, or HB_NORM_TANH = tanh(alpha x) * w + b with a scalar
+ *      the same x (RMS norms; HB_FF_RELU2, the gated units and mixtures of experts); with one_norm both read norm1(x) and there
+ *      is no norm2.  layer_scale: the mixer's output is multiplied entry by entry by ls1, the feed-forward's by ls2, and
+ *      resid_mult (0 = 1) multiplies their sum (HB_NORM_PARALLEL).  norm_kind: HB_NORM_RMS, or HB_NORM_TANH = tanh(alpha x) * w + b with a scalar
  *      alpha and a vector b stored beside the gain as <name>.alpha and <name>.b (no statistic of the row; eps unused).
  *      f = mixer and, when ff > 0, the feed-forward (ff_kind):
  *        HB_FF_CLAMPED    g = min(gate, limit), u = clamp(up, +-limit), y = down(g sigmoid(1.702 g) (u + 1)), with biases
@@ -183,23 +189,26 @@ typedef struct hb_model_desc {
  *                         corrected scores and only experts of the route_keep best groups can be chosen; route_renorm: the
  *                         chosen scores are divided by their sum (+ 1e-20); route_scale (0 = 1) multiplies the weights;
  *                         expert_kind HB_EXPERT_CLAMPED: experts are clamped units (as HB_FF_CLAMPED without biases, limit
- *                         ff_limit); shared_ff > 0: one more unit of that inner size and kind (limit shared_limit,
+ *                         ff_limit), HB_EXPERT_GELU: experts are ungated units down(gelu_erf(up h)) (no e<j>.gate);
+ *                         router_kind HB_ROUTER_CHOSEN: the top_k largest logits are chosen and weighted by the softmax over
+ *                         the chosen logits alone; route_bias: mlp.router.b is added to the logits and there is no
+ *                         correction tensor; shared_ff > 0: one more unit of that inner size and kind (limit shared_limit,
  *                         mlp.shared.*) runs for every token and is added.
  *        HB_FF_SILU       y = down(silu(gate) * up), no biases
  *        HB_FF_RELU2      y = down(relu(up)^2): mlp.up, mlp.down, no gate, no biases
  *      Norm gains are stored as offsets from 1 unless plain_gains.  embed_norm: the embedding row is normed (embed.norm) before
  *      the first layer.  tie_head: the logits come from the embedding table (no head tensor).  Logits are soft-capped: cap * tanh(z / cap) (cap <= 0: off).  Tensor names: embed[.norm], final.norm,
- *      head, l<i>.norm1/2[b], l<i>.mix.{q,k,v,g,o,norm,a1,a2,a2.b | dq,dq.norm,uq,dkv,dkv.norm,uk,uv,sink,g,o | q,k,[v,]g,o |
+ *      head, l<i>.norm1/2[b], l<i>.ls1/2, l<i>.mix.{q,k,v,g,o,norm,a1,a2,a2.b | dq,dq.norm,uq (or q),dkv,dkv.norm,uk,uv,[sink,]g,o | q,k,[v,]g,o |
  *      q,k,v,{q,k,v}.conv,b,a,A_log,dt_bias,norm,g,o | in,conv,conv.b,dt_bias,A_log,D,norm,o | q,k,v,g,i,i.b,f,f.b,norm,o},
  *      l<i>.mlp.{gate,up,down}[.b] or
- *      l<i>.mlp.{router,correction,e<j>.gate,e<j>.up,e<j>.down[,shared.gate,shared.up,shared.down]}. ---- */
+ *      l<i>.mlp.{router,correction | router.b,[e<j>.gate,]e<j>.up,e<j>.down[,shared.gate,shared.up,shared.down]}. ---- */
 typedef enum hb_mixer { HB_MIXER_GLA = 0, HB_MIXER_LATENT = 1, HB_MIXER_GQA = 2, HB_MIXER_DELTA = 3, HB_MIXER_MAMBA2 = 4, HB_MIXER_MLSTM = 5 } hb_mixer;
 typedef enum hb_mask { HB_MASK_WINDOW = 0, HB_MASK_CHUNK = 1, HB_MASK_CAUSAL = 2 } hb_mask;
 typedef enum hb_ff_kind { HB_FF_CLAMPED = 0, HB_FF_GELU_TANH = 1, HB_FF_MOE = 2, HB_FF_SILU = 3, HB_FF_RELU2 = 4 } hb_ff_kind;
 typedef enum hb_norm_place { HB_NORM_OF_SUM = 0, HB_NORM_OF_OUTPUT = 1, HB_NORM_BOTH_SIDES = 2, HB_NORM_PARALLEL = 3 } hb_norm_place;
 typedef enum hb_norm_kind { HB_NORM_RMS = 0, HB_NORM_TANH = 1 } hb_norm_kind;
-typedef enum hb_router_kind { HB_ROUTER_SOFTMAX = 0, HB_ROUTER_SIGMOID = 1 } hb_router_kind;
-typedef enum hb_expert_kind { HB_EXPERT_SILU = 0, HB_EXPERT_CLAMPED = 1 } hb_expert_kind;
+typedef enum hb_router_kind { HB_ROUTER_SOFTMAX = 0, HB_ROUTER_SIGMOID = 1, HB_ROUTER_CHOSEN = 2 } hb_router_kind;
+typedef enum hb_expert_kind { HB_EXPERT_SILU = 0, HB_EXPERT_CLAMPED = 1, HB_EXPERT_GELU = 2 } hb_expert_kind;
 enum {
   HB_ATTN_QK_UNIT_NORM = 1,  /* q and k divided by their root mean square over dim after rotation (no gain) */
   HB_ATTN_V_IS_K = 2,        /* values are the key projections before rotation and normalisation; no mix.v tensor */
@@ -211,7 +220,8 @@ enum {
   HB_ATTN_V_BLEND = 128,     /* v <- (1 - l) v + l v_first (mix.vmix; the first such layer of the stack supplies v_first) */
   HB_ATTN_QKV_CONV = 256,    /* q, k, v (after their biases) pass a causal convolution over conv_taps tokens per channel */
   HB_ATTN_OUT_GATE = 512,    /* the concatenated heads times sigmoid(mix.g x) entry by entry (mix.g has heads * vdim rows) */
-  HB_ATTN_OUT_BIAS = 1024    /* the output projection has a bias (mix.o.b) */
+  HB_ATTN_OUT_BIAS = 1024,   /* the output projection has a bias (mix.o.b) */
+  HB_ATTN_NO_SINK = 2048     /* LATENT: no learned sink in the softmax denominator */
 };
 typedef struct hb_layer_desc {
   int32_t mixer;       /* hb_mixer */
@@ -226,9 +236,9 @@ typedef struct hb_layer_desc {
   int32_t ff;          /* 0: the layer has no feed-forward sublayer; HB_FF_MOE: inner size of one expert */
   float ff_limit;
   int32_t kv_heads;    /* GQA */
-  int32_t mask;        /* hb_mask (GQA; LATENT layers are HB_MASK_WINDOW) */
-  int32_t attn_flags;  /* HB_ATTN_* (GQA) */
-  int32_t rope_pairing;  /* 0: entry i pairs with i + rope_dims/2; 1: entry 2i pairs with 2i+1 (GQA) */
+  int32_t mask;        /* hb_mask (GQA; LATENT: HB_MASK_WINDOW or HB_MASK_CAUSAL) */
+  int32_t attn_flags;  /* HB_ATTN_* (GQA; LATENT: HB_ATTN_NO_SINK, HB_ATTN_HEAD_GATE) */
+  int32_t rope_pairing;  /* 0: entry i pairs with i + rope_dims/2; 1: entry 2i pairs with 2i+1 (GQA, LATENT) */
   float rope_factor, rope_low, rope_high; /* GQA: frequency scaling, rope_factor <= 0: off.  With wavelength l = 2 pi / f: f stays */
   int32_t rope_original;                  /* where l < original/high, becomes f/factor where l > original/low, blends between */
   int32_t ff_kind;     /* hb_ff_kind */
@@ -250,7 +260,8 @@ typedef struct hb_layer_desc {
   int32_t side_heads, side_dim, side_vdim;
   float side_gate_cap;
   float mix_scale, side_scale;      /* weights of the two mixers' outputs; 0 = 1 */
-  int32_t reserved[5];
+  int32_t route_bias;               /* HB_FF_MOE: 1: mlp.router.b joins the logits, no correction tensor */
+  int32_t reserved[4];
 } hb_layer_desc;
 typedef struct hb_stack_desc {
   int32_t width, vocab, n_layers;
@@ -263,7 +274,10 @@ typedef struct hb_stack_desc {
   float embed_scale;   /* x = embed[token] * embed_scale; 0 = 1 */
   float logit_scale;   /* logits = head(norm(x)) * logit_scale (before the soft cap); 0 = 1 */
   int32_t tie_head;    /* 1: the embedding table is the output matrix (no head tensor) */
-  int32_t reserved[4];
+  int32_t one_norm;    /* HB_NORM_PARALLEL: 1: both sublayers read norm1(x), no norm2 */
+  int32_t layer_scale; /* HB_NORM_PARALLEL: 1: gains ls1 / ls2 on the sublayers' outputs */
+  float resid_mult;    /* HB_NORM_PARALLEL: factor of the sublayers' sum; 0 = 1 */
+  int32_t reserved[1];
 } hb_stack_desc;
 
 typedef struct hb_sampling {
