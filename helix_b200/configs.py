@@ -157,6 +157,29 @@ def funudra_stack(width, layers, ff=None, vocab=32768, share=False, compute_f32=
                        norm_place=E.NORM_PARALLEL, embed_norm=1, plain_gains=1, tie_head=1)
 
 
+def kamivik_stack(width, layers, ff=None, window=1024, experts=16, top=4, kv_rank=512, vocab=32768, compute_f32=False):
+    """A Kamivik-design stack at sizes that resemble a served model's layers (random-init benchmarks): heads of 128 unrotated and
+    64 rotated query / key channels and 128 value channels over a latent of kv_rank entries; layers alternate attention over the
+    whole context (a gate per head) with a sliding window (a gate per entry); every layer has a mixture of `experts` ungated
+    experts of which a token uses `top`, sized so that a token spends the products of a dense gated unit of size ff."""
+    from . import engine as E
+    heads = max(1, width // 128)
+    ff = ff or (width * 4)
+    out = []
+    for i in range(layers):
+        l = E.LayerDesc(mixer=E.MIXER_LATENT, heads=heads, dim=128, vdim=128, kv_rank=kv_rank, rot_dim=64, rope_dims=64, rope_pairing=1,
+                        rope_base=500000.0 if i % 2 == 0 else 10000.0, scale=(128 + 64) ** -0.5, attn_flags=E.ATTN_NO_SINK)
+        if i % 2 == 0:
+            l.mask, l.attn_flags = E.MASK_CAUSAL, l.attn_flags | E.ATTN_HEAD_GATE
+        else:
+            l.mask, l.window = E.MASK_WINDOW, window
+        l.ff_kind, l.ff, l.experts, l.top_k = E.FF_MOE, max(64, 3 * ff // (2 * top)), experts, top
+        l.router_kind, l.expert_kind, l.route_bias = E.ROUTER_CHOSEN, E.EXPERT_GELU, 1
+        out.append(l)
+    return E.StackDesc(width=width, vocab=vocab, layers=out, compute_f32=int(compute_f32), norm_eps=1e-5, resid_alpha=1.0,
+                       norm_place=E.NORM_PARALLEL, plain_gains=1, one_norm=1, layer_scale=1, resid_mult=0.5)
+
+
 def llama_like(width, layers, ff, vocab=32768):
     """The closest existing decoder at equal width / depth / feed-forward size (comparison arm of the layer-list benchmarks)."""
     heads = max(1, width // 128)

@@ -399,12 +399,16 @@ __global__ void __launch_bounds__(128) latent_q_heads_kernel(const bf16* __restr
 template <int NQ>
 bool pick_rings(int nc, int np, Rings* rings, size_t* smem) {
   const size_t fixed = (size_t)(nc + 1) * NQ * 128 + 2 * NQ * 128 + 4 * NQ * 4 + (2 * kMaxC + 2 * kMaxR + 9) * 8 + 16 + 1024;
-  const size_t total = np <= 2 ? 113 * 1024 : 227 * 1024;  // narrow rows: two blocks per SM
+  const size_t total = np <= 2 && NQ == 16 ? 113 * 1024 : 227 * 1024;  // narrow rows: two blocks per SM
   if (fixed >= total) return false;
   const size_t room = total - fixed, tile = (size_t)np * kPair + kSub;
-  rings->rs = std::min<int>(kMaxR, (int)((room + tile - 1) / tile));
-  rings->cs = std::min<int>(kMaxC, (int)((room - (size_t)rings->rs * kSub) / kPair));
-  if (rings->cs < 2 * np || rings->rs < 2) return false;  // S of the next tile is issued while this tile's latents are held
+  // about as many rotated parts as tiles of latents; at least two tiles of both (S of the next tile is issued while this tile's
+  // latents are held)
+  int rs = std::min<int>(kMaxR, (int)((room + tile - 1) / tile));
+  while (rs > 2 && (room - (size_t)rs * kSub) / kPair < (size_t)2 * np) --rs;
+  if (rs < 2 || room < (size_t)rs * kSub + (size_t)2 * np * kPair) return false;
+  rings->rs = rs;
+  rings->cs = std::min<int>(kMaxC, (int)((room - (size_t)rs * kSub) / kPair));
   *smem = fixed + (size_t)rings->cs * kPair + (size_t)rings->rs * kSub;
   return true;
 }

@@ -99,6 +99,12 @@ def route(h, router, bias, top):
     return ids, e / e.sum(-1, keepdims=True)
 
 
+def route_margin(h, router, bias, top):
+    """how far the last chosen biased logit lies above the best one left out (inf when all are chosen), per token"""
+    z = -np.sort(-(h @ router.T + bias), axis=-1)
+    return z[:, top - 1] - z[:, top] if z.shape[1] > top else np.full(len(z), np.inf)
+
+
 def expert(h, up, down):
     return gelu_erf(h @ up.T) @ down.T
 
@@ -148,8 +154,9 @@ class KamivikOracle:
         o = gate_heads(o, h, p["g"]) if ly["type"] == "latent_attention" else gate_entries(o, h, p["g"])
         return o.reshape(h.shape[0], -1) @ p["o"].T
 
-    def forward(self, tokens, st=None, taps=None):
-        """tokens -> logits [T, vocab]; st is updated in place.  taps (a list) receives the stream after every layer."""
+    def forward(self, tokens, st=None, taps=None, margins=None):
+        """tokens -> logits [T, vocab]; st is updated in place.  taps / margins (lists) receive the stream after every layer /
+        every router's margins."""
         cfg, sd = self.cfg, self.sd
         st = self.new_state() if st is None else st
         pos = np.arange(st["pos"], st["pos"] + len(tokens))
@@ -158,9 +165,115 @@ class KamivikOracle:
             h = rms_norm(x, sd[f"l{i}.norm1"], self.eps)
             y = self.mixer(i, ly, h, st, pos) * sd[f"l{i}.ls1"]
             if ly.get("mlp") is not None:
+                if margins is not None:
+                    margins.append(route_margin(h, sd[f"l{i}.mlp.router"], sd[f"l{i}.mlp.router.b"], ly["mlp"]["router"]["top"]))
                 y = y + mixture(h, self.sub(f"l{i}.mlp."), ly["mlp"]) * sd[f"l{i}.ls2"]
             x = x + cfg["residual_mult"] * y
             if taps is not None:
                 taps.append(x.copy())
         st["pos"] += len(tokens)
         return rms_norm(x, sd["final.norm"], self.eps) @ sd["head"].T
+
+
+# ------------------------------------------------------------------ random checkpoints for tests
+FULL, WIN = "latent_attention", "latent_attention_2"
+
+
+def mixer_cfg(heads=3, dim=16, rot_dim=8, vdim=24, kv_rank=40, base=1000.0, window=None, scale=None):
+    m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, rot=dict(dims=rot_dim, base=float(base)),
+             scale=float(scale if scale is not None else (dim + rot_dim) ** -0.5))
+    if window:
+        m["mask"] = dict(size=window)
+    return m
+
+
+def random_config(width=96, vocab=120, order=((FULL, True), (WIN, True), (FULL, False)), full=None, win=None, window=37, experts=6, top=2, ff=40,
+                  mult=0.8, eps=1e-5, per_layer=None, per_mlp=None):
+    """order: (type, has a feed-forward) per layer; per_layer / per_mlp {i: dict}: that layer's mixer / feed-forward."""
+    layers = []
+    for i, (kind, has_ff) in enumerate(order):
+        mixer = dict(full or mixer_cfg()) if kind == FULL else dict(win or mixer_cfg(heads=4, dim=24, rot_dim=16, vdim=16, kv_rank=48, base=300.0))
+        if kind == WIN and "mask" not in mixer:
+            mixer["mask"] = dict(size=window)
+        if per_layer and i in per_layer:
+            mixer = per_layer[i]
+        mlp = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=experts, top=top)) if has_ff else None
+        if per_mlp and i in per_mlp:
+            mlp = per_mlp[i]
+        layers.append(dict(type=kind, mixer=mixer, mlp=mlp))
+    return dict(architecture="Kamivik", width=width, vocab=vocab, layers=layers, norm=dict(eps=eps), residual_mult=float(mult))
+
+
+def reserved(cfg):
+    """leading stream entries that no sublayer writes (their gains are zero): one per expert, then two for planted features"""
+    return max([ly["mlp"]["router"]["experts"] for ly in cfg["layers"] if ly["mlp"]] + [0]) + 2
+
+
+def random_state_dict(cfg, seed=0):
+    """Router choices are made by the leading stream entries, which hold a shuffled grid of values per token and stay as
+    embedded, so that no choice is a close call; everything else is random."""
+    from .weights import _rng, _t, to_bf16_f32
+    W, V = cfg["width"], cfg["vocab"]
+    s = lambda n: 1.0 / math.sqrt(n)
+    n_res = reserved(cfg)
+    E0 = n_res - 2
+    embed = _t(seed, "embed", (V, W), 0.5)
+    g = _rng(seed, "grid")
+    for v in range(V):
+        embed[v, :E0] = (g.permutation(E0) - (E0 - 1) / 2.0) * min(0.5, 4.0 / max(E0, 1))
+    embed[:, E0:n_res] = 0.0
+    sd = {"embed": to_bf16_f32(embed), "final.norm": _t(seed, "fn", (W,), 0.1, 1.0), "head": _t(seed, "head", (V, W), s(W))}
+    for i, ly in enumerate(cfg["layers"]):
+        m, p = ly["mixer"], f"l{i}."
+        H, Dk, Dr, Dv, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        sd[p + "norm1"] = _t(seed, p + "n1", (W,), 0.1, 1.0)
+        sd[p + "norm1"][:n_res] = 1.0
+        sd[p + "mix.q"] = _t(seed, p + "q", (H * (Dk + Dr), W), 1.5 * s(W))
+        sd[p + "mix.dkv"] = _t(seed, p + "dkv", (R + Dr, W), 1.5 * s(W))
+        sd[p + "mix.dkv.norm"] = _t(seed, p + "dkvn", (R,), 0.1, 1.0)
+        sd[p + "mix.uk"] = _t(seed, p + "uk", (H * Dk, R), 1.5 * s(R))
+        sd[p + "mix.uv"] = _t(seed, p + "uv", (H * Dv, R), 1.5 * s(R))
+        sd[p + "mix.g"] = _t(seed, p + "g", (H if ly["type"] == FULL else H * Dv, W), 1.5 * s(W))
+        sd[p + "mix.o"] = _t(seed, p + "o", (W, H * Dv), 2.0 * s(H * Dv))
+        for n in ("ls1", "ls2"):
+            gain = _t(seed, p + n, (W,), 0.2, 0.8)
+            gain[:n_res] = 0.0
+            if n == "ls1" or ly["mlp"]:
+                sd[p + n] = gain
+        if ly["mlp"]:
+            E, Fn = ly["mlp"]["router"]["experts"], ly["mlp"]["expert"]["ff"]
+            router = _t(seed, p + "router", (E, W), (0.3 if E0 <= 12 else 0.1) * s(W))
+            router[:, :n_res] = 0.0
+            for e in range(E):
+                router[e, e] = 8.0 / min(0.5, 4.0 / E0) * 0.5
+            sd[p + "mlp.router"] = to_bf16_f32(router)
+            sd[p + "mlp.router.b"] = _t(seed, p + "rb", (E,), 0.2)
+            for e in range(E):
+                sd[p + f"mlp.e{e}.up"] = _t(seed, p + f"e{e}u", (Fn, W), 2.0 * s(W))
+                sd[p + f"mlp.e{e}.down"] = _t(seed, p + f"e{e}d", (W, Fn), 2.0 * s(Fn))
+    return sd
+
+
+def plant_marker(cfg, sd, layers, strength=14.0):
+    """Token vocab - 1 becomes a marker: in the named layers every head's score for it stands out by `strength` wherever it is
+    seen, and its latent is unlike any other token's, so whether a position sees it shows in the logits."""
+    sd = {k: v.copy() for k, v in sd.items()}
+    const, mark = reserved(cfg) - 2, reserved(cfg) - 1
+    sd["embed"][:, const], sd["embed"][:, mark] = 1.0, 0.0
+    sd["embed"][-1, mark] = 4.0
+    for i in layers:
+        m, p = cfg["layers"][i]["mixer"], f"l{i}."
+        H, Dk, Dr, R = m["heads"], m["dim"], m["rot_dim"], m["kv_rank"]
+        sd[p + "mix.dkv.norm"][0] = 1.0
+        sd[p + "mix.dkv"][0] = 0.0
+        sd[p + "mix.dkv"][0, mark] = 16.0
+        for h in range(H):
+            q = sd[p + "mix.q"][h * (Dk + Dr):(h + 1) * (Dk + Dr)]
+            q *= 0.25
+            q[0] = 0.0
+            q[0, const] = float(np.float32(strength / (0.5 * math.sqrt(R) * m["scale"])))
+            uk = sd[p + "mix.uk"][h * Dk:(h + 1) * Dk]
+            uk[0] = 0.0
+            uk[0, 0] = 1.0
+    from .weights import to_bf16_f32
+    return {k: to_bf16_f32(v) for k, v in sd.items()}
