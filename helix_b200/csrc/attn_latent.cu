@@ -7,7 +7,7 @@
 //
 // Grid (splits, head groups, tokens).  A kv tile is one 64-position page; its 64-column sub-tiles travel in pairs through one
 // ring (16 KB slots) and the rotated part through a second ring, so loads of the next tiles overlap the products of this one.
-//   warp 0 : TMA producer      warp 1 : MMA issuer (S(j + 1) is issued before PV(j))
+//   warp 0 : TMA producer      warp 1 : MMA issuer, program order S(j) S(j + 1) PV(j) PV(j + 1)
 //   warps 2..5 : softmax.  The S^T tile of an M = 64 product sits in lanes 0..15 of every 32-lane quadrant; the running maximum is
 //                only reduced when some score passes it by more than 2^8 (the first tile, rarely later), sums stay per thread.
 // A second kernel merges the splits.  Further kernels here move rows into the layouts of the per-head products.
@@ -30,6 +30,7 @@ constexpr int kPair = 2 * kSub;
 constexpr int kMaxC = 12, kMaxR = 6;  // ring slots
 constexpr float kRescale = 8.0f;      // log2 units
 constexpr int kTokRows = kLatentTokRows;
+constexpr int kMaxSplits = 32;
 
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
@@ -62,10 +63,11 @@ struct Rings { int cs, rs; };  // slots of the latent-pair ring / of the rotated
 template <int NQ>
 __global__ void __launch_bounds__(kThreads)
 latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_constant__ CUtensorMap map_r,
+                     const __grid_constant__ CUtensorMap map_ql, const __grid_constant__ CUtensorMap map_qr,
                      const __grid_constant__ LatentDecodeArgs a, Rings rings, int num_splits) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int R = a.R, Dr = a.Dr;
+  const int R = a.R;
   const int nc = (R + 63) / 64, np = (nc + 1) / 2;
   const int CS = rings.cs, RS = rings.rs;
   uint8_t* ring_c = smem;                        // [CS][2][64 rows][128 B]
@@ -73,7 +75,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
   uint8_t* sQ = ring_r + RS * kSub;              // [nc + 1][NQ rows][128 B]
   uint8_t* sP = sQ + (nc + 1) * NQ * 128;        // [2][NQ rows][128 B]
   float* sRed = reinterpret_cast<float*>(sP + 2 * NQ * 128);  // [4 warps][NQ]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sRed + 4 * NQ);
+  float* sFac = sRed + 4 * NQ;                   // [NQ] rescale factors; at the end the maxima
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sFac + NQ);
   uint64_t* c_full = bars;
   uint64_t* c_empty = c_full + kMaxC;
   uint64_t* r_full = c_empty + kMaxC;
@@ -95,7 +98,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
   const int n_tiles = min(n_total, t_begin + tps) - t_begin;
   const int h0 = hg * NQ, nh = min(NQ, a.H - h0);
   float* ws = a.workspace + (((size_t)tq * gridDim.y + hg) * num_splits + split) * NQ * (R + 2);
+  pdl_launch_dependents();
   if (n_tiles <= 0) {
+    pdl_wait();  // the partials may still be read by an earlier launch's combine pass
     for (int i = threadIdx.x; i < NQ * (R + 2); i += kThreads) ws[i] = (i % (R + 2) == R) ? -INFINITY : 0.f;
     return;
   }
@@ -104,6 +109,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&map_c);
     tma_prefetch_desc(&map_r);
+    tma_prefetch_desc(&map_ql);
+    tma_prefetch_desc(&map_qr);
     for (int i = 0; i < CS; ++i) { mbar_init(&c_full[i], 1); mbar_init(&c_empty[i], 1); }
     for (int i = 0; i < RS; ++i) { mbar_init(&r_full[i], 1); mbar_init(&r_empty[i], 1); }
     for (int i = 0; i < 2; ++i) {
@@ -112,7 +119,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
       mbar_init(&p_full[i], 4);
       mbar_init(&pv_done[i], 1);
     }
-    mbar_init(q_ready, 4);
+    mbar_init(q_ready, 1);
     fence_barrier_init();
   }
   constexpr uint32_t kCols = NQ == 32 ? 256 : 128;  // two S tiles, up to four O blocks of NQ columns
@@ -125,11 +132,17 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
   tc_fence_after();
   const uint32_t tmem_base = __shfl_sync(0xffffffffu, *tmem_ptr, 0);
   const uint32_t tmem_S = tmem_base, tmem_O = tmem_base + 2 * NQ;
+  pdl_wait();  // launched while the kernel in front of it drains: nothing above depends on it
 
   if (warp == 0) {
     const bool elected = elect_one_sync();
     int cs = 0, rs = 0;
     uint32_t cph = 0, rph = 0;
+    if (elected) {  // the token's queries, one row per head (zeros where a head or an entry does not exist)
+      mbar_arrive_expect_tx(q_ready, (nc + 1) * NQ * 128);
+      for (int c = 0; c < nc; ++c) tma_load_3d(sQ + c * (NQ * 128), &map_ql, q_ready, c * 64, tq, h0);
+      tma_load_3d(sQ + nc * (NQ * 128), &map_qr, q_ready, 0, h0, tq);
+    }
     for (int j = 0; j < n_tiles; ++j) {
       const int row = pt[t_begin + j] * PAGE;
       for (int p = 0; p < np; ++p) {
@@ -153,82 +166,78 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
     const bool elected = elect_one_sync();
     constexpr uint32_t idesc_s = umma_idesc_bf16(PAGE, NQ, 0, 0);
     constexpr uint32_t idesc_o = umma_idesc_bf16(128, NQ, 1, 0);
-    const uint32_t c_addr = smem_u32(ring_c), r_addr = smem_u32(ring_r), q_addr = smem_u32(sQ), p_addr = smem_u32(sP);
+    // descriptors are a base per operand plus offsets in 16-byte units (the address field never carries)
+    const uint64_t kdesc0 = umma_desc_kmajor_sw128(smem_u32(ring_c)), rdesc0 = umma_desc_kmajor_sw128(smem_u32(ring_r));
+    const uint64_t qdesc0 = umma_desc_kmajor_sw128(smem_u32(sQ)), pdesc0 = umma_desc_kmajor_sw128(smem_u32(sP));
+    const uint64_t vdesc0 = umma_desc_mnmajor_sw128(smem_u32(ring_c), kSub, 1024);
     int cs = 0, rs = 0, vs = 0;  // ring slots of the next S pair / rotated part / PV pair
     uint32_t cph = 0, rph = 0;
     auto issue_s = [&](int j) {
       mbar_wait(&s_empty[j & 1], ((j >> 1) & 1) ^ 1);
       const uint32_t d = tmem_S + (j & 1) * NQ;
-      for (int c = 0; c < nc; ++c) {
-        if ((c & 1) == 0) {
-          mbar_wait(&c_full[cs], cph);
-          tc_fence_after();
-        }
+      uint64_t qd = qdesc0;
+      for (int p = 0; p < np; ++p) {
+        const bool two = 2 * p + 1 < nc;
+        mbar_wait(&c_full[cs], cph);
+        tc_fence_after();
+        const uint64_t kd = kdesc0 + (uint64_t)(cs * (kPair >> 4));
         if (elected) {
 #pragma unroll
-          for (int k = 0; k < 4; ++k)
-            umma_f16_ss(d, umma_desc_kmajor_sw128(c_addr + cs * kPair + (c & 1) * kSub + k * 32),
-                        umma_desc_kmajor_sw128(q_addr + c * (NQ * 128) + k * 32), idesc_s, (c | k) != 0 ? 1u : 0u);
+          for (int k = 0; k < 4; ++k) umma_f16_ss(d, kd + k * 2, qd + k * 2, idesc_s, k != 0 ? 1u : (p != 0 ? 1u : 0u));
+          if (two) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k) umma_f16_ss(d, kd + (kSub >> 4) + k * 2, qd + (NQ * 128 >> 4) + k * 2, idesc_s, 1u);
+          }
         }
-        if ((c & 1) || c == nc - 1) { if (++cs == CS) { cs = 0; cph ^= 1; } }
+        qd += two ? 2 * (NQ * 128 >> 4) : (NQ * 128 >> 4);
+        if (++cs == CS) { cs = 0; cph ^= 1; }
       }
       mbar_wait(&r_full[rs], rph);
       tc_fence_after();
       if (elected) {
+        const uint64_t rd = rdesc0 + (uint64_t)(rs * (kSub >> 4));
 #pragma unroll
-        for (int k = 0; k < 4; ++k)
-          umma_f16_ss(d, umma_desc_kmajor_sw128(r_addr + rs * kSub + k * 32), umma_desc_kmajor_sw128(q_addr + nc * (NQ * 128) + k * 32), idesc_s, 1u);
+        for (int k = 0; k < 4; ++k) umma_f16_ss(d, rd + k * 2, qd + k * 2, idesc_s, 1u);
         umma_commit(&r_empty[rs]);
         umma_commit(&s_full[j & 1]);
       }
       if (++rs == RS) { rs = 0; rph ^= 1; }
     };
-    mbar_wait(q_ready, 0);
-    tc_fence_after();
-    issue_s(0);
-    for (int j = 0; j < n_tiles; ++j) {
-      if (j + 1 < n_tiles) issue_s(j + 1);
+    auto issue_pv = [&](int j) {
       mbar_wait(&p_full[j & 1], (j >> 1) & 1);
       tc_fence_after();
       for (int p = 0; p < np; ++p) {
         if (elected) {
 #pragma unroll
           for (int k = 0; k < 4; ++k)
-            umma_f16_ss(tmem_O + p * NQ, umma_desc_mnmajor_sw128(c_addr + vs * kPair + k * (16 * 128), kSub, 1024),
-                        umma_desc_kmajor_sw128(p_addr + (j & 1) * (NQ * 128) + k * 32), idesc_o, (j | k) != 0 ? 1u : 0u);
+            umma_f16_ss(tmem_O + p * NQ, vdesc0 + (uint64_t)(vs * (kPair >> 4)) + k * (16 * 128 >> 4),
+                        pdesc0 + (uint64_t)((j & 1) * (NQ * 128 >> 4)) + k * 2, idesc_o, k != 0 ? 1u : (j != 0 ? 1u : 0u));
           umma_commit(&c_empty[vs]);
         }
         if (++vs == CS) vs = 0;
       }
       if (elected) umma_commit(&pv_done[j & 1]);
+    };
+    // two tiles at a time: while the slots of the first are refilled, the tensor pipe works on the second
+    mbar_wait(q_ready, 0);
+    tc_fence_after();
+    for (int j = 0; j < n_tiles; j += 2) {
+      issue_s(j);
+      if (j + 1 < n_tiles) issue_s(j + 1);
+      issue_pv(j);
+      if (j + 1 < n_tiles) issue_pv(j + 1);
     }
   } else {
     const int qd = warp & 3;
     const int t = qd * 32 + lane;
     const uint32_t lane_sel = static_cast<uint32_t>(qd * 32) << 16;
-    {  // queries into the K-major swizzled B-operand layout, zeros where a head, a latent entry or a rotated entry does not exist
-      const int Dq = a.Dk + Dr;
-      for (int i = t; i < (nc + 1) * NQ * 8; i += 128) {
-        const int ch = i & 7, g = (i >> 3) % NQ, c = (i >> 3) / NQ;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (g < nh) {
-          if (c < nc) {
-            if (c * 64 + ch * 8 < R) v = *reinterpret_cast<const uint4*>(a.q_lat + ((size_t)(h0 + g) * kTokRows + tq) * R + c * 64 + ch * 8);
-          } else if (ch * 8 < Dr) {
-            v = *reinterpret_cast<const uint4*>(a.q + (size_t)tq * a.ldq + (size_t)(h0 + g) * Dq + a.Dk + ch * 8);
-          }
-        }
-        *reinterpret_cast<uint4*>(sQ + c * (NQ * 128) + g * 128 + ((ch ^ (g & 7)) << 4)) = v;
-      }
-      fence_proxy_async_smem();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(q_ready);
-    }
-    const bool row_lane = lane < 16;      // lanes that hold a row of S^T
-    const int kv = qd * 16 + lane;        // its position within the tile
-    float m_used[NQ], l_run[NQ];
+    // lanes 0..15 hold the rows of S^T; lane l + 16 takes the upper half of the heads of lane l's row
+    constexpr int HN = NQ / 2;
+    const int kv = qd * 16 + (lane & 15);  // position within the tile
+    const int g0 = lane < 16 ? 0 : HN;     // first head of this lane
+    float m_used[HN], l_run[HN];
 #pragma unroll
-    for (int g = 0; g < NQ; ++g) { m_used[g] = -INFINITY; l_run[g] = 0.f; }
+    for (int g = 0; g < HN; ++g) { m_used[g] = -INFINITY; l_run[g] = 0.f; }
     const float scale_log2 = a.scale * 1.4426950408889634f;
     for (int j = 0; j < n_tiles; ++j) {
       mbar_wait(&s_full[j & 1], (j >> 1) & 1);
@@ -240,12 +249,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[j & 1]);
       const int pos = (t_begin + j) * PAGE + kv;
-      const bool valid = row_lane && pos < ctx && pos >= kv_lo;
-      float sc[NQ];
+      const bool valid = pos < ctx && pos >= kv_lo;
+      float sc[HN];
       bool need = j == 0;
 #pragma unroll
-      for (int g = 0; g < NQ; ++g) {
-        sc[g] = valid ? __uint_as_float(sv[g]) * scale_log2 : -INFINITY;
+      for (int g = 0; g < HN; ++g) {
+        const uint32_t up = __shfl_sync(0xffffffffu, sv[HN + g], lane & 15);
+        sc[g] = valid ? __uint_as_float(lane < 16 ? sv[g] : up) * scale_log2 : -INFINITY;
         need |= sc[g] > m_used[g] + kRescale;
       }
       if (j >= 2) {  // the P buffer is free
@@ -254,50 +264,47 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
       }
       if (bar_any(need)) {
 #pragma unroll
-        for (int g = 0; g < NQ; ++g) {
+        for (int g = 0; g < HN; ++g) {
           float mx = sc[g];
 #pragma unroll
           for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-          if (lane == 0) sRed[qd * NQ + g] = mx;
+          if ((lane & 15) == 0) sRed[qd * NQ + g0 + g] = mx;
         }
         bar_sync(1, 128);
+#pragma unroll
+        for (int g = 0; g < HN; ++g) {
+          const int h = g0 + g;
+          const float tm = fmaxf(fmaxf(sRed[h], sRed[NQ + h]), fmaxf(sRed[2 * NQ + h], sRed[3 * NQ + h]));
+          float f = 1.f;
+          if (tm > m_used[g] + kRescale) {  // the first tile too (m_used = -inf; some position of every tile is visible)
+            f = m_used[g] == -INFINITY ? 0.f : fast_exp2(m_used[g] - tm);
+            m_used[g] = tm;
+            l_run[g] *= f;
+          }
+          if (qd == 0 && (lane & 15) == 0) sFac[h] = f;
+        }
+        bar_sync(1, 128);  // sRed may be rewritten, sFac is complete
         if (j > 0) {
           mbar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1);  // O^T is consistent
           tc_fence_after();
-        }
-        float f[NQ];
-#pragma unroll
-        for (int g = 0; g < NQ; ++g) {
-          const float tm = fmaxf(fmaxf(sRed[g], sRed[NQ + g]), fmaxf(sRed[2 * NQ + g], sRed[3 * NQ + g]));
-          f[g] = 1.f;
-          if (tm > m_used[g] + kRescale) {  // the first tile too (m_used = -inf; some position of every tile is visible)
-            f[g] = m_used[g] == -INFINITY ? 0.f : fast_exp2(m_used[g] - tm);
-            m_used[g] = tm;
-            l_run[g] *= f[g];
-          }
-        }
-        if (j > 0) {
           for (int p = 0; p < np; ++p) {
             uint32_t o[NQ];
             tmem_ld_cols<NQ>(tmem_O + lane_sel + p * NQ, o);
             tmem_ld_wait();
 #pragma unroll
-            for (int g = 0; g < NQ; ++g) o[g] = __float_as_uint(__uint_as_float(o[g]) * f[g]);
+            for (int g = 0; g < NQ; ++g) o[g] = __float_as_uint(__uint_as_float(o[g]) * sFac[g]);
             tmem_st_32x32b_x16(tmem_O + lane_sel + p * NQ, *reinterpret_cast<uint32_t(*)[16]>(&o[0]));
             if constexpr (NQ == 32) tmem_st_32x32b_x16(tmem_O + lane_sel + p * NQ + 16, *reinterpret_cast<uint32_t(*)[16]>(&o[16]));
           }
           tmem_st_wait();
         }
-        bar_sync(1, 128);  // sRed may be rewritten
       }
-      if (row_lane) {
-        uint8_t* dst = sP + (j & 1) * (NQ * 128) + (kv & 7) * 2;
+      uint8_t* dst = sP + (j & 1) * (NQ * 128) + g0 * 128 + (kv & 7) * 2;
 #pragma unroll
-        for (int g = 0; g < NQ; ++g) {
-          const float pr = fast_exp2(sc[g] - m_used[g]);
-          l_run[g] += pr;
-          *reinterpret_cast<bf16*>(dst + g * 128 + (((kv >> 3) ^ (g & 7)) << 4)) = __float2bfloat16(pr);
-        }
+      for (int g = 0; g < HN; ++g) {  // g0 is a multiple of 8: the swizzle phase of row g0 + g is g & 7
+        const float pr = fast_exp2(sc[g] - m_used[g]);
+        l_run[g] += pr;
+        *reinterpret_cast<bf16*>(dst + g * 128 + (((kv >> 3) ^ (g & 7)) << 4)) = __float2bfloat16(pr);
       }
       fence_proxy_async_smem();
       tc_fence_before();
@@ -305,16 +312,19 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
       if (lane == 0) mbar_arrive(&p_full[j & 1]);
     }
     // ---- epilogue: O^T lane r, column g; l over all positions of the split
-    mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1);
-    tc_fence_after();
 #pragma unroll
-    for (int g = 0; g < NQ; ++g) {
+    for (int g = 0; g < HN; ++g) {
       float v = l_run[g];
 #pragma unroll
       for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-      if (lane == 0) sRed[qd * NQ + g] = v;
+      if ((lane & 15) == 0) sRed[qd * NQ + g0 + g] = v;
+      if (qd == 0 && (lane & 15) == 0) sFac[g0 + g] = m_used[g];
     }
     bar_sync(1, 128);
+    if (t < NQ) sRed[t] = (sRed[t] + sRed[NQ + t]) + (sRed[2 * NQ + t] + sRed[3 * NQ + t]);
+    bar_sync(1, 128);
+    mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1);
+    tc_fence_after();
     for (int p = 0; p < np; ++p) {
       uint32_t o[NQ];
       tmem_ld_cols<NQ>(tmem_O + lane_sel + p * NQ, o);
@@ -325,8 +335,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
 #pragma unroll
           for (int g = 0; g < NQ; ++g) {
             if (g >= nh) break;
-            float lg = (sRed[g] + sRed[NQ + g]) + (sRed[2 * NQ + g] + sRed[3 * NQ + g]);
-            if (a.sink) lg += fast_exp2(__bfloat162float(a.sink[h0 + g]) * 1.4426950408889634f - m_used[g]);
+            float lg = sRed[g];
+            if (a.sink) lg += fast_exp2(__bfloat162float(a.sink[h0 + g]) * 1.4426950408889634f - sFac[g]);
             a.ctx[((size_t)(h0 + g) * kTokRows + tq) * R + r] = __float2bfloat16(__uint_as_float(o[g]) / lg);
           }
         } else {
@@ -335,12 +345,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
         }
       }
     }
-    if (num_splits > 1 && t == 0) {
-#pragma unroll
-      for (int g = 0; g < NQ; ++g) {
-        ws[(size_t)g * (R + 2) + R] = m_used[g];
-        ws[(size_t)g * (R + 2) + R + 1] = (sRed[g] + sRed[NQ + g]) + (sRed[2 * NQ + g] + sRed[3 * NQ + g]);
-      }
+    if (num_splits > 1 && t < NQ) {
+      ws[(size_t)t * (R + 2) + R] = sFac[t];
+      ws[(size_t)t * (R + 2) + R + 1] = sRed[t];
     }
   }
   tc_fence_before();
@@ -351,24 +358,38 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
   }
 }
 
-// merges the splits of one (head, token)
+// merges the splits of one (head, token): every thread weighs the splits itself (their maxima and sums are a few loads that all
+// threads share), then sums four latent entries per pass
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ ws, bf16* __restrict__ ctx, const bf16* __restrict__ sink,
                                                              int R, int NQ, int groups, int num_splits) {
+  __shared__ float wts[kMaxSplits];
+  pdl_wait();
   const int h = blockIdx.x, tq = blockIdx.y, hg = h / NQ, g = h % NQ;
   const float* base = ws + ((size_t)tq * groups + hg) * num_splits * NQ * (R + 2) + (size_t)g * (R + 2);
   const size_t stride = (size_t)NQ * (R + 2);
-  float m = -INFINITY;
-  for (int s = 0; s < num_splits; ++s) m = fmaxf(m, base[s * stride + R]);
-  float l = sink ? fast_exp2(__bfloat162float(sink[h]) * 1.4426950408889634f - m) : 0.f;
-  for (int s = 0; s < num_splits; ++s) l += fast_exp2(base[s * stride + R] - m) * base[s * stride + R + 1];
-  const float inv = 1.f / l;
-  for (int r = threadIdx.x; r < R; r += 128) {
-    float o = 0.f;
+  if (threadIdx.x < 32) {
+    const int s = threadIdx.x;
+    const float ms = s < num_splits ? base[s * stride + R] : -INFINITY, ls = s < num_splits ? base[s * stride + R + 1] : 0.f;
+    float m = ms;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+    const float w = ms == -INFINITY ? 0.f : fast_exp2(ms - m);
+    float l = w * ls;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+    if (sink) l += fast_exp2(__bfloat162float(sink[h]) * 1.4426950408889634f - m);
+    wts[s] = w / l;
+  }
+  __syncthreads();
+  for (int r = threadIdx.x * 2; r < R; r += 256) {  // R is a multiple of 8
+    float2 o = make_float2(0.f, 0.f);
+#pragma unroll 4
     for (int s = 0; s < num_splits; ++s) {
-      const float ms = base[s * stride + R];
-      if (ms != -INFINITY) o = fmaf(fast_exp2(ms - m), base[s * stride + r], o);
+      const float2 v = *reinterpret_cast<const float2*>(base + s * stride + r);
+      o.x = fmaf(wts[s], v.x, o.x);
+      o.y = fmaf(wts[s], v.y, o.y);
     }
-    ctx[((size_t)h * kTokRows + tq) * R + r] = __float2bfloat16(o * inv);
+    *reinterpret_cast<__nv_bfloat162*>(ctx + ((size_t)h * kTokRows + tq) * R + r) = __floats2bfloat162_rn(o.x, o.y);
   }
 }
 
@@ -398,7 +419,7 @@ __global__ void __launch_bounds__(128) latent_q_heads_kernel(const bf16* __restr
 
 template <int NQ>
 bool pick_rings(int nc, int np, Rings* rings, size_t* smem) {
-  const size_t fixed = (size_t)(nc + 1) * NQ * 128 + 2 * NQ * 128 + 4 * NQ * 4 + (2 * kMaxC + 2 * kMaxR + 9) * 8 + 16 + 1024;
+  const size_t fixed = (size_t)(nc + 1) * NQ * 128 + 2 * NQ * 128 + 5 * NQ * 4 + (2 * kMaxC + 2 * kMaxR + 9) * 8 + 16 + 1024;
   const size_t total = np <= 2 && NQ == 16 ? 113 * 1024 : 227 * 1024;  // narrow rows: two blocks per SM
   if (fixed >= total) return false;
   const size_t room = total - fixed, tile = (size_t)np * kPair + kSub;
@@ -421,15 +442,16 @@ cudaError_t launch_decode(cudaStream_t s, const LatentDecodeArgs& a) {
   Rings rings;
   size_t smem = 0;
   if (!pick_rings<NQ>(nc, np, &rings, &smem)) return cudaErrorInvalidValue;
-  CUtensorMap mc, mr;
+  CUtensorMap mc, mr, mql, mqr;
   const uint64_t rows = (uint64_t)a.num_pages * PAGE, stride = (uint64_t)(a.R + a.Dr) * 2;
   if (!make_tmap_2d(&mc, a.cache, TM_BF16, a.R, rows, stride, 64, PAGE)) return cudaErrorInvalidValue;
   if (!make_tmap_2d(&mr, a.cache + a.R, TM_BF16, a.Dr, rows, stride, 64, PAGE)) return cudaErrorInvalidValue;
-  latent_decode_kernel<NQ><<<dim3(a.num_splits, groups, a.T), kThreads, smem, s>>>(mc, mr, a, rings, a.num_splits);
-  cudaError_t e = cudaGetLastError();
+  const uint64_t qs = (uint64_t)(a.Dk + a.Dr) * 2;
+  if (!make_tmap_3d(&mql, a.q_lat, TM_BF16, a.R, kTokRows, a.H, (uint64_t)a.R * 2, (uint64_t)kTokRows * a.R * 2, 64, 1, NQ)) return cudaErrorInvalidValue;
+  if (!make_tmap_3d(&mqr, a.q + a.Dk, TM_BF16, a.Dr, a.H, a.T, qs, (uint64_t)a.ldq * 2, 64, NQ, 1)) return cudaErrorInvalidValue;
+  cudaError_t e = launch_k(latent_decode_kernel<NQ>, dim3(a.num_splits, groups, a.T), dim3(kThreads), smem, s, true, mc, mr, mql, mqr, a, rings, a.num_splits);
   if (e != cudaSuccess || a.num_splits == 1) return e;
-  latent_combine_kernel<<<dim3(a.H, a.T), 128, 0, s>>>(a.workspace, a.ctx, a.sink, a.R, NQ, groups, a.num_splits);
-  return cudaGetLastError();
+  return launch_k(latent_combine_kernel, dim3(a.H, a.T), dim3(128), 0, s, true, (const float*)a.workspace, a.ctx, a.sink, a.R, NQ, groups, a.num_splits);
 }
 
 }  // namespace
@@ -440,7 +462,7 @@ bool latent_decode_ok(int Dk, int R, int Dr) {
 int latent_decode_splits(int T, int H, int max_keys, int sms) {
   const int blocks = T * ((H + pick_nq(H) - 1) / pick_nq(H));
   const int tiles = std::max(1, (max_keys + PAGE - 1) / PAGE);
-  return std::max(1, std::min(std::min(32, (tiles + 1) / 2), sms / std::max(1, blocks)));
+  return std::max(1, std::min(std::min(kMaxSplits, (tiles + 1) / 2), sms / std::max(1, blocks)));
 }
 size_t latent_decode_ws_floats(int T, int H, int R, int splits) {
   return splits <= 1 ? 0 : (size_t)T * ((H + pick_nq(H) - 1) / pick_nq(H)) * splits * pick_nq(H) * (R + 2);
@@ -453,7 +475,7 @@ cudaError_t attn_latent_init() {
 
 cudaError_t latent_decode(cudaStream_t s, const LatentDecodeArgs& a) {
   if (a.T <= 0) return cudaSuccess;
-  if (a.T > kTokRows || !latent_decode_ok(a.Dk, a.R, a.Dr) || a.page_size != PAGE || a.num_splits < 1 || a.num_pages <= 0 || a.window < 0 ||
+  if (a.T > kTokRows || !latent_decode_ok(a.Dk, a.R, a.Dr) || a.page_size != PAGE || a.num_splits < 1 || a.num_splits > kMaxSplits || a.num_pages <= 0 || a.window < 0 ||
       a.ldq % 8 || (a.num_splits > 1 && !a.workspace))
     return cudaErrorInvalidValue;
   return pick_nq(a.H) == 16 ? launch_decode<16>(s, a) : launch_decode<32>(s, a);

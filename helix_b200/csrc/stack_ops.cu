@@ -459,6 +459,37 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
   const int t = blockIdx.x;
   const float* p = a.p + (size_t)t * a.ldp;
   const float* cs = a.rope_dims > 0 ? a.cs + (size_t)t * a.rope_dims : nullptr;
+  if (blockIdx.y > 0) {  // query heads as bf16, eight entries per thread (head parts are multiples of eight)
+    const int Dq = a.Dk + a.Dr, i8 = (blockIdx.y - 1) * blockDim.x + threadIdx.x;
+    if (i8 >= a.H * Dq / 8) return;
+    const int tq = t - a.qh_t0, h = i8 * 8 / Dq, e = i8 * 8 - h * Dq, er = e - a.Dk;
+    const float* src = p + a.q_off + (size_t)h * Dq;
+    const float4 x = *reinterpret_cast<const float4*>(src + e), y = *reinterpret_cast<const float4*>(src + e + 4);
+    float v[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
+    if (er >= 0 && er < a.rope_dims) {
+      if (a.pairing && er + 8 <= a.rope_dims && (a.rope_dims & 3) == 0 && ((uintptr_t)a.cs & 15) == 0) {  // four whole pairs, their cosines and sines side by side
+        const float4 c0 = *reinterpret_cast<const float4*>(cs + er), c1 = *reinterpret_cast<const float4*>(cs + er + 4);
+        const float cc[8] = {c0.x, c0.y, c0.z, c0.w, c1.x, c1.y, c1.z, c1.w};
+#pragma unroll
+        for (int k = 0; k < 8; k += 2) {
+          const float u = v[k], w = v[k + 1];
+          v[k] = u * cc[k] - w * cc[k + 1];
+          v[k + 1] = w * cc[k] + u * cc[k + 1];
+        }
+      } else {
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          if (er + k < a.rope_dims) v[k] = rope_entry(src + a.Dk, er + k, cs, a.rope_dims, a.pairing);
+      }
+    }
+    __nv_bfloat162 b[4] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3]), __floats2bfloat162_rn(v[4], v[5]),
+                           __floats2bfloat162_rn(v[6], v[7])};
+    const uint4 u = *reinterpret_cast<uint4*>(b);
+    *reinterpret_cast<uint4*>(a.q16 + (size_t)t * a.H * Dq + i8 * 8) = u;
+    if (a.qh && e < a.Dk && tq >= 0 && tq < kLatentTokRows)
+      *reinterpret_cast<uint4*>(a.qh + ((size_t)h * kLatentTokRows + tq) * a.Dk + e) = u;
+    return;
+  }
   if (a.Q > 0) {
     float ss = 0.f;
     for (int i = threadIdx.x; i < a.Q; i += blockDim.x) ss += p[a.q_off + i] * p[a.q_off + i];
@@ -468,29 +499,6 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
       const float v = p[a.q_off + i] * rs * ldf<WT>((const WT*)a.wq, i);
       a.cq[(size_t)t * a.Q + i] = v;
       if (a.cq_b16) a.cq_b16[(size_t)t * a.Q + i] = __float2bfloat16(v);
-    }
-  }
-  if (a.q16) {  // query heads as bf16, eight entries per thread (head parts are multiples of eight)
-    const int Dq = a.Dk + a.Dr, n8 = a.H * Dq / 8;
-    const int tq = t - a.qh_t0;
-    for (int i8 = threadIdx.x; i8 < n8; i8 += blockDim.x) {
-      const int h = i8 * 8 / Dq, e = i8 * 8 - h * Dq;
-      const float* src = p + a.q_off + (size_t)h * Dq;
-      float v[8];
-      if (e < a.Dk || e - a.Dk >= a.rope_dims) {
-        const float4 x = *reinterpret_cast<const float4*>(src + e), y = *reinterpret_cast<const float4*>(src + e + 4);
-        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
-      } else {
-#pragma unroll
-        for (int k = 0; k < 8; ++k)
-          v[k] = e - a.Dk + k < a.rope_dims ? rope_entry(src + a.Dk, e - a.Dk + k, cs, a.rope_dims, a.pairing) : src[e + k];
-      }
-      __nv_bfloat162 b[4] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3]), __floats2bfloat162_rn(v[4], v[5]),
-                             __floats2bfloat162_rn(v[6], v[7])};
-      const uint4 u = *reinterpret_cast<uint4*>(b);
-      *reinterpret_cast<uint4*>(a.q16 + (size_t)t * a.H * Dq + i8 * 8) = u;
-      if (a.qh && e < a.Dk && tq >= 0 && tq < kLatentTokRows)
-        *reinterpret_cast<uint4*>(a.qh + ((size_t)h * kLatentTokRows + tq) * a.Dk + e) = u;
     }
   }
   if (a.kv_off < 0) return;
@@ -996,8 +1004,10 @@ cudaError_t latent_prep(cudaStream_t s, const LatentPrepArgs& a) {
   if (a.T <= 0) return cudaSuccess;
   if (a.rope_dims % 2 || a.rope_dims > a.Dr || (a.rope_dims > 0 && !a.cs)) return cudaErrorInvalidValue;
   if (a.q16 && (a.Dk % 8 || a.Dr % 8 || a.ldp % 4 || a.q_off % 4 || ((uintptr_t)a.p & 15))) return cudaErrorInvalidValue;
-  if (a.f32) latent_prep_kernel<float, float><<<a.T, 256, 0, s>>>(a);
-  else latent_prep_kernel<bf16, bf16><<<a.T, 256, 0, s>>>(a);
+  // block (t, 0): the query latent and the cache row; blocks (t, 1 ..): the query heads
+  dim3 grid(a.T, 1 + (a.q16 ? (a.H * (a.Dk + a.Dr) / 8 + 255) / 256 : 0));
+  if (a.f32) latent_prep_kernel<float, float><<<grid, 256, 0, s>>>(a);
+  else latent_prep_kernel<bf16, bf16><<<grid, 256, 0, s>>>(a);
   return KERR();
 }
 
