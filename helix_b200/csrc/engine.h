@@ -214,7 +214,7 @@ class Engine {
     int att_qb = 0;       // tokens per query block
     size_t att_rows = 0, att_keys = 0;  // capacity: score rows (tokens x heads) and key columns of one block
     // mixture of experts: router logits [T][ldz], chosen outputs and their weights [T][top_k], expert outputs [(T, top_k)][W]
-    float *moe_z = nullptr, *moe_w = nullptr, *moe_y = nullptr;
+    float *moe_z = nullptr, *moe_w = nullptr, *moe_y = nullptr, *moe_h = nullptr;
     int32_t* moe_ids = nullptr;
     int ldz = 0;
     float* dec_ws = nullptr;  // split partials of the tensor-core decode attention (grouped-query layers, bf16 mode)

@@ -224,6 +224,7 @@ struct StackDims {
   int gu = 0;                // widest [gate | up] row of a plain gated unit (bf16 intermediate of the tensor-core path)
   int att_heads = 0, att_dim = 0;  // ... and their most heads / widest head (split workspace of the decode kernel)
   int att = 0;               // grouped-query layers the fused tcgen05 attention takes: widest heads * vdim
+  size_t moe_h = 0;          // inner activations of experts that run item by item (floats)
   int moe_e = 0, moe_f = 0;  // grouped tensor-core experts: most experts / widest expert over the layers that qualify
   int vf = 0;                // layers that blend values: kv_heads * vdim
   bool shared = false;       // some mixture has a unit every token uses
@@ -246,7 +247,7 @@ static bool moe_grouped_ok(const Model& m, const hb_layer_desc& l) {
   return !off && !m.sd.compute_f32 && l.ff > 0 && l.ff_kind == HB_FF_MOE && m.sd.width % 8 == 0 && l.ff % 8 == 0 && m.sd.width >= 64 &&
          l.ff >= 64;
 }
-static StackDims stack_dims(const Model& m, int max_ctx) {
+static StackDims stack_dims(const Model& m, int max_ctx, int tokens) {
   StackDims d;
   for (int i = 0; i < m.sd.n_layers; ++i) {
     const hb_layer_desc& l = m.sl[i];
@@ -309,6 +310,9 @@ static StackDims stack_dims(const Model& m, int max_ctx) {
     if (l.ff > 0 && l.ff_kind == HB_FF_MOE) {
       d.moe_r = std::max(d.moe_r, l.experts + l.identity_experts);
       d.moe_top = std::max(d.moe_top, l.top_k);
+      // grouped experts run item by item only in steps of fewer than 2 E items
+      const size_t items = (size_t)tokens * l.top_k;
+      d.moe_h = std::max(d.moe_h, (moe_grouped_ok(m, l) ? std::min<size_t>(items, 2 * (size_t)l.experts) : items) * l.ff);
       if (moe_grouped_ok(m, l)) {
         d.moe_e = std::max(d.moe_e, l.experts);
         d.moe_f = std::max(d.moe_f, l.ff);
@@ -321,14 +325,15 @@ static StackDims stack_dims(const Model& m, int max_ctx) {
 size_t Engine::workspace_bytes_stack() const {
   const hb_stack_desc& sd = model_.sd;
   const size_t T = t_cap_, W = sd.width;
-  const StackDims dm = stack_dims(model_, cfg_.max_ctx);
+  const StackDims dm = stack_dims(model_, cfg_.max_ctx, t_cap_);
   const int n1 = dm.n1, n2 = dm.n2, q = dm.q, qa = dm.qa, cx = dm.cx, mo = dm.mo;
   size_t b = 0;
   b += al256((size_t)std::max(dm.rope_half, 1) * 8) + al256(T * 2 * (size_t)std::max(dm.rope_half, 1) * 4);
   if (dm.att > 0) b += al256(T * (size_t)up8(dm.att) * 2) + al256(attn_decode_workspace_floats(cfg_.max_seqs, dm.att_heads, dm.att_dim, 16) * 4);
   if (dm.moe_r > 0) {
     const size_t rows = dm.moe_e > 0 ? (size_t)moe_group_max_rows((int)T * dm.moe_top, dm.moe_e) : T * (size_t)dm.moe_top;
-    b += al256(T * (size_t)std::max(64, up8(dm.moe_r)) * 4) + 2 * al256(T * (size_t)dm.moe_top * 4) + al256(T * (size_t)dm.moe_top * W * 4);
+    b += al256(T * (size_t)std::max(64, up8(dm.moe_r)) * 4) + 2 * al256(T * (size_t)dm.moe_top * 4) + al256(T * (size_t)dm.moe_top * W * 4) +
+         al256(dm.moe_h * 4);
     if (dm.moe_e > 0)
       b += al256(T * (size_t)dm.moe_top * 4) + al256(rows * 4) + al256(rows / 128 * 4) + 2 * al256(rows * W * 2) + al256(rows * dm.moe_f * 2) +
            al256((size_t)3 * dm.moe_e * 4);
@@ -406,7 +411,7 @@ int Engine::alloc_runtime_stack() {
     return r;
   };
   const size_t T = t_cap_, W = sd.width;
-  const StackDims dm = stack_dims(model_, cfg_.max_ctx);
+  const StackDims dm = stack_dims(model_, cfg_.max_ctx, t_cap_);
   const int n1 = dm.n1, n2 = dm.n2, q = dm.q, qa = dm.qa, cx = dm.cx, mo = dm.mo;
   {  // rotation frequencies of the attention layers (double precision, formed on the host)
     double* fq = (double*)take((size_t)std::max(dm.rope_half, 1) * 8);
@@ -443,6 +448,7 @@ int Engine::alloc_runtime_stack() {
     sk_.moe_ids = (int32_t*)take(T * (size_t)dm.moe_top * 4);
     sk_.moe_w = (float*)take(T * (size_t)dm.moe_top * 4);
     const size_t rows = dm.moe_e > 0 ? (size_t)moe_group_max_rows((int)T * dm.moe_top, dm.moe_e) : T * (size_t)dm.moe_top;
+    sk_.moe_h = (float*)take(dm.moe_h * 4);
     sk_.moe_y = (float*)take(T * (size_t)dm.moe_top * W * 4);  // per-item outputs of the GEMV path
     if (dm.moe_e > 0) {
       sk_.moe_rows = (int)rows;
@@ -865,8 +871,9 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
         SPAN(3, 2.0 * T * (l.top_k + 4) * W, moe_combine_rows(stream_, ff_in, k.moe_y16, k.moe_row_of, k.moe_w, l.top_k, out, T, W, add));
       }
     } else {
-      SPAN(5, 6.0 * items * F * W, moe_expert_rows(stream_, ff_in, ff_in16, w.w_gu, w.w_down, f32, k.moe_ids, l.top_k, E, F, W, k.moe_y, T, w.gu_packed,
+      SPAN(5, 6.0 * items * F * W, moe_expert_rows(stream_, ff_in, ff_in16, w.w_gu, w.w_down, f32, k.moe_ids, l.top_k, E, F, W, k.moe_h, k.moe_y, T, w.gu_packed,
                                                    eact, l.ff_limit));
+      launches_.fetch_add(1, std::memory_order_relaxed);  // two kernels behind one call
       SPAN(3, 4.0 * T * (l.top_k + 2) * W, moe_combine(stream_, ff_in, k.moe_y, k.moe_ids, k.moe_w, l.top_k, E, out, T, W, add));
     }
     return HB_OK;

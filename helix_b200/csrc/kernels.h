@@ -642,12 +642,12 @@ cudaError_t moe_router(cudaStream_t s, const float* x, const void* router, const
                        int32_t* ids, float* wts, int T, int sms, const RouteOpts& ro = RouteOpts());
 // bf16 form of gated_unit for the tensor-core path: gu and out are bf16, F and ldg multiples of eight
 cudaError_t gated_unit_b16(cudaStream_t s, const bf16* gu, long ldg, int act, bf16* out, int T, int F, float limit = 0.f);
-// One block per (token, choice): y[(t, k), :] = down_e(silu(gate_e x_t) * (up_e x_t)) for ids[t, k] = e < E (rows of choices
+// Few items, or the exact mode: y[(t, k), :] = down_e(silu(gate_e x_t) * (up_e x_t)) for ids[t, k] = e < E (rows of choices
 // that name an identity output are left alone).  x_b16 != null: the unit reads the bf16 copy of x and rounds its inner
 // activation to bf16, as the tensor-core path does.  w_gu: [E][2F][W] ([gate | up] rows), w_down: [E][W][F].
 cudaError_t moe_expert_rows(cudaStream_t s, const float* x, const bf16* x_b16, const void* w_gu, const void* w_down, bool f32,
-                            const int32_t* ids, int top_k, int E, int F, int W, float* y, int T, bool packed = false, int act = GLU_SILU,
-                            float limit = 0.f);
+                            const int32_t* ids, int top_k, int E, int F, int W, float* hbuf, float* y, int T, bool packed = false,
+                            int act = GLU_SILU, float limit = 0.f);  // hbuf: [T * top_k][F] inner activations; two launches
 // The same experts as grouped tensor-core products (bf16 mode): moe_group_rows sorts the (token, choice) items by expert into
 // a row buffer of moe_group_max_rows(items, E) rows whose per-expert segments start on multiples of 128 rows (row_of[item] =
 // its row or -1 for an identity output, src_of_row[row] = its token or -1, tile_group[row / 128] = the expert whose weights

@@ -234,6 +234,7 @@ __global__ void __launch_bounds__(kRouterWarps * 32) moe_router_small_kernel(con
     const WT* row = router + (size_t)r * W;
     float acc = 0.f;
     if (vec) {
+#pragma unroll 8
       for (int i = l * 4; i < W; i += 128) {
         const float4 xv = ld4(xr + i), wv = ld4(row + i);
         acc = fmaf(xv.x, wv.x, acc); acc = fmaf(xv.y, wv.y, acc); acc = fmaf(xv.z, wv.z, acc); acc = fmaf(xv.w, wv.w, acc);
@@ -290,45 +291,51 @@ __device__ __forceinline__ float warp_dot(const WT* __restrict__ wrow, const flo
 
 __device__ __forceinline__ float gelu_erf_(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
-// block per (token, choice).  act GLU_NONE_GELU: ungated units (w_gu: [E][F][W] up rows).  dynamic smem: x [Wp] + inner activation [F]
+// Experts of steps with few items, in two launches so that the weights of one expert are read by many blocks.  Blocks
+// (item, kExpRows rows): inner activations h[item][F] (act GLU_NONE_GELU: ungated units, w_gu: [E][F][W] up rows), then the
+// item's output rows y[item][W].  dynamic smem: the input vector.
+constexpr int kExpRows = 32;
 template <typename WT>
-__global__ void __launch_bounds__(256) moe_expert_rows_kernel(const float* __restrict__ x, const bf16* __restrict__ xb,
-                                                              const WT* __restrict__ w_gu, const WT* __restrict__ w_down,
-                                                              const int32_t* __restrict__ ids, int E, int F, int W,
-                                                              float* __restrict__ y, int packed, int act, float limit) {
-  extern __shared__ float sm[];
-  const int t = blockIdx.x;
-  const size_t item = (size_t)t * gridDim.y + blockIdx.y;  // (token, choice)
+__global__ void __launch_bounds__(256) moe_expert_up_kernel(const float* __restrict__ x, const bf16* __restrict__ xb, const WT* __restrict__ w_gu,
+                                                            const int32_t* __restrict__ ids, int top_k, int E, int F, int W,
+                                                            float* __restrict__ hbuf, int packed, int act, float limit) {
+  extern __shared__ float xs[];
+  const size_t item = blockIdx.x;  // (token, choice)
+  const size_t t = item / top_k;
   const int e = ids[item];
   if (e >= E) return;
-  float* xs = sm;
-  float* hs = sm + (W + 3) / 4 * 4;
-  for (int i = threadIdx.x; i < W; i += blockDim.x) xs[i] = xb ? __bfloat162float(xb[(size_t)t * W + i]) : x[(size_t)t * W + i];
+  for (int i = threadIdx.x; i < W; i += blockDim.x) xs[i] = xb ? __bfloat162float(xb[t * W + i]) : x[t * W + i];
   __syncthreads();
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
   const bool gated = act != GLU_NONE_GELU;
   const WT* gu = w_gu + (size_t)e * (gated ? 2 : 1) * F * W;
-  for (int f = w; f < F; f += nw) {
-    if (!gated) {
-      const float u = warp_dot<WT>(gu + (size_t)f * W, xs, W, l);
-      if (l == 0) {
-        const float v = gelu_erf_(u);
-        hs[f] = xb ? __bfloat162float(__float2bfloat16(v)) : v;
-      }
-      continue;
+  const int f1 = min(F, (int)(blockIdx.y + 1) * kExpRows);
+  for (int f = blockIdx.y * kExpRows + w; f < f1; f += nw) {
+    float v;
+    if (gated) {
+      const size_t gr = packed ? (size_t)(f >> 7) * 256 + (f & 127) : (size_t)f, ur = packed ? gr + 128 : (size_t)F + f;
+      const float g = warp_dot<WT>(gu + gr * W, xs, W, l);
+      const float u = warp_dot<WT>(gu + ur * W, xs, W, l);
+      v = glu_pair(g, u, act, limit);
+    } else {
+      v = gelu_erf_(warp_dot<WT>(gu + (size_t)f * W, xs, W, l));
     }
-    const size_t gr = packed ? (size_t)(f >> 7) * 256 + (f & 127) : (size_t)f, ur = packed ? gr + 128 : (size_t)F + f;
-    const float g = warp_dot<WT>(gu + gr * W, xs, W, l);
-    const float u = warp_dot<WT>(gu + ur * W, xs, W, l);
-    if (l == 0) {
-      float v = glu_pair(g, u, act, limit);
-      if (xb) v = __bfloat162float(__float2bfloat16(v));
-      hs[f] = v;
-    }
+    if (l == 0) hbuf[item * F + f] = xb ? __bfloat162float(__float2bfloat16(v)) : v;
   }
+}
+template <typename WT>
+__global__ void __launch_bounds__(256) moe_expert_down_kernel(const float* __restrict__ hbuf, const WT* __restrict__ w_down,
+                                                              const int32_t* __restrict__ ids, int E, int F, int W, float* __restrict__ y) {
+  extern __shared__ float hs[];
+  const size_t item = blockIdx.x;
+  const int e = ids[item];
+  if (e >= E) return;
+  for (int i = threadIdx.x; i < F; i += blockDim.x) hs[i] = hbuf[item * F + i];
   __syncthreads();
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
   const WT* dn = w_down + (size_t)e * W * F;
-  for (int c = w; c < W; c += nw) {
+  const int c1 = min(W, (int)(blockIdx.y + 1) * kExpRows);
+  for (int c = blockIdx.y * kExpRows + w; c < c1; c += nw) {
     const float v = warp_dot<WT>(dn + (size_t)c * F, hs, F, l);
     if (l == 0) y[item * W + c] = v;
   }
@@ -337,7 +344,7 @@ __global__ void __launch_bounds__(256) moe_expert_rows_kernel(const float* __res
 __global__ void moe_combine_kernel(const float* __restrict__ x, const float* __restrict__ y, const int32_t* __restrict__ ids,
                                    const float* __restrict__ wts, int top_k, int E, float* out, int W, const float* add) {
   const int t = blockIdx.x;
-  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < W; c += gridDim.y * blockDim.x) {
     float acc = add ? add[(size_t)t * W + c] : 0.f;
     for (int k = 0; k < top_k; ++k) {
       const size_t item = (size_t)t * top_k + k;
@@ -448,7 +455,7 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const bf16* __restrict_
 __global__ void moe_combine_rows_kernel(const float* __restrict__ x, const bf16* __restrict__ y, const int32_t* __restrict__ row_of,
                                         const float* __restrict__ wts, int top_k, float* out, int W, const float* add) {
   const int t = blockIdx.x;
-  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < W; c += gridDim.y * blockDim.x) {
     float acc = add ? add[(size_t)t * W + c] : 0.f;
     for (int k = 0; k < top_k; ++k) {
       const size_t item = (size_t)t * top_k + k;
@@ -491,7 +498,7 @@ cudaError_t moe_gather_rows(cudaStream_t s, const bf16* x16, int W, const int32_
 cudaError_t moe_combine_rows(cudaStream_t s, const float* x, const bf16* y, const int32_t* row_of, const float* wts, int top_k,
                              float* out, int T, int W, const float* add) {
   if (T <= 0) return cudaSuccess;
-  moe_combine_rows_kernel<<<T, 256, 0, s>>>(x, y, row_of, wts, top_k, out, W, add);
+  moe_combine_rows_kernel<<<dim3(T, T <= 256 ? (W + 255) / 256 : 1), 256, 0, s>>>(x, y, row_of, wts, top_k, out, W, add);
   return cudaGetLastError();
 }
 
@@ -500,8 +507,10 @@ cudaError_t stack_moe_init() {
   const int big = 200 * 1024;
   if ((e = cudaFuncSetAttribute(moe_router_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)) != cudaSuccess) return e;
   if ((e = cudaFuncSetAttribute(moe_router_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)) != cudaSuccess) return e;
-  if ((e = cudaFuncSetAttribute(moe_expert_rows_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)) != cudaSuccess) return e;
-  if ((e = cudaFuncSetAttribute(moe_expert_rows_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)) != cudaSuccess) return e;
+  if ((e = cudaFuncSetAttribute(moe_expert_up_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)) != cudaSuccess) return e;
+  if ((e = cudaFuncSetAttribute(moe_expert_up_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)) != cudaSuccess) return e;
+  if ((e = cudaFuncSetAttribute(moe_expert_down_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)) != cudaSuccess) return e;
+  if ((e = cudaFuncSetAttribute(moe_expert_down_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)) != cudaSuccess) return e;
   return cudaSuccess;
 }
 
@@ -556,20 +565,26 @@ cudaError_t gated_unit_b16(cudaStream_t s, const bf16* gu, long ldg, int act, bf
 }
 
 cudaError_t moe_expert_rows(cudaStream_t s, const float* x, const bf16* xb, const void* w_gu, const void* w_down, bool f32,
-                            const int32_t* ids, int top_k, int E, int F, int W, float* y, int T, bool packed, int act, float limit) {
+                            const int32_t* ids, int top_k, int E, int F, int W, float* hbuf, float* y, int T, bool packed, int act,
+                            float limit) {
   if (T <= 0) return cudaSuccess;
-  const size_t smem = ((size_t)(W + 3) / 4 * 4 + F) * 4;
-  if (smem > 200 * 1024) return cudaErrorInvalidValue;
-  dim3 grid(T, top_k);
-  if (f32) moe_expert_rows_kernel<float><<<grid, 256, smem, s>>>(x, xb, (const float*)w_gu, (const float*)w_down, ids, E, F, W, y, packed ? 1 : 0, act, limit);
-  else moe_expert_rows_kernel<bf16><<<grid, 256, smem, s>>>(x, xb, (const bf16*)w_gu, (const bf16*)w_down, ids, E, F, W, y, packed ? 1 : 0, act, limit);
+  const size_t smem_x = (size_t)W * 4, smem_h = (size_t)F * 4;
+  if (smem_x > 200 * 1024 || smem_h > 200 * 1024) return cudaErrorInvalidValue;
+  const dim3 g1(T * top_k, (F + kExpRows - 1) / kExpRows), g2(T * top_k, (W + kExpRows - 1) / kExpRows);
+  if (f32) {
+    moe_expert_up_kernel<float><<<g1, 256, smem_x, s>>>(x, xb, (const float*)w_gu, ids, top_k, E, F, W, hbuf, packed ? 1 : 0, act, limit);
+    moe_expert_down_kernel<float><<<g2, 256, smem_h, s>>>(hbuf, (const float*)w_down, ids, E, F, W, y);
+  } else {
+    moe_expert_up_kernel<bf16><<<g1, 256, smem_x, s>>>(x, xb, (const bf16*)w_gu, ids, top_k, E, F, W, hbuf, packed ? 1 : 0, act, limit);
+    moe_expert_down_kernel<bf16><<<g2, 256, smem_h, s>>>(hbuf, (const bf16*)w_down, ids, E, F, W, y);
+  }
   return cudaGetLastError();
 }
 
 cudaError_t moe_combine(cudaStream_t s, const float* x, const float* y, const int32_t* ids, const float* wts, int top_k, int E, float* out,
                         int T, int W, const float* add) {
   if (T <= 0) return cudaSuccess;
-  moe_combine_kernel<<<T, 256, 0, s>>>(x, y, ids, wts, top_k, E, out, W, add);
+  moe_combine_kernel<<<dim3(T, T <= 256 ? (W + 255) / 256 : 1), 256, 0, s>>>(x, y, ids, wts, top_k, E, out, W, add);
   return cudaGetLastError();
 }
 

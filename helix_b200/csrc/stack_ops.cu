@@ -69,7 +69,7 @@ __global__ void embed_rows_kernel(const int32_t* __restrict__ tokens, const WT* 
                                   bf16* __restrict__ xb, int W, float scale) {
   const int t = blockIdx.x;
   const WT* src = table + (size_t)tokens[t] * W;
-  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < W; i += gridDim.y * blockDim.x) {
     const float v = ldf<WT>(src, i) * scale;
     x[(size_t)t * W + i] = v;
     if (xb) xb[(size_t)t * W + i] = __float2bfloat16(v);
@@ -888,8 +888,9 @@ cudaError_t tanh_norm_step(cudaStream_t s, const float* x, const int32_t* row_in
 
 cudaError_t embed_rows_f32(cudaStream_t s, const int32_t* tokens, const void* table, bool f32, float* x, bf16* xb, int T, int W, float scale) {
   if (T <= 0) return cudaSuccess;
-  if (f32) embed_rows_kernel<float><<<T, 128, 0, s>>>(tokens, (const float*)table, x, xb, W, scale);
-  else embed_rows_kernel<bf16><<<T, 128, 0, s>>>(tokens, (const bf16*)table, x, xb, W, scale);
+  const dim3 grid(T, T <= 256 ? (W + 127) / 128 : 1);
+  if (f32) embed_rows_kernel<float><<<grid, 128, 0, s>>>(tokens, (const float*)table, x, xb, W, scale);
+  else embed_rows_kernel<bf16><<<grid, 128, 0, s>>>(tokens, (const bf16*)table, x, xb, W, scale);
   return KERR();
 }
 
