@@ -121,7 +121,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     int max_pages, int Hkv, int chunk, int sink, const float* __restrict__ head_gate, int ldg,
                     int window, float cap_in, float cap_out, const bf16* __restrict__ sink_w,
                     const __grid_constant__ CUtensorMap map_qr, const __grid_constant__ CUtensorMap map_kr,
-                    const __grid_constant__ AttnRuns runs, int vdim, const float* __restrict__ entry_gate) {
+                    const __grid_constant__ AttnRuns runs, int vdim) {
   using C = ACfg<DK, DV, SRC>;
   constexpr bool PAGED = SRC == KV_PAGED, EXPANDED = SRC == KV_EXPANDED;
   constexpr int KST = C::STAGES;
@@ -561,7 +561,6 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       if (!staged) {
         const int dv = EXPANDED ? vdim : DV;
         bf16* orow = out + (size_t)(it.seq0 + qrow) * ldo + it.h * dv;
-        const float* grow = EXPANDED && entry_gate ? entry_gate + (size_t)(it.seq0 + qrow) * ldg + it.h * dv : nullptr;
 #pragma unroll
         for (int c = 0; c < DV / 32; ++c) {
           uint32_t o[32];
@@ -571,16 +570,6 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
               if (EXPANDED && c * 32 + i * 8 >= dv) break;  // vdim is a multiple of 8
-              if constexpr (EXPANDED) {
-                if (grow != nullptr) {  // one gate per output entry
-                  const float4 ga = *reinterpret_cast<const float4*>(grow + c * 32 + i * 8);
-                  const float4 gb = *reinterpret_cast<const float4*>(grow + c * 32 + i * 8 + 4);
-                  const float gg[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
-#pragma unroll
-                  for (int e = 0; e < 8; ++e)
-                    o[8 * i + e] = __float_as_uint(__fdividef(__uint_as_float(o[8 * i + e]), 1.f + __expf(-gg[e])));
-                }
-              }
               uint4 w;
               w.x = pack_bf16x2(__uint_as_float(o[8 * i + 0]) * inv_l, __uint_as_float(o[8 * i + 1]) * inv_l);
               w.y = pack_bf16x2(__uint_as_float(o[8 * i + 2]) * inv_l, __uint_as_float(o[8 * i + 3]) * inv_l);
@@ -641,7 +630,7 @@ cudaError_t launch_p(cudaStream_t stream, const AttnPrefillArgs& a) {
                                             scale_log2, max_q_pairs, a.kv_lens, a.page_table, a.max_pages, a.Hkv,
                                             paged_only(a.block_mask, PAGED), a.unit_sink, a.head_gate, a.ldg,
                                             paged_only(a.window, PAGED), a.softcap > 0.f ? a.scale / a.softcap : 0.f,
-                                            a.softcap > 0.f ? a.softcap * 1.4426950408889634f : 0.f, a.sink, mq, mk, AttnRuns{}, D, nullptr);
+                                            a.softcap > 0.f ? a.softcap * 1.4426950408889634f : 0.f, a.sink, mq, mk, AttnRuns{}, D);
   return cudaGetLastError();
 }
 
@@ -667,7 +656,7 @@ cudaError_t launch_expanded(cudaStream_t stream, const AttnExpandedArgs& a) {
   const int grid = (int)std::min<long long>(items, effective_sms(num_sms));
   kern<<<grid, kThreads, C::SMEM, stream>>>(mq, mk, mv, mq, a.out, a.ldo, nullptr, a.runs.n, a.H, 1, 1, a.scale * 1.4426950408889634f,
                                             max_q_pairs, nullptr, nullptr, 0, a.H, 0, 0, a.head_gate, a.ldg, a.window, 0.f, 0.f, a.sink,
-                                            mqr, mkr, a.runs, a.vdim, a.entry_gate);
+                                            mqr, mkr, a.runs, a.vdim);
   return cudaGetLastError();
 }
 
@@ -765,7 +754,6 @@ cudaError_t attn_expanded(cudaStream_t stream, const AttnExpandedArgs& a) {
   if (a.runs.n <= 0) return cudaSuccess;
   if (!attn_expanded_ok(a.nope, a.rot, a.vdim) || a.H <= 0 || a.T <= 0 || a.rows <= 0 || a.runs.n > AttnRuns::kMax || a.window < 0) return cudaErrorInvalidValue;
   if (a.ldq % 8 || a.ldkv % 8 || a.ldkr % 8 || a.ldo % 8) return cudaErrorInvalidValue;
-  if (a.entry_gate && (a.ldg % 4 || ((uintptr_t)a.entry_gate & 15))) return cudaErrorInvalidValue;
   const bool wide = a.nope > 64;
   if (a.vdim <= 64) return wide ? launch_expanded<192, 64>(stream, a) : launch_expanded<128, 64>(stream, a);
   return wide ? launch_expanded<192, 128>(stream, a) : launch_expanded<128, 128>(stream, a);

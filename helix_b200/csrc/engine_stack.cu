@@ -652,7 +652,7 @@ int Engine::latent_attention_tc(int T, const StepLayout& L, const hb_layer_desc&
     ea.k_rot = k.lat_kr; ea.ldkr = Dr;
     ea.out = k.mo16; ea.ldo = H * Dv;
     ea.T = T; ea.rows = rows; ea.H = H; ea.nope = Dk; ea.rot = Dr; ea.vdim = Dv; ea.window = window; ea.scale = l.scale;
-    if (head_gate) ea.head_gate = k.p1 + w.off_g; else ea.entry_gate = k.p1 + w.off_g;
+    ea.head_gate = head_gate ? k.p1 + w.off_g : nullptr;
     ea.ldg = k.ld1; ea.sink = (const bf16*)w.sink;
     ar.n = lr.n;
     ea.runs = ar;
@@ -676,6 +676,25 @@ int Engine::latent_attention_tc(int T, const StepLayout& L, const hb_layer_desc&
   }
   int rc = launch_group();
   if (rc != HB_OK) return rc;
+  if (!head_gate) {  // a gate per entry: neighbouring long portions in one pass
+    int g0 = 0, g1 = 0;
+    auto gate = [&]() -> int {
+      if (g1 > g0)
+        SPAN(3, 8.0 * (g1 - g0) * H * Dv, gate_rows_b16(stream_, k.mo16 + (size_t)g0 * H * Dv, k.p1 + (size_t)g0 * k.ld1 + w.off_g, k.ld1, g1 - g0, H * Dv));
+      return HB_OK;
+    };
+    for (const StepEntry& en : step_entries_) {
+      if (en.n < kAttDenseMin) continue;
+      if (en.t0 != g1) {
+        rc = gate();
+        if (rc != HB_OK) return rc;
+        g0 = en.t0;
+      }
+      g1 = en.t0 + en.n;
+    }
+    rc = gate();
+    if (rc != HB_OK) return rc;
+  }
   // ---- single tokens and short portions, in blocks of up to 128 tokens: q_h^T W_uk,h per head as one grouped product (the head's
   // weights per 128-row m tile), attention over the cached rows, values out of the weighted latents, gate
   bool first = true;

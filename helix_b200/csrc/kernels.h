@@ -154,8 +154,7 @@ struct AttnExpandedArgs {
   bf16* out; int ldo;                // [T, H * vdim]
   int T, rows, H, nope, rot, vdim, window;  // window 0: causal
   float scale;
-  const float* head_gate = nullptr;  // optional sigmoid gates, row stride ldg: one per head, or one per output entry
-  const float* entry_gate = nullptr;
+  const float* head_gate = nullptr;  // optional [T][>= H] fp32, row stride ldg: head h leaves times sigmoid(head_gate[t][h])
   int ldg = 0;
   const bf16* sink = nullptr;        // [H] learned logits whose exponential joins the denominator
   AttnRuns runs;
@@ -441,6 +440,8 @@ cudaError_t latent_softmax(cudaStream_t s, const float* S, bf16* P, int ld, int 
                            float scale, const bf16* sink);
 // dst[h][r][d] = src[h][d][r] (bf16): the key up-projection per head, transposed once at load time
 cudaError_t transpose_heads_bf16(cudaStream_t s, const bf16* src, bf16* dst, int H, int Dk, int R);
+// o[t, e] *= sigmoid(g[t, e]), e < N, on bf16 rows of N entries (N a multiple of 8, ldg of 4)
+cudaError_t gate_rows_b16(cudaStream_t s, bf16* o, const float* g, long ldg, int T, int N);
 // f32 -> bf16 copy of a [T, N] block (row strides lds / ldd)
 cudaError_t to_bf16_rows(cudaStream_t s, const float* src, long lds, bf16* dst, long ldd, int T, int N);
 

@@ -293,6 +293,22 @@ __global__ void latent_gate_kernel(const float* __restrict__ o, long o_ts, long 
   }
 }
 
+__global__ void __launch_bounds__(256) gate_rows_b16_kernel(bf16* __restrict__ o, const float* __restrict__ g, long ldg, int N) {
+  const size_t t = blockIdx.y;
+  const int j = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  if (j >= N) return;
+  uint4 u = *reinterpret_cast<uint4*>(o + t * N + j);
+  const float4 a = *reinterpret_cast<const float4*>(g + t * ldg + j), b = *reinterpret_cast<const float4*>(g + t * ldg + j + 4);
+  const float gg[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+  __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float2 v = __bfloat1622float2(p[e]);
+    p[e] = __floats2bfloat162_rn(v.x * sigmoidf_(gg[2 * e]), v.y * sigmoidf_(gg[2 * e + 1]));
+  }
+  *reinterpret_cast<uint4*>(o + t * N + j) = u;
+}
+
 // VEC = 4: N, both strides and both bases are multiples of four elements (16-byte loads, 8-byte stores)
 template <int VEC>
 __global__ void to_bf16_kernel(const float* __restrict__ src, long lds, bf16* __restrict__ dst, long ldd, int N) {
@@ -955,6 +971,12 @@ cudaError_t latent_out_gate(cudaStream_t s, const float* o, long o_ts, long o_hs
   dim3 grid(((vec ? N / 4 : N) + 255) / 256, T);
   if (vec) latent_gate_kernel<4><<<grid, 256, 0, s>>>(o, o_ts, o_hs, g, ldg, per_head ? 1 : 0, out, outb, H, Dv);
   else latent_gate_kernel<1><<<grid, 256, 0, s>>>(o, o_ts, o_hs, g, ldg, per_head ? 1 : 0, out, outb, H, Dv);
+  return KERR();
+}
+cudaError_t gate_rows_b16(cudaStream_t s, bf16* o, const float* g, long ldg, int T, int N) {
+  if (T <= 0) return cudaSuccess;
+  if (N % 8 || ldg % 4 || ((uintptr_t)o & 15) || ((uintptr_t)g & 15)) return cudaErrorInvalidValue;
+  gate_rows_b16_kernel<<<dim3((N / 8 + 255) / 256, T), 256, 0, s>>>(o, g, ldg, N);
   return KERR();
 }
 cudaError_t to_bf16_rows(cudaStream_t s, const float* src, long lds, bf16* dst, long ldd, int T, int N) {
