@@ -7,7 +7,8 @@
 //
 // Grid (splits, head groups, tokens).  A kv tile is one 64-position page; its 64-column sub-tiles travel in pairs through one
 // ring (16 KB slots) and the rotated part through a second ring, so loads of the next tiles overlap the products of this one.
-//   warp 0 : TMA producer      warp 1 : MMA issuer, program order S(j) S(j + 1) PV(j) PV(j + 1)
+//   warp 0 : TMA producer      warp 1 / warp 6 : issuers of the S / PV products (one warp for both was the bottleneck: an issue
+//                takes about 50 cycles whatever the product's size, and a tile needs 36 + 16 of them)
 //   warps 2..5 : softmax.  The S^T tile of an M = 64 product sits in lanes 0..15 of every 32-lane quadrant; the running maximum is
 //                only reduced when some score passes it by more than 2^8 (the first tile, rarely later), sums stay per thread.
 // A second kernel merges the splits.  Further kernels here move rows into the layouts of the per-head products.
@@ -23,7 +24,7 @@
 namespace hb {
 namespace {
 
-constexpr int kThreads = 192;
+constexpr int kThreads = 224;
 constexpr int PAGE = 64;
 constexpr int kSub = PAGE * 128;    // one 64-column sub-tile of a page (bf16)
 constexpr int kPair = 2 * kSub;
@@ -61,7 +62,7 @@ __device__ __forceinline__ void tmem_ld_cols(uint32_t taddr, uint32_t (&r)[NQ]) 
 struct Rings { int cs, rs; };  // slots of the latent-pair ring / of the rotated-part ring
 
 template <int NQ>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, NQ == 16 ? 2 : 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_constant__ CUtensorMap map_r,
                      const __grid_constant__ CUtensorMap map_ql, const __grid_constant__ CUtensorMap map_qr,
                      const __grid_constant__ LatentDecodeArgs a, Rings rings, int num_splits) {
@@ -165,12 +166,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
   } else if (warp == 1) {
     const bool elected = elect_one_sync();
     constexpr uint32_t idesc_s = umma_idesc_bf16(PAGE, NQ, 0, 0);
-    constexpr uint32_t idesc_o = umma_idesc_bf16(128, NQ, 1, 0);
     // descriptors are a base per operand plus offsets in 16-byte units (the address field never carries)
     const uint64_t kdesc0 = umma_desc_kmajor_sw128(smem_u32(ring_c)), rdesc0 = umma_desc_kmajor_sw128(smem_u32(ring_r));
-    const uint64_t qdesc0 = umma_desc_kmajor_sw128(smem_u32(sQ)), pdesc0 = umma_desc_kmajor_sw128(smem_u32(sP));
-    const uint64_t vdesc0 = umma_desc_mnmajor_sw128(smem_u32(ring_c), kSub, 1024);
-    int cs = 0, rs = 0, vs = 0;  // ring slots of the next S pair / rotated part / PV pair
+    const uint64_t qdesc0 = umma_desc_kmajor_sw128(smem_u32(sQ));
+    int cs = 0, rs = 0;  // ring slots of the next latent pair / rotated part
     uint32_t cph = 0, rph = 0;
     auto issue_s = [&](int j) {
       mbar_wait(&s_empty[j & 1], ((j >> 1) & 1) ^ 1);
@@ -203,29 +202,30 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_con
       }
       if (++rs == RS) { rs = 0; rph ^= 1; }
     };
-    auto issue_pv = [&](int j) {
-      mbar_wait(&p_full[j & 1], (j >> 1) & 1);
-      tc_fence_after();
-      for (int p = 0; p < np; ++p) {
-        if (elected) {
-#pragma unroll
-          for (int k = 0; k < 4; ++k)
-            umma_f16_ss(tmem_O + p * NQ, vdesc0 + (uint64_t)(vs * (kPair >> 4)) + k * (16 * 128 >> 4),
-                        pdesc0 + (uint64_t)((j & 1) * (NQ * 128 >> 4)) + k * 2, idesc_o, k != 0 ? 1u : (j != 0 ? 1u : 0u));
-          umma_commit(&c_empty[vs]);
-        }
-        if (++vs == CS) vs = 0;
-      }
-      if (elected) umma_commit(&pv_done[j & 1]);
-    };
-    // two tiles at a time: while the slots of the first are refilled, the tensor pipe works on the second
     mbar_wait(q_ready, 0);
     tc_fence_after();
-    for (int j = 0; j < n_tiles; j += 2) {
-      issue_s(j);
-      if (j + 1 < n_tiles) issue_s(j + 1);
-      issue_pv(j);
-      if (j + 1 < n_tiles) issue_pv(j + 1);
+    for (int j = 0; j < n_tiles; ++j) issue_s(j);
+  } else if (warp == 6) {
+    const bool elected = elect_one_sync();
+    constexpr uint32_t idesc_o = umma_idesc_bf16(128, NQ, 1, 0);
+    const uint64_t pdesc0 = umma_desc_kmajor_sw128(smem_u32(sP)), vdesc0 = umma_desc_mnmajor_sw128(smem_u32(ring_c), kSub, 1024);
+    int vs = 0;
+    uint32_t vph = 0;
+    for (int j = 0; j < n_tiles; ++j) {
+      mbar_wait(&p_full[j & 1], (j >> 1) & 1);
+      const uint64_t pd = pdesc0 + (uint64_t)((j & 1) * (NQ * 128 >> 4));
+      for (int p = 0; p < np; ++p) {
+        mbar_wait(&c_full[vs], vph);  // landed long ago (S(j) read it): the wait orders this warp's reads behind the copy
+        tc_fence_after();
+        if (elected) {
+          const uint64_t vd = vdesc0 + (uint64_t)(vs * (kPair >> 4));
+#pragma unroll
+          for (int k = 0; k < 4; ++k) umma_f16_ss(tmem_O + p * NQ, vd + k * (16 * 128 >> 4), pd + k * 2, idesc_o, k != 0 ? 1u : (j != 0 ? 1u : 0u));
+          umma_commit(&c_empty[vs]);
+        }
+        if (++vs == CS) { vs = 0; vph ^= 1; }
+      }
+      if (elected) umma_commit(&pv_done[j & 1]);
     }
   } else {
     const int qd = warp & 3;
