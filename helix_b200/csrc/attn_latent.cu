@@ -62,7 +62,7 @@ __device__ __forceinline__ void tmem_ld_cols(uint32_t taddr, uint32_t (&r)[NQ]) 
 struct Rings { int cs, rs; };  // slots of the latent-pair ring / of the rotated-part ring
 
 template <int NQ>
-__global__ void __launch_bounds__(kThreads, NQ == 16 ? 2 : 1)
+__global__ void __launch_bounds__(kThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_constant__ CUtensorMap map_r,
                      const __grid_constant__ CUtensorMap map_ql, const __grid_constant__ CUtensorMap map_qr,
                      const __grid_constant__ LatentDecodeArgs a, Rings rings, int num_splits) {
@@ -420,7 +420,7 @@ __global__ void __launch_bounds__(128) latent_q_heads_kernel(const bf16* __restr
 template <int NQ>
 bool pick_rings(int nc, int np, Rings* rings, size_t* smem) {
   const size_t fixed = (size_t)(nc + 1) * NQ * 128 + 2 * NQ * 128 + 5 * NQ * 4 + (2 * kMaxC + 2 * kMaxR + 9) * 8 + 16 + 1024;
-  const size_t total = np <= 2 && NQ == 16 ? 113 * 1024 : 227 * 1024;  // narrow rows: two blocks per SM
+  const size_t total = 227 * 1024;
   if (fixed >= total) return false;
   const size_t room = total - fixed, tile = (size_t)np * kPair + kSub;
   // about as many rotated parts as tiles of latents; at least two tiles of both (S of the next tile is issued while this tile's

@@ -189,7 +189,11 @@ static size_t stack_skinny_floats(const Model& m) {
 constexpr int kAttDenseMin = 64;
 // Latent layers on the tensor cores: bf16 mode and head / latent sizes that both kernels take (attn_expanded, latent_decode)
 static bool latent_tc_ok(const Model& m, const hb_layer_desc& l) {
-  static const bool off = [] { const char* e = getenv("HB_STACK_LATENT_TC"); return e && atoi(e) == 0; }();
+  static const bool off = [] {
+    const char* e = getenv("HB_STACK_LATENT_TC");
+    const char* s = getenv("HB_STACK_SIMT");
+    return (e && atoi(e) == 0) || (s && atoi(s) != 0);
+  }();
   const int W = m.sd.width, o = l.heads * l.vdim;
   return !off && !m.sd.compute_f32 && l.mixer == HB_MIXER_LATENT && attn_expanded_ok(l.dim, l.rot_dim, l.vdim) &&
          latent_decode_ok(l.dim, l.kv_rank, l.rot_dim) && W % 4 == 0 && W >= 64 && o % 8 == 0 && o >= 64 && l.window > 0;
@@ -1126,7 +1130,7 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
       const int R = l.kv_rank, Dr = l.rot_dim, Q = l.q_rank;
       uint8_t* plane = (uint8_t*)kv_ + plane_off_[w.cache_plane];
       const bool head_gate = (l.attn_flags & HB_ATTN_HEAD_GATE) != 0;
-      const bool tc = latent_tc_ok(model_, l) && k.lat_kv && page_ == 64 && stack_tc(W, H * Dv, H * Dv, W);
+      const bool tc = latent_tc_ok(model_, l);
       // tokens that attend over the latent rows themselves: runs of neighbouring entries below kAttDenseMin tokens
       std::vector<std::pair<int, int>> runs;
       if (tc)
