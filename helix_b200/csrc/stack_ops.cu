@@ -582,199 +582,199 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(LatentAttnArgs
     l_run[hh] = a.sink ? 1.f : 0.f;
   }
   for (int kb = 0; kb < n_all; kb += KB) {
-  const int n = min(KB, n_all - kb), j0 = first + kb;
-  const bool last_block = kb + KB >= n_all;
-  float inv[HG], fac[HG];
-  __syncthreads();  // the previous block's scores and rows have been read
-  for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
-    const int j = j0 + jj;
-    rowoff[jj] = pt[j / a.page_size] * a.page_size + j % a.page_size;
-  }
-  __syncthreads();
-  if (sizeof(CT) == 2 && (D & 7) == 0) {
-    // bf16 rows that start on 16-byte boundaries: two keys per iteration, their loads issued together
-    for (int jj = w; jj < n; jj += 2 * nw) {
-      const int jb = jj + nw;
-      const bool two = jb < n;
-      const bf16* ra = reinterpret_cast<const bf16*>(cache) + (size_t)rowoff[jj] * D;
-      const bf16* rb = reinterpret_cast<const bf16*>(cache) + (size_t)rowoff[two ? jb : jj] * D;
-      float sa[HG] = {}, sb[HG] = {};
-      for (int i = l * 8; i < D; i += 256) {
-        const uint4 ua = *reinterpret_cast<const uint4*>(ra + i), ub = *reinterpret_cast<const uint4*>(rb + i);
-        const __nv_bfloat162* pa = reinterpret_cast<const __nv_bfloat162*>(&ua);
-        const __nv_bfloat162* pb = reinterpret_cast<const __nv_bfloat162*>(&ub);
+    const int n = min(KB, n_all - kb), j0 = first + kb;
+    const bool last_block = kb + KB >= n_all;
+    float inv[HG], fac[HG];
+    __syncthreads();  // the previous block's scores and rows have been read
+    for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
+      const int j = j0 + jj;
+      rowoff[jj] = pt[j / a.page_size] * a.page_size + j % a.page_size;
+    }
+    __syncthreads();
+    if (sizeof(CT) == 2 && (D & 7) == 0) {
+      // bf16 rows that start on 16-byte boundaries: two keys per iteration, their loads issued together
+      for (int jj = w; jj < n; jj += 2 * nw) {
+        const int jb = jj + nw;
+        const bool two = jb < n;
+        const bf16* ra = reinterpret_cast<const bf16*>(cache) + (size_t)rowoff[jj] * D;
+        const bf16* rb = reinterpret_cast<const bf16*>(cache) + (size_t)rowoff[two ? jb : jj] * D;
+        float sa[HG] = {}, sb[HG] = {};
+        for (int i = l * 8; i < D; i += 256) {
+          const uint4 ua = *reinterpret_cast<const uint4*>(ra + i), ub = *reinterpret_cast<const uint4*>(rb + i);
+          const __nv_bfloat162* pa = reinterpret_cast<const __nv_bfloat162*>(&ua);
+          const __nv_bfloat162* pb = reinterpret_cast<const __nv_bfloat162*>(&ub);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float2 fa = __bfloat1622float2(pa[e]), fb = __bfloat1622float2(pb[e]);
+          for (int e = 0; e < 4; ++e) {
+            const float2 fa = __bfloat1622float2(pa[e]), fb = __bfloat1622float2(pb[e]);
+#pragma unroll
+            for (int hh = 0; hh < HG; ++hh) {
+              const float2 q = *reinterpret_cast<const float2*>(qs + hh * Dp + i + 2 * e);
+              sa[hh] = fmaf(q.x, fa.x, sa[hh]); sa[hh] = fmaf(q.y, fa.y, sa[hh]);
+              sb[hh] = fmaf(q.x, fb.x, sb[hh]); sb[hh] = fmaf(q.y, fb.y, sb[hh]);
+            }
+          }
+        }
+#pragma unroll
+        for (int hh = 0; hh < HG; ++hh) {
+          sa[hh] = warp_sum(sa[hh]);
+          sb[hh] = warp_sum(sb[hh]);
+        }
+        if (l == 0) {
 #pragma unroll
           for (int hh = 0; hh < HG; ++hh) {
-            const float2 q = *reinterpret_cast<const float2*>(qs + hh * Dp + i + 2 * e);
-            sa[hh] = fmaf(q.x, fa.x, sa[hh]); sa[hh] = fmaf(q.y, fa.y, sa[hh]);
-            sb[hh] = fmaf(q.x, fb.x, sb[hh]); sb[hh] = fmaf(q.y, fb.y, sb[hh]);
+            sc[jj * HG + hh] = sa[hh] * a.scale;
+            if (two) sc[jb * HG + hh] = sb[hh] * a.scale;
           }
         }
       }
+    }
+    for (int jj = (sizeof(CT) == 2 && (D & 7) == 0) ? n : w; jj < n; jj += nw) {  // rows read element by element
+      const CT* row = cache + (size_t)rowoff[jj] * D;
+      float s[HG] = {};
+      for (int i = l; i < D; i += 32) {
+        const float kv = ldf<CT>(row, i);
 #pragma unroll
-      for (int hh = 0; hh < HG; ++hh) {
-        sa[hh] = warp_sum(sa[hh]);
-        sb[hh] = warp_sum(sb[hh]);
+        for (int hh = 0; hh < HG; ++hh) s[hh] = fmaf(qs[hh * Dp + i], kv, s[hh]);
       }
+#pragma unroll
+      for (int hh = 0; hh < HG; ++hh) s[hh] = warp_sum(s[hh]);
       if (l == 0) {
 #pragma unroll
-        for (int hh = 0; hh < HG; ++hh) {
-          sc[jj * HG + hh] = sa[hh] * a.scale;
-          if (two) sc[jb * HG + hh] = sb[hh] * a.scale;
-        }
+        for (int hh = 0; hh < HG; ++hh) sc[jj * HG + hh] = s[hh] * a.scale;
       }
     }
-  }
-  for (int jj = (sizeof(CT) == 2 && (D & 7) == 0) ? n : w; jj < n; jj += nw) {  // rows read element by element
-    const CT* row = cache + (size_t)rowoff[jj] * D;
-    float s[HG] = {};
-    for (int i = l; i < D; i += 32) {
-      const float kv = ldf<CT>(row, i);
+    __syncthreads();
+    // fp32 softmax; the HG heads share each block reduction
+    float mx[HG];
 #pragma unroll
-      for (int hh = 0; hh < HG; ++hh) s[hh] = fmaf(qs[hh * Dp + i], kv, s[hh]);
+    for (int hh = 0; hh < HG; ++hh) mx[hh] = m_run[hh];
+    for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
+      const float4 v = *reinterpret_cast<const float4*>(sc + jj * HG);
+      mx[0] = fmaxf(mx[0], v.x); mx[1] = fmaxf(mx[1], v.y); mx[2] = fmaxf(mx[2], v.z); mx[3] = fmaxf(mx[3], v.w);
     }
 #pragma unroll
-    for (int hh = 0; hh < HG; ++hh) s[hh] = warp_sum(s[hh]);
+    for (int hh = 0; hh < HG; ++hh) mx[hh] = warp_max(mx[hh]);
+    __syncthreads();
     if (l == 0) {
 #pragma unroll
-      for (int hh = 0; hh < HG; ++hh) sc[jj * HG + hh] = s[hh] * a.scale;
+      for (int hh = 0; hh < HG; ++hh) red[w * HG + hh] = mx[hh];
     }
-  }
-  __syncthreads();
-  // fp32 softmax; the HG heads share each block reduction
-  float mx[HG];
+    __syncthreads();
 #pragma unroll
-  for (int hh = 0; hh < HG; ++hh) mx[hh] = m_run[hh];
-  for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
-    const float4 v = *reinterpret_cast<const float4*>(sc + jj * HG);
-    mx[0] = fmaxf(mx[0], v.x); mx[1] = fmaxf(mx[1], v.y); mx[2] = fmaxf(mx[2], v.z); mx[3] = fmaxf(mx[3], v.w);
-  }
-#pragma unroll
-  for (int hh = 0; hh < HG; ++hh) mx[hh] = warp_max(mx[hh]);
-  __syncthreads();
-  if (l == 0) {
-#pragma unroll
-    for (int hh = 0; hh < HG; ++hh) red[w * HG + hh] = mx[hh];
-  }
-  __syncthreads();
-#pragma unroll
-  for (int hh = 0; hh < HG; ++hh) mx[hh] = warp_max(l < nw ? red[l * HG + hh] : -INFINITY);
-  float sum[HG] = {};
-  for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
-    float4 v = *reinterpret_cast<const float4*>(sc + jj * HG);
-    v.x = expf(v.x - mx[0]); v.y = expf(v.y - mx[1]); v.z = expf(v.z - mx[2]); v.w = expf(v.w - mx[3]);
-    *reinterpret_cast<float4*>(sc + jj * HG) = v;
-    sum[0] += v.x; sum[1] += v.y; sum[2] += v.z; sum[3] += v.w;
-  }
-#pragma unroll
-  for (int hh = 0; hh < HG; ++hh) sum[hh] = warp_sum(sum[hh]);
-  __syncthreads();  // every thread has read the maxima
-  if (l == 0) {
-#pragma unroll
-    for (int hh = 0; hh < HG; ++hh) red[w * HG + hh] = sum[hh];
-  }
-  __syncthreads();  // also publishes the exponentials in sc[]
-#pragma unroll
-  for (int hh = 0; hh < HG; ++hh) {
-    fac[hh] = m_run[hh] == -INFINITY ? 0.f : expf(m_run[hh] - mx[hh]);
-    l_run[hh] = l_run[hh] * fac[hh] + warp_sum(l < nw ? red[l * HG + hh] : 0.f);
-    m_run[hh] = mx[hh];
-    inv[hh] = last_block ? 1.f / l_run[hh] : 1.f;
-  }
-  // entry r of head hh: this block's weighted sum joins the earlier ones; the last block leaves
-  auto put = [&](int hh, int r, float tot) {
-    const float v = acc_s[hh * a.R + r] * fac[hh] + tot;
-    if (!last_block) acc_s[hh * a.R + r] = v;
-    else if (hh < nh) a.ctx[(size_t)t * a.ldc + (size_t)(h0 + hh) * a.R + r] = v * inv[hh];
-  };
-  if (sizeof(CT) == 2 && (D & 7) == 0 && (a.R & 7) == 0 && a.R / 8 <= (int)blockDim.x) {
-    // bf16 rows: a thread owns 8 consecutive latent entries (one 16-byte load per key), the block's threads form G groups
-    // that take every G-th key, so many loads are in flight per SM; groups are summed in group order, one head at a time
-    const int RC = a.R / 8, G = blockDim.x / RC, g = threadIdx.x / RC, c = threadIdx.x % RC;
-    const bf16* base = reinterpret_cast<const bf16*>(cache) + c * 8;
-    float acc[HG][8] = {};
-    auto add_key = [&](const uint4& u, const float4& p) {
-      const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&u);
-      const float pw[HG] = {p.x, p.y, p.z, p.w};
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = __bfloat1622float2(p2[e]);
-#pragma unroll
-        for (int hh = 0; hh < HG; ++hh) {
-          acc[hh][2 * e] = fmaf(pw[hh], f.x, acc[hh][2 * e]);
-          acc[hh][2 * e + 1] = fmaf(pw[hh], f.y, acc[hh][2 * e + 1]);
-        }
-      }
-    };
-    if (g < G) {
-      int jj = g;
-      for (; jj + G < n; jj += 2 * G) {  // two rows in flight; added in key order
-        const uint4 u0 = *reinterpret_cast<const uint4*>(base + (size_t)rowoff[jj] * D);
-        const uint4 u1 = *reinterpret_cast<const uint4*>(base + (size_t)rowoff[jj + G] * D);
-        add_key(u0, *reinterpret_cast<const float4*>(sc + jj * HG));
-        add_key(u1, *reinterpret_cast<const float4*>(sc + (jj + G) * HG));
-      }
-      if (jj < n) add_key(*reinterpret_cast<const uint4*>(base + (size_t)rowoff[jj] * D), *reinterpret_cast<const float4*>(sc + jj * HG));
+    for (int hh = 0; hh < HG; ++hh) mx[hh] = warp_max(l < nw ? red[l * HG + hh] : -INFINITY);
+    float sum[HG] = {};
+    for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
+      float4 v = *reinterpret_cast<const float4*>(sc + jj * HG);
+      v.x = expf(v.x - mx[0]); v.y = expf(v.y - mx[1]); v.z = expf(v.z - mx[2]); v.w = expf(v.w - mx[3]);
+      *reinterpret_cast<float4*>(sc + jj * HG) = v;
+      sum[0] += v.x; sum[1] += v.y; sum[2] += v.z; sum[3] += v.w;
     }
+#pragma unroll
+    for (int hh = 0; hh < HG; ++hh) sum[hh] = warp_sum(sum[hh]);
+    __syncthreads();  // every thread has read the maxima
+    if (l == 0) {
+#pragma unroll
+      for (int hh = 0; hh < HG; ++hh) red[w * HG + hh] = sum[hh];
+    }
+    __syncthreads();  // also publishes the exponentials in sc[]
 #pragma unroll
     for (int hh = 0; hh < HG; ++hh) {
-      __syncthreads();
+      fac[hh] = m_run[hh] == -INFINITY ? 0.f : expf(m_run[hh] - mx[hh]);
+      l_run[hh] = l_run[hh] * fac[hh] + warp_sum(l < nw ? red[l * HG + hh] : 0.f);
+      m_run[hh] = mx[hh];
+      inv[hh] = last_block ? 1.f / l_run[hh] : 1.f;
+    }
+    // entry r of head hh: this block's weighted sum joins the earlier ones; the last block leaves
+    auto put = [&](int hh, int r, float tot) {
+      const float v = acc_s[hh * a.R + r] * fac[hh] + tot;
+      if (!last_block) acc_s[hh * a.R + r] = v;
+      else if (hh < nh) a.ctx[(size_t)t * a.ldc + (size_t)(h0 + hh) * a.R + r] = v * inv[hh];
+    };
+    if (sizeof(CT) == 2 && (D & 7) == 0 && (a.R & 7) == 0 && a.R / 8 <= (int)blockDim.x) {
+      // bf16 rows: a thread owns 8 consecutive latent entries (one 16-byte load per key), the block's threads form G groups
+      // that take every G-th key, so many loads are in flight per SM; groups are summed in group order, one head at a time
+      const int RC = a.R / 8, G = blockDim.x / RC, g = threadIdx.x / RC, c = threadIdx.x % RC;
+      const bf16* base = reinterpret_cast<const bf16*>(cache) + c * 8;
+      float acc[HG][8] = {};
+      auto add_key = [&](const uint4& u, const float4& p) {
+        const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&u);
+        const float pw[HG] = {p.x, p.y, p.z, p.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = __bfloat1622float2(p2[e]);
+#pragma unroll
+          for (int hh = 0; hh < HG; ++hh) {
+            acc[hh][2 * e] = fmaf(pw[hh], f.x, acc[hh][2 * e]);
+            acc[hh][2 * e + 1] = fmaf(pw[hh], f.y, acc[hh][2 * e + 1]);
+          }
+        }
+      };
       if (g < G) {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) part[g * a.R + c * 8 + e] = acc[hh][e];
-      }
-      __syncthreads();
-      if (hh < nh)
-        for (int r = threadIdx.x; r < a.R; r += blockDim.x) {
-          float tot = 0.f;
-          for (int gg = 0; gg < G; ++gg) tot += part[gg * a.R + r];
-          put(hh, r, tot);
+        int jj = g;
+        for (; jj + G < n; jj += 2 * G) {  // two rows in flight; added in key order
+          const uint4 u0 = *reinterpret_cast<const uint4*>(base + (size_t)rowoff[jj] * D);
+          const uint4 u1 = *reinterpret_cast<const uint4*>(base + (size_t)rowoff[jj + G] * D);
+          add_key(u0, *reinterpret_cast<const float4*>(sc + jj * HG));
+          add_key(u1, *reinterpret_cast<const float4*>(sc + (jj + G) * HG));
         }
-    }
-    continue;
-  }
-  const int Rp = (a.R + 31) / 32 * 32;
-  const int G = max(1, (int)blockDim.x / Rp);
-  for (int r0 = 0; r0 < a.R; r0 += blockDim.x) {  // one pass unless the latent is wider than the block
-    const int g = (G > 1) ? threadIdx.x / Rp : 0, r = r0 + ((G > 1) ? threadIdx.x % Rp : threadIdx.x);
-    float acc[HG] = {};
-    if (g < G && r < a.R) {
-      const CT* col = cache + r;
-      int jj = g;
-      for (; jj + G < n; jj += 2 * G) {  // two independent loads in flight; the sum keeps key order
-        const float c0 = ldf<CT>(col, (size_t)rowoff[jj] * D), c1 = ldf<CT>(col, (size_t)rowoff[jj + G] * D);
-        const float4 p0 = *reinterpret_cast<const float4*>(sc + jj * HG), p1 = *reinterpret_cast<const float4*>(sc + (jj + G) * HG);
-        acc[0] = fmaf(p0.x, c0, acc[0]); acc[1] = fmaf(p0.y, c0, acc[1]); acc[2] = fmaf(p0.z, c0, acc[2]); acc[3] = fmaf(p0.w, c0, acc[3]);
-        acc[0] = fmaf(p1.x, c1, acc[0]); acc[1] = fmaf(p1.y, c1, acc[1]); acc[2] = fmaf(p1.z, c1, acc[2]); acc[3] = fmaf(p1.w, c1, acc[3]);
+        if (jj < n) add_key(*reinterpret_cast<const uint4*>(base + (size_t)rowoff[jj] * D), *reinterpret_cast<const float4*>(sc + jj * HG));
       }
-      for (; jj < n; jj += G) {
-        const float c0 = ldf<CT>(col, (size_t)rowoff[jj] * D);
-        const float4 p0 = *reinterpret_cast<const float4*>(sc + jj * HG);
-        acc[0] = fmaf(p0.x, c0, acc[0]); acc[1] = fmaf(p0.y, c0, acc[1]); acc[2] = fmaf(p0.z, c0, acc[2]); acc[3] = fmaf(p0.w, c0, acc[3]);
+#pragma unroll
+      for (int hh = 0; hh < HG; ++hh) {
+        __syncthreads();
+        if (g < G) {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) part[g * a.R + c * 8 + e] = acc[hh][e];
+        }
+        __syncthreads();
+        if (hh < nh)
+          for (int r = threadIdx.x; r < a.R; r += blockDim.x) {
+            float tot = 0.f;
+            for (int gg = 0; gg < G; ++gg) tot += part[gg * a.R + r];
+            put(hh, r, tot);
+          }
       }
+      continue;
     }
-    if (G > 1) {
-      __syncthreads();
-#pragma unroll
-      for (int hh = 0; hh < HG; ++hh) part[threadIdx.x * HG + hh] = acc[hh];
-      __syncthreads();
-      if (threadIdx.x < a.R) {
-#pragma unroll
-        for (int hh = 0; hh < HG; ++hh) {
-          float tot = 0.f;
-          for (int gg = 0; gg < G; ++gg) tot += part[(gg * Rp + threadIdx.x) * HG + hh];
-          put(hh, threadIdx.x, tot);
+    const int Rp = (a.R + 31) / 32 * 32;
+    const int G = max(1, (int)blockDim.x / Rp);
+    for (int r0 = 0; r0 < a.R; r0 += blockDim.x) {  // one pass unless the latent is wider than the block
+      const int g = (G > 1) ? threadIdx.x / Rp : 0, r = r0 + ((G > 1) ? threadIdx.x % Rp : threadIdx.x);
+      float acc[HG] = {};
+      if (g < G && r < a.R) {
+        const CT* col = cache + r;
+        int jj = g;
+        for (; jj + G < n; jj += 2 * G) {  // two independent loads in flight; the sum keeps key order
+          const float c0 = ldf<CT>(col, (size_t)rowoff[jj] * D), c1 = ldf<CT>(col, (size_t)rowoff[jj + G] * D);
+          const float4 p0 = *reinterpret_cast<const float4*>(sc + jj * HG), p1 = *reinterpret_cast<const float4*>(sc + (jj + G) * HG);
+          acc[0] = fmaf(p0.x, c0, acc[0]); acc[1] = fmaf(p0.y, c0, acc[1]); acc[2] = fmaf(p0.z, c0, acc[2]); acc[3] = fmaf(p0.w, c0, acc[3]);
+          acc[0] = fmaf(p1.x, c1, acc[0]); acc[1] = fmaf(p1.y, c1, acc[1]); acc[2] = fmaf(p1.z, c1, acc[2]); acc[3] = fmaf(p1.w, c1, acc[3]);
+        }
+        for (; jj < n; jj += G) {
+          const float c0 = ldf<CT>(col, (size_t)rowoff[jj] * D);
+          const float4 p0 = *reinterpret_cast<const float4*>(sc + jj * HG);
+          acc[0] = fmaf(p0.x, c0, acc[0]); acc[1] = fmaf(p0.y, c0, acc[1]); acc[2] = fmaf(p0.z, c0, acc[2]); acc[3] = fmaf(p0.w, c0, acc[3]);
         }
       }
-    } else if (r < a.R) {
+      if (G > 1) {
+        __syncthreads();
 #pragma unroll
-      for (int hh = 0; hh < HG; ++hh)
-        put(hh, r, acc[hh]);
+        for (int hh = 0; hh < HG; ++hh) part[threadIdx.x * HG + hh] = acc[hh];
+        __syncthreads();
+        if (threadIdx.x < a.R) {
+#pragma unroll
+          for (int hh = 0; hh < HG; ++hh) {
+            float tot = 0.f;
+            for (int gg = 0; gg < G; ++gg) tot += part[(gg * Rp + threadIdx.x) * HG + hh];
+            put(hh, threadIdx.x, tot);
+          }
+        }
+      } else if (r < a.R) {
+#pragma unroll
+        for (int hh = 0; hh < HG; ++hh)
+          put(hh, r, acc[hh]);
+      }
     }
-  }
   }
 }
 
