@@ -40,7 +40,9 @@ class LayerDescC(C.Structure):
                 ("weights_of", C.c_int32), ("rope_linear", C.c_float), ("norm_groups", C.c_int32), ("gate_cap", C.c_float),
                 ("side_mixer", C.c_int32), ("side_heads", C.c_int32), ("side_dim", C.c_int32), ("side_vdim", C.c_int32),
                 ("side_gate_cap", C.c_float), ("mix_scale", C.c_float), ("side_scale", C.c_float),
-                ("route_bias", C.c_int32), ("reserved", C.c_int32 * 4)]
+                ("route_bias", C.c_int32), ("route_group_max", C.c_int32), ("route_plain", C.c_int32),
+                ("rope_yarn_factor", C.c_float), ("rope_yarn_fast", C.c_float), ("rope_yarn_slow", C.c_float),
+                ("reserved", C.c_int32 * 3), ("head_decay", C.POINTER(C.c_float))]
 
 
 class StackDescC(C.Structure):
@@ -48,7 +50,9 @@ class StackDescC(C.Structure):
                 ("norm_eps", C.c_float), ("resid_alpha", C.c_float), ("logit_softcap", C.c_float), ("norm_place", C.c_int32),
                 ("embed_norm", C.c_int32), ("plain_gains", C.c_int32), ("norm_kind", C.c_int32), ("embed_scale", C.c_float),
                 ("logit_scale", C.c_float), ("tie_head", C.c_int32), ("one_norm", C.c_int32),
-                ("layer_scale", C.c_int32), ("resid_mult", C.c_float), ("reserved", C.c_int32 * 1)]
+                ("layer_scale", C.c_int32), ("resid_mult", C.c_float), ("streams", C.c_int32), ("bigram_buckets", C.c_int32),
+                ("bigram_mul_prev", C.c_int32), ("bigram_mul_cur", C.c_int32), ("loop_start", C.c_int32), ("loop_stop", C.c_int32),
+                ("loop_times", C.c_int32), ("reserved", C.c_int32 * 2)]
 
 
 class SeqFeedC(C.Structure):

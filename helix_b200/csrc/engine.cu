@@ -255,6 +255,7 @@ StepLayout Engine::layout(int T, int B, size_t pen_entries) const {
   L.first = o; o = al16(o + 4 * (size_t)B);
   L.seqof = o; o = al16(o + 4 * (size_t)T);   // entry of each token, rows whose logits are wanted
   L.rows = o; o = al16(o + 4 * (size_t)T);
+  L.prev = o; o = al16(o + 4 * (size_t)T);    // the token before each token (-1: none), read by bigram embeddings
   L.pen = o; o = al16(o + 8 * pen_entries);  // {int32 token; float value} entries, last so no offset depends on their number
   L.total = o;
   return L;
@@ -1320,6 +1321,7 @@ int Engine::run_prefill(std::vector<Request*>& batch) {
   int32_t* first = (int32_t*)(h_step_ + L.first);
   int32_t* seqof = (int32_t*)(h_step_ + L.seqof);
   int32_t* rows = (int32_t*)(h_step_ + L.rows);
+  int32_t* prev = (int32_t*)(h_step_ + L.prev);
   int n_rows = 0;
   step_entries_.clear();
   int32_t* tok = (int32_t*)(h_step_ + L.tokens);
@@ -1345,6 +1347,7 @@ int Engine::run_prefill(std::vector<Request*>& batch) {
       pos[t] = j;
       slot[t] = r->pages[j / page_] * page_ + j % page_;
       seqof[t] = i;
+      prev[t] = j > 0 ? token_at(r, j - 1) : -1;
     }
     last[i] = t - 1;
     ctx[i] = end;
@@ -1414,6 +1417,7 @@ int Engine::run_decode(std::vector<Request*>& batch) {
     ((int32_t*)(h_step_ + L.sslot))[i] = r->state_slot;
     ((int32_t*)(h_step_ + L.first))[i] = p;
     ((int32_t*)(h_step_ + L.seqof))[i] = i;
+    ((int32_t*)(h_step_ + L.prev))[i] = p > 0 ? token_at(r, p - 1) : -1;
     if (i == 0) step_entries_.clear();
     step_entries_.push_back(StepEntry{i, p, 1});
     tok[i] = r->out.back();

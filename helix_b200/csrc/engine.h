@@ -52,7 +52,7 @@ struct Request {
 };
 
 struct StepLayout {
-  size_t tokens, positions, slots, cu, last, ctx, pt, temp, seed, topk, topp, lpw, pen_off, sslot, first, seqof, rows, pen, total;
+  size_t tokens, positions, slots, cu, last, ctx, pt, temp, seed, topk, topp, lpw, pen_off, sslot, first, seqof, rows, prev, pen, total;
 };
 enum StepFlags : int { STEP_FILTER = 1, STEP_PENALTY = 2, STEP_LOGPROBS = 4 };
 
@@ -192,7 +192,8 @@ class Engine {
   struct StackWs {
     float *x, *p1, *p2, *cq, *qabs, *ctx, *mo, *y;
     bf16 *x16, *cq16, *mo16;
-    float* hn = nullptr;      // HB_NORM_BOTH_SIDES: the normed input of the current sublayer [T][width] (x16 is then ITS bf16 copy)
+    // x: [T][width], with stream copies [T][streams][width]
+    float* hn = nullptr;      // HB_NORM_BOTH_SIDES, HB_NORM_PRE: the normed input of the current sublayer [T][width] (x16 is then ITS bf16 copy)
     float* y2 = nullptr;      // mixture of experts with a unit every token uses: that unit's output [T][width]; HB_NORM_PARALLEL: the feed-forward's
     float* hn2 = nullptr;     // HB_NORM_PARALLEL: the normed input of the feed-forward [T][width] and its bf16 copy (hn / x16: the mixer's)
     bf16* x16b = nullptr;
@@ -231,6 +232,7 @@ class Engine {
     std::vector<const double*> freq_sets;
     std::vector<int> freq_half;
     std::vector<float*> rope_cs;
+    std::vector<float> freq_mult;  // factor of cos and sin (YaRN scaling), part of what makes two rotations distinct
     std::vector<int> layer_set;
   } sk_{};
   struct StepEntry { int t0, first, n; };  // host copy of the step's entries: first packed row, first position, tokens

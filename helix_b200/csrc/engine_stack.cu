@@ -1,4 +1,4 @@
-// Layer-list decoders (HB_ARCH_STACK: the Risepel, Lurepel, Latanex, Funudra and Kamivik designs) inside hb::Engine: model load, the page pool's planes and recurrent state slots,
+// Layer-list decoders (HB_ARCH_STACK: the Risepel, Lurepel, Latanex, Funudra, Kamivik and Pupalix designs) inside hb::Engine: model load, the page pool's planes and recurrent state slots,
 // the step's forward pass and the driven-sequence entry points.  Scheduling, page bookkeeping, the step block, sampling
 // and request records are the engine's own (engine.cu); this file adds what differs from the Llama path:
 //   * the residual stream is fp32 and post-normed; every sublayer reads the stream itself;
@@ -33,6 +33,10 @@
 //     and state of their own; logits from the embedding table;
 //   * parallel sublayers behind ONE norm, with gains on both outputs and a factor of their sum; a mixture's weighted rows join the
 //     same launch.
+//   * pre-normed stacks over several copies of the stream (hyper-connections): one launch between two sublayers mixes the copies,
+//     adds the output, reads the next input and norms it; linear attention with constant decays per head on the scalar-decay
+//     recurrence; rows picked by token pairs added to the embedding; runs of layers passed through several times (unrolled at
+//     load: later passes share the tensors, their planes and state are their own).
 #include "engine.h"
 #include "launch.h"
 
@@ -84,20 +88,24 @@ __global__ void fill_uniform_kernel(T* p, size_t n, uint64_t seed, float amp, fl
   } while (0)
 
 // ------------------------------------------------------------------ load
-int Engine::load_begin_stack(const hb_stack_desc& sd, const hb_layer_desc* layers) {
+int Engine::load_begin_stack(const hb_stack_desc& desc, const hb_layer_desc* layers) {
   std::lock_guard<std::mutex> g(gpu_mu_);
   if (loaded_ || load_open_) return fail(HB_ERR_STATE, "model already loaded on this engine");
-  if (!layers || sd.n_layers <= 0) return fail(HB_ERR_INVALID, "unsupported model description: no layer list");
+  if (!layers || desc.n_layers <= 0) return fail(HB_ERR_INVALID, "unsupported model description: no layer list");
   // no position reaches max_ctx, so a longer window sees what a window of max_ctx sees: size the kernels for the shorter one
-  std::vector<hb_layer_desc> lv(layers, layers + sd.n_layers);
+  std::vector<hb_layer_desc> lv(layers, layers + desc.n_layers);
   for (hb_layer_desc& l : lv) {
     if (l.mixer == HB_MIXER_LATENT && (l.mask == HB_MASK_CAUSAL || l.window > cfg_.max_ctx)) { l.mask = HB_MASK_WINDOW; l.window = cfg_.max_ctx; }
     if (l.mixer == HB_MIXER_GQA) {  // a block or window that no sequence outgrows is the causal mask
       if (l.mask == HB_MASK_CAUSAL || l.window >= cfg_.max_ctx) { l.mask = HB_MASK_WINDOW; l.window = cfg_.max_ctx; }
     }
   }
+  hb_stack_desc sd = desc;
+  std::vector<int> ids;
+  std::string why = unroll_stack(sd, lv, ids);
+  if (!why.empty()) return fail(HB_ERR_INVALID, "unsupported model description: " + why);
   layers = lv.data();
-  const std::string why = validate_stack(sd, layers);
+  why = validate_stack(sd, layers);
   if (!why.empty()) return fail(HB_ERR_INVALID, "unsupported model description: " + why);
   // the per-token attention kernel keeps one position's scores in shared memory.  Steps replayed from graphs fix that size at
   // capture, so a full context has to fit; otherwise each launch is sized by its step's longest context and a sequence that
@@ -110,6 +118,12 @@ int Engine::load_begin_stack(const hb_stack_desc& sd, const hb_layer_desc* layer
   CU(cudaMemGetInfo(&free_b, &total_b));
   budget_ = cfg_.memory_budget_bytes ? cfg_.memory_budget_bytes : (free_b > (1ull << 30) ? free_b - (1ull << 30) : free_b);
   model_.sd = sd;
+  model_.layer_id = ids;
+  model_.head_decay.assign(sd.n_layers, {});
+  for (int i = 0; i < sd.n_layers; ++i) {  // the caller's arrays live for this call only
+    if (lv[i].mixer == HB_MIXER_LIGHTNING) model_.head_decay[i].assign(lv[i].head_decay, lv[i].head_decay + lv[i].heads);
+    lv[i].head_decay = model_.head_decay[i].empty() ? nullptr : model_.head_decay[i].data();
+  }
   model_.sl.assign(layers, layers + sd.n_layers);
   hb_model_desc d{};
   d.arch = HB_ARCH_RISEPEL;
@@ -235,6 +249,7 @@ struct StackDims {
   int cv = 0;                // widest convolved row (state-space layers, grouped-query layers with convolved projections)
   size_t lat_qh = 0, lat_r = 0, lat_v = 0, lat_ws = 0;  // latent layers on the tensor cores: elements per head-major block / split partials
   int lat_rank = 0, lat_rot = 0, lat_kv = 0, lat_heads = 0;  // ... and widest latent, rotated part, expanded row, most heads
+  size_t decays = 0;         // constant decays over all layer runs
   int ab = 0;                // most heads of a scalar-decay recurrence (decay, input weight, exp(-m), n . q per head and token)
 };
 // Grouped-query layers whose prompt portions run on the fused tcgen05 attention kernel (the one the Llama path uses, with
@@ -274,6 +289,9 @@ static StackDims stack_dims(const Model& m, int max_ctx, int tokens) {
       d.cv = std::max(d.cv, l.heads * l.vdim + 2 * l.kv_heads * l.dim);
       d.ab = std::max(d.ab, l.heads);
     } else if (l.mixer == HB_MIXER_MLSTM) {
+    } else if (l.mixer == HB_MIXER_LIGHTNING) {
+      d.cx = std::max(d.cx, l.heads * l.vdim);
+      d.decays += l.heads;
     } else if (l.mixer == HB_MIXER_DELTA) {
       d.n2 = std::max(d.n2, 2 * l.kv_heads * l.dim + l.heads * l.vdim + 2 * l.heads + l.kv_heads);
       d.cx = std::max(d.cx, l.heads * l.vdim);
@@ -332,6 +350,7 @@ size_t Engine::workspace_bytes_stack() const {
   const StackDims dm = stack_dims(model_, cfg_.max_ctx, t_cap_);
   const int n1 = dm.n1, n2 = dm.n2, q = dm.q, qa = dm.qa, cx = dm.cx, mo = dm.mo;
   size_t b = 0;
+  b += al256(dm.decays * 4);
   b += al256((size_t)std::max(dm.rope_half, 1) * 8) + al256(T * 2 * (size_t)std::max(dm.rope_half, 1) * 4);
   if (dm.att > 0) b += al256(T * (size_t)up8(dm.att) * 2) + al256(attn_decode_workspace_floats(cfg_.max_seqs, dm.att_heads, dm.att_dim, 16) * 4);
   if (dm.moe_r > 0) {
@@ -351,8 +370,8 @@ size_t Engine::workspace_bytes_stack() const {
     b += al256(dm.lat_qh * 2) + 2 * al256(dm.lat_r * 2) + al256(dm.lat_v * 4) + al256(dm.lat_ws * 4) + al256((size_t)dm.lat_heads * 4) +
          al256(rows * dm.lat_rank * 2) + al256(rows * dm.lat_rot * 2) + al256(rows * dm.lat_kv * 2);
   }
-  b += 2 * al256(T * W * 4) + al256(T * W * 2);                       // x, y, x16
-  if (sd.norm_place == HB_NORM_BOTH_SIDES || sd.norm_place == HB_NORM_PARALLEL) b += al256(T * W * 4);     // hn
+  b += al256(T * W * 4 * std::max(sd.streams, 1)) + al256(T * W * 4) + al256(T * W * 2);  // x, y, x16
+  if (sd.norm_place == HB_NORM_BOTH_SIDES || sd.norm_place == HB_NORM_PARALLEL || sd.norm_place == HB_NORM_PRE) b += al256(T * W * 4);     // hn
   if (sd.norm_place == HB_NORM_PARALLEL) b += al256(T * W * 4) + al256(T * W * 2);  // hn2, x16b
   if (dm.shared || sd.norm_place == HB_NORM_PARALLEL) b += al256(T * W * 4);                               // y2
   b += al256(T * (size_t)up8(dm.cv) * 4) + al256(T * (size_t)up8(4 * dm.ab) * 4);  // cv, ab
@@ -382,6 +401,7 @@ int Engine::alloc_runtime_stack() {
   CU(stack_moe_init());
   CU(stack_delta_init());
   CU(stack_ssm_init());
+  CU(stack_streams_init());
   CU(attn_latent_init());
   if (!sd.compute_f32) {  // stream-K plans allocate on first use of a shape: make them now, not inside a graph capture
     SmLimitScope sm_scope(cfg_.sm_budget);
@@ -417,24 +437,36 @@ int Engine::alloc_runtime_stack() {
   const size_t T = t_cap_, W = sd.width;
   const StackDims dm = stack_dims(model_, cfg_.max_ctx, t_cap_);
   const int n1 = dm.n1, n2 = dm.n2, q = dm.q, qa = dm.qa, cx = dm.cx, mo = dm.mo;
+  {  // constant decays of the linear-attention layers
+    float* dc = (float*)take(dm.decays * 4);
+    for (int i = 0; i < sd.n_layers; ++i) {
+      const std::vector<float>& v = model_.head_decay[i];
+      if (v.empty()) continue;
+      CU(cudaMemcpy(dc, v.data(), v.size() * 4, cudaMemcpyHostToDevice));
+      model_.sw[i].decay = dc;
+      dc += v.size();
+    }
+  }
   {  // rotation frequencies of the attention layers (double precision, formed on the host)
     double* fq = (double*)take((size_t)std::max(dm.rope_half, 1) * 8);
     float* cs = (float*)take(T * 2 * (size_t)std::max(dm.rope_half, 1) * 4);
     sk_.layer_set.assign(sd.n_layers, -1);
-    sk_.freq_sets.clear(); sk_.freq_half.clear(); sk_.rope_cs.clear();
+    sk_.freq_sets.clear(); sk_.freq_half.clear(); sk_.rope_cs.clear(); sk_.freq_mult.clear();
     std::vector<std::vector<double>> sets;
     size_t at = 0;
     for (int i = 0; i < sd.n_layers; ++i) {
       const hb_layer_desc& l = model_.sl[i];
       if ((l.mixer != HB_MIXER_GQA && l.mixer != HB_MIXER_LATENT) || l.rope_dims <= 0) continue;
       const std::vector<double> f = stack_rope_freqs(l);
+      const float mult = stack_rope_mult(l);
       size_t sidx = 0;
-      while (sidx < sets.size() && sets[sidx] != f) ++sidx;
+      while (sidx < sets.size() && (sets[sidx] != f || sk_.freq_mult[sidx] != mult)) ++sidx;
       if (sidx == sets.size()) {
         CU(cudaMemcpy(fq + at, f.data(), f.size() * 8, cudaMemcpyHostToDevice));
         sets.push_back(f);
         sk_.freq_sets.push_back(fq + at);
         sk_.freq_half.push_back((int)f.size());
+        sk_.freq_mult.push_back(mult);
         sk_.rope_cs.push_back(cs + T * 2 * at);
         at += f.size();
       }
@@ -487,11 +519,11 @@ int Engine::alloc_runtime_stack() {
     CU(cudaMemcpy(sk_.lat_heads, ids.data(), ids.size() * 4, cudaMemcpyHostToDevice));
   }
   sk_.ld1 = up8(n1); sk_.ld2 = up8(n2); sk_.ldcq = up8(q); sk_.ldqa = up8(qa); sk_.ldctx = up8(cx); sk_.ldmo = up8(mo);
-  sk_.x = (float*)take(T * W * 4);
+  sk_.x = (float*)take(T * W * 4 * std::max(sd.streams, 1));
   sk_.y = (float*)take(T * W * 4);
   sk_.x16 = (bf16*)take(T * W * 2);
   const bool par = sd.norm_place == HB_NORM_PARALLEL;
-  sk_.hn = (sd.norm_place == HB_NORM_BOTH_SIDES || par) ? (float*)take(T * W * 4) : nullptr;
+  sk_.hn = (sd.norm_place == HB_NORM_BOTH_SIDES || sd.norm_place == HB_NORM_PRE || par) ? (float*)take(T * W * 4) : nullptr;
   sk_.hn2 = par ? (float*)take(T * W * 4) : nullptr;
   sk_.x16b = par ? (bf16*)take(T * W * 2) : nullptr;
   sk_.y2 = (dm.shared || par) ? (float*)take(T * W * 4) : nullptr;
@@ -637,7 +669,7 @@ int Engine::latent_attention_tc(int T, const StepLayout& L, const hb_layer_desc&
   StackWs& k = sk_;
   const int H = l.heads, Dk = l.dim, Dv = l.vdim, R = l.kv_rank, Dr = l.rot_dim, Dq = Dk + Dr;
   const int window = l.window < cfg_.max_ctx ? l.window : 0;
-  const bool head_gate = (l.attn_flags & HB_ATTN_HEAD_GATE) != 0;
+  const bool head_gate = (l.attn_flags & HB_ATTN_HEAD_GATE) != 0, no_gate = (l.attn_flags & HB_ATTN_NO_GATE) != 0;
   const bf16* cache = (const bf16*)((uint8_t*)kv_ + plane_off_[w.cache_plane]);
   // ---- long portions: the rows each of them sees are expanded, then one attention launch per group of portions
   LatentRuns lr{};
@@ -680,7 +712,7 @@ int Engine::latent_attention_tc(int T, const StepLayout& L, const hb_layer_desc&
   }
   int rc = launch_group();
   if (rc != HB_OK) return rc;
-  if (!head_gate) {  // a gate per entry: neighbouring long portions in one pass
+  if (!head_gate && !no_gate) {  // a gate per entry: neighbouring long portions in one pass
     int g0 = 0, g1 = 0;
     auto gate = [&]() -> int {
       if (g1 > g0)
@@ -723,8 +755,8 @@ int Engine::latent_attention_tc(int T, const StepLayout& L, const hb_layer_desc&
       GemmArgs g2{k.lat_ctx, R, (const bf16*)w.uv, R, k.lat_ov, Dv, nullptr, 0, nullptr, M, Dv, R, EPI_F32, 0};
       g2.m_tile_group = k.lat_heads; g2.groups = H;
       SPAN(0, 2.0 * M * Dv * R, gemm_bf16_tn(stream_, g2));
-      SPAN(3, 12.0 * n * H * Dv, latent_out_gate(stream_, k.lat_ov, Dv, (long)kLatentTokRows * Dv, k.p1 + (size_t)t0 * k.ld1 + w.off_g, k.ld1,
-                                                 head_gate, nullptr, k.mo16 + (size_t)t0 * H * Dv, n, H, Dv));
+      SPAN(3, 12.0 * n * H * Dv, latent_out_gate(stream_, k.lat_ov, Dv, (long)kLatentTokRows * Dv,
+                                                 no_gate ? nullptr : k.p1 + (size_t)t0 * k.ld1 + w.off_g, k.ld1, head_gate, nullptr, k.mo16 + (size_t)t0 * H * Dv, n, H, Dv));
     }
   return HB_OK;
 }
@@ -753,7 +785,8 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
   const bool par = sd.norm_place == HB_NORM_PARALLEL;
   // what a sublayer reads: the stream itself, or (norms on both sides, parallel sublayers) its normed copy; x16 is the bf16
   // copy of that.  With parallel sublayers the feed-forward has a normed copy of its own (hn2 / x16b).
-  const float* xin = (both || par) ? k.hn : k.x;
+  const bool pre = sd.norm_place == HB_NORM_PRE;
+  const float* xin = (both || par || pre) ? k.hn : k.x;
   const bool two_norms = par && !sd.one_norm;
   const float* ff_in = two_norms ? k.hn2 : xin;
   const bf16* ff_in16 = two_norms ? (f32 ? nullptr : k.x16b) : x16;
@@ -775,6 +808,29 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     }
     return parallel_step(stream_, k.x, nullptr, y, y2, bias, bias_scale, w1, w2, f32, sd.norm_eps, y ? k.x : nullptr, h1_f32 ? k.hn : nullptr, x16,
                          h2_f32 ? k.hn2 : nullptr, f32 ? nullptr : k.x16b, T, W, scale);
+  };
+  // pre-normed stacks: the output y of a sublayer (or its expert rows) joins the stream copies, and the input of what follows —
+  // sublayer `sub` (0 mixer, 1 feed-forward) of layer `next`, or behind the last layer the sum of the copies — is read and normed
+  auto pre_step = [&](const float* x0, const float* y, const void* bias, const HyperW* from, int next, int sub, const ParScale* fuse) -> cudaError_t {
+    StreamStep a{};
+    a.x = k.x; a.x0 = x0; a.y = y; a.bias = bias;
+    if (from && sd.streams > 0) { a.mix = from->mix; a.out = from->out; }
+    a.S = std::max(sd.streams, 1); a.W = W; a.f32 = f32; a.eps = sd.norm_eps; a.last = next >= sd.n_layers;
+    if (fuse && fuse->top_k > 0) { a.rows = fuse->rows; a.row_of = fuse->row_of; a.wts = fuse->wts; a.top_k = fuse->top_k; }
+    bool h_f32 = true;
+    if (!a.last) {
+      const hb_layer_desc& nl = model_.sl[next];
+      const StackLayerW& nw = model_.sw[next];
+      if (sd.streams > 0) a.in = sub == 0 ? nw.hc1.in : nw.hc2.in;
+      a.w = sub == 0 ? nw.norm1 : nw.norm2;
+      // the fp32 copy is written only where a product reads it (shapes the tensor-core GEMMs do not take)
+      if (sub == 0) h_f32 = !stack_tc(nw.n_in, W, W, nl.mixer == HB_MIXER_GQA ? up8(nw.n_in) : k.ld1);
+      else if (nl.ff_kind == HB_FF_MOE) h_f32 = f32 || nl.identity_experts > 0 || !router_tc(nl) || nl.shared_ff > 0;
+      else h_f32 = !stack_tc(nl.ff_kind == HB_FF_RELU2 ? nl.ff : 2 * nl.ff, W, W, k.ld1);
+    }
+    if (h_f32) a.h = k.hn;
+    a.h16 = a.last ? nullptr : x16;
+    return stream_step(stream_, a, T);
   };
   // the residual step: the norm covers the sum (post-norm stream) or the sublayer's output alone; with norms on both sides
   // the same launch also norms the input of the sublayer that follows (`pre`, null behind the last one)
@@ -821,6 +877,15 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     }
     return stack_gemm(k.mo, mo16, F, w_down, W, F, out, W, T);
   };
+  // clamped unit with biases into k.y (the residual step adds the last bias)
+  auto clamped_ff = [&](const hb_layer_desc& l, const StackLayerW& w) -> int {
+    const int F = l.ff;
+    int rc = stack_gemm(xin, x16, W, w.w_gu, 2 * F, W, k.p1, k.ld1, T);
+    if (rc != HB_OK) return rc;
+    const void* bu = (const uint8_t*)w.b_gu + (size_t)F * model_.elem;
+    SPAN(3, 12.0 * T * F, clamped_glu(stream_, k.p1, k.ld1, w.b_gu, bu, f32, l.ff_limit, 1.702f, k.mo, mo16, T, F));
+    return stack_gemm(k.mo, mo16, F, w.w_down, W, F, k.y, W, T);
+  };
   // ungated unit y = down(relu(up h)^2)
   auto relu2_ff = [&](const void* w_up, const void* w_down, int F, float* out) -> int {
     if (T > 256 && k.gu16 && F % 8 == 0 && stack_tc(F, W, W, F) && stack_tc(W, F, F, W)) {
@@ -840,7 +905,7 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     const int E = l.experts, R = l.experts + l.identity_experts, F = l.ff;
     RouteOpts ro;
     ro.sigmoid = l.router_kind == HB_ROUTER_SIGMOID; ro.groups = l.route_groups; ro.keep = l.route_keep; ro.renorm = l.route_renorm;
-    ro.chosen = l.router_kind == HB_ROUTER_CHOSEN; ro.bias = l.route_bias;
+    ro.chosen = l.router_kind == HB_ROUTER_CHOSEN; ro.bias = l.route_bias; ro.group_max = l.route_group_max;
     ro.scale = l.route_scale != 0.f ? l.route_scale : 1.f;
     const int eact = l.expert_kind == HB_EXPERT_CLAMPED ? GLU_CLAMPED : l.expert_kind == HB_EXPERT_GELU ? GLU_NONE_GELU : GLU_SILU;
     const float* add = nullptr;
@@ -928,12 +993,20 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
                                                   sd.norm_eps, scale, out_f32, mo16, ldout, col0, T, q.H, q.Dv));
     return HB_OK;
   };
-  SPAN(3, rowb, embed_rows_f32(stream_, tokens, model_.s_embed, f32, k.x, x16, T, W, sd.embed_scale != 0.f ? sd.embed_scale : 1.f));
-  if (sd.embed_norm) SPAN(3, 2 * rowb, norm_rows(k.x, nullptr, model_.s_embed_norm, k.x, both ? nullptr : x16, T));
+  BigramArgs bigram;
+  if (sd.bigram_buckets > 0) {
+    bigram.table = model_.s_bigram; bigram.prev = (const int32_t*)(d_step_ + L.prev);
+    bigram.buckets = sd.bigram_buckets; bigram.mul_prev = sd.bigram_mul_prev; bigram.mul_cur = sd.bigram_mul_cur;
+  }
+  float* x_emb = pre ? k.y : k.x;  // (pre-normed stacks: the first step below makes the copies)
+  SPAN(3, rowb, embed_rows_f32(stream_, tokens, model_.s_embed, f32, x_emb, pre ? nullptr : x16, T, W, sd.embed_scale != 0.f ? sd.embed_scale : 1.f, bigram));
+  if (sd.embed_norm) SPAN(3, 2 * rowb, norm_rows(x_emb, nullptr, model_.s_embed_norm, x_emb, both || pre ? nullptr : x16, T));
+  const double preb = (2.0 * std::max(sd.streams, 1) + 2.0) * rowb;
+  if (pre) SPAN(3, preb, pre_step(k.y, nullptr, nullptr, nullptr, 0, 0, nullptr));
   if (both) SPAN(3, 2 * rowb, norm_rows(k.x, nullptr, model_.sw[0].norm1, k.hn, x16, T));
   if (par) SPAN(3, 3 * rowb, par_step(nullptr, nullptr, nullptr, 0.f, 0, nullptr));
   for (size_t si = 0; si < k.freq_sets.size(); ++si)  // cos / sin of the step's positions, once per distinct rotation
-    SPAN(3, 8.0 * T * k.freq_half[si], stack_rope_table(stream_, positions, k.freq_sets[si], k.freq_half[si], k.rope_cs[si], T));
+    SPAN(3, 8.0 * T * k.freq_half[si], stack_rope_table(stream_, positions, k.freq_sets[si], k.freq_half[si], k.rope_cs[si], T, k.freq_mult[si]));
   for (int i = 0; i < sd.n_layers; ++i) {
     const hb_layer_desc& l = model_.sl[i];
     const StackLayerW& w = model_.sw[i];
@@ -975,6 +1048,20 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     } else if (l.mixer == HB_MIXER_MLSTM) {
       rc = run_memory(w, k.ld1, 0, ocols, 1.f, mo_f32);
       if (rc != HB_OK) return rc;
+    } else if (l.mixer == HB_MIXER_LIGHTNING) {
+      LinRecArgs ra{};
+      ra.q = k.p1; ra.ldq = k.ld1; ra.q_off = w.off_q;
+      ra.k = k.p1; ra.ldk = k.ld1; ra.k_off = w.off_k;
+      ra.v = k.p1; ra.ldv = k.ld1; ra.v_off = w.off_v;
+      ra.head_decay = w.decay; ra.silu = 1;
+      ra.out = k.ctx; ra.ldo = k.ldctx;
+      ra.f32 = f32; ra.q_scale = 1.f;
+      ra.state = state_; ra.slot_stride = (long)model_.state_floats; ra.s_off = w.state_off;
+      ra.cu = cu; ra.first_pos = first; ra.slots = sslot;
+      ra.B = B; ra.H = H; ra.G = H; ra.Dk = Dk; ra.Dv = Dv;
+      SPAN(6, 4.0 * T * H * Dk * Dv, lin_recurrence(stream_, ra));
+      SPAN(3, 16.0 * T * H * Dv, gated_group_norm(stream_, k.ctx, k.ldctx, k.p1 + w.off_g, k.ld1, w.hnorm, f32, sd.norm_eps, 1, mo_f32, mo16, T, H * Dv,
+                                                  true));
     } else if (l.mixer == HB_MIXER_DELTA) {
       const int G = l.kv_heads, GD = G * Dk, C = 2 * GD + H * Dv;
       DeltaPrepArgs pa{};
@@ -1248,7 +1335,8 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
         GemmRtArgs g{k.ctx, ldcx, (long)R, w.uv, (long)R, 1, (long)Dv * R, ov, ldov, (long)Dv, nullptr, T, Dv, R, H, f32};
         SPAN(5, 2.0 * T * H * Dv * R, gemm_rt(stream_, g));
       }
-      SPAN(3, 12.0 * T * H * Dv, latent_out_gate(stream_, ov, ldov, Dv, k.p1 + w.off_g, k.ld1, head_gate, k.mo, mo16, T, H, Dv));
+      SPAN(3, 12.0 * T * H * Dv, latent_out_gate(stream_, ov, ldov, Dv, (l.attn_flags & HB_ATTN_NO_GATE) ? nullptr : k.p1 + w.off_g, k.ld1,
+                                                 head_gate, k.mo, mo16, T, H, Dv));
       }
     }
     rc = stack_gemm(k.mo, mo16, ocols, w.wo, W, ocols, k.y, W, T);
@@ -1269,6 +1357,25 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
       SPAN(3, 5 * rowb, par_step(k.y, y2, w.o_bias, l.mix_scale != 0.f ? l.mix_scale : 1.f, i + 1, &scale));
       continue;
     }
+    if (pre) {
+      ParScale fuse;
+      SPAN(3, preb, pre_step(nullptr, k.y, w.o_bias, &w.hc1, l.ff > 0 ? i : i + 1, l.ff > 0 ? 1 : 0, nullptr));
+      if (l.ff <= 0) continue;
+      const void* bias = nullptr;
+      if (l.ff_kind == HB_FF_MOE) {
+        rc = moe_ff(l, w, k.y, &fuse);
+      } else if (l.ff_kind == HB_FF_RELU2) {
+        rc = relu2_ff(w.w_gu, w.w_down, l.ff, k.y);
+      } else if (l.ff_kind == HB_FF_CLAMPED) {
+        rc = clamped_ff(l, w);
+        bias = w.b_down;
+      } else {
+        rc = gated_ff(w.w_gu, w.w_down, l.ff, l.ff_kind == HB_FF_SILU ? GLU_SILU : GLU_GELU_TANH, 0.f, w.gu_packed, k.y);
+      }
+      if (rc != HB_OK) return rc;
+      SPAN(3, preb, pre_step(nullptr, fuse.top_k > 0 ? nullptr : k.y, bias, &w.hc2, i + 1, 0, &fuse));
+      continue;
+    }
     SPAN(3, 3 * rowb, resid(w.o_bias, both ? w.norm1b : w.norm1, l.ff > 0 ? w.norm2 : pre_next));
     if (l.ff > 0 && l.ff_kind == HB_FF_RELU2) {
       rc = relu2_ff(w.w_gu, w.w_down, l.ff, k.y);
@@ -1283,12 +1390,7 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
       if (rc != HB_OK) return rc;
       SPAN(3, 3 * rowb, resid(nullptr, both ? w.norm2b : w.norm2, pre_next));
     } else if (l.ff > 0) {
-      const int F = l.ff;
-      rc = stack_gemm(xin, x16, W, w.w_gu, 2 * F, W, k.p1, k.ld1, T);
-      if (rc != HB_OK) return rc;
-      const void* bu = (const uint8_t*)w.b_gu + (size_t)F * model_.elem;
-      SPAN(3, 12.0 * T * F, clamped_glu(stream_, k.p1, k.ld1, w.b_gu, bu, f32, l.ff_limit, 1.702f, k.mo, mo16, T, F));
-      rc = stack_gemm(k.mo, mo16, F, w.w_down, W, F, k.y, W, T);
+      rc = clamped_ff(l, w);
       if (rc != HB_OK) return rc;
       SPAN(3, 3 * rowb, resid(w.b_down, both ? w.norm2b : w.norm2, pre_next));
     }
@@ -1298,7 +1400,8 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     for (int r0 = 0; r0 < n; r0 += t_cap_) {  // the normed rows go through the (free) projection buffers, t_cap_ rows at a time
       const int m = std::min(t_cap_, n - r0);
       const int32_t* idx = rows ? rows + r0 : nullptr;
-      const float* src = rows ? k.x : k.x + (size_t)r0 * W;
+      const float* sum = pre ? k.hn : k.x;  // (pre-normed stacks: the last step left the sum of the copies there)
+      const float* src = rows ? sum : sum + (size_t)r0 * W;
       LAUNCH(norm_rows(src, idx, model_.s_final_norm, k.y, x16, m));
       int rc = stack_gemm(k.y, x16, W, model_.s_head, V, W, out + (size_t)r0 * V, V, m);
       if (rc != HB_OK) return rc;

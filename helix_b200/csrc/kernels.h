@@ -308,9 +308,15 @@ struct GemmRtArgs {
 };
 cudaError_t gemm_rt(cudaStream_t s, const GemmRtArgs& a);
 
-// x[t, :] = table[tokens[t], :] * scale as fp32 (+ bf16 copy)
+// A row picked by the pair (previous token, token) that is added to the embedding: (prev * mul_prev + token * mul_cur) mod buckets
+// (64-bit), row `buckets` where prev < 0 (the first token of a sequence).  prev [T].
+struct BigramArgs {
+  const void* table = nullptr; const int32_t* prev = nullptr;
+  int buckets = 0, mul_prev = 0, mul_cur = 0;
+};
+// x[t, :] = table[tokens[t], :] * scale (+ the bigram row) as fp32 (+ bf16 copy)
 cudaError_t embed_rows_f32(cudaStream_t s, const int32_t* tokens, const void* table, bool f32, float* x, bf16* x_b16, int T, int W,
-                           float scale = 1.f);
+                           float scale = 1.f, const BigramArgs& bigram = BigramArgs());
 // Residual step between element-wise norms N(v) = tanh(alpha v) * w + b; `post` / `pre` are blocks [w (W) | b (W) | alpha] of
 // the weight type or null.  v = x[row_index ? row_index[r] : r]; with y: v += post ? N_post(y[r]) : y[r] and x_out[r] = v
 // (x_out may be x); with pre: h[r] = N_pre(v) as fp32 (h) and / or bf16 (h_b16).
@@ -424,7 +430,8 @@ cudaError_t latent_rows(cudaStream_t s, const bf16* cache, const int32_t* page_t
                         const LatentRuns& runs, int rows);
 // qh[h][t][:] = the unrotated part of q[t]'s head h (t < T <= kLatentTokRows)
 cudaError_t latent_q_heads(cudaStream_t s, const bf16* q, int ldq, bf16* qh, int T, int H, int Dk, int Dr);
-// out[t, h Dv + i] = o[t * o_ts + h * o_hs + i] * sigmoid(g[t, per_head ? h : h Dv + i])   (fp32 in, fp32 + bf16 copy out)
+// out[t, h Dv + i] = o[t * o_ts + h * o_hs + i] * sigmoid(g[t, per_head ? h : h Dv + i])   (fp32 in, fp32 + bf16 copy out; g null:
+// no gate)
 cudaError_t latent_out_gate(cudaStream_t s, const float* o, long o_ts, long o_hs, const float* g, long ldg, bool per_head, float* out,
                             bf16* out_b16, int T, int H, int Dv);
 // The same attention as three dense products for a block of consecutive tokens of ONE sequence (long prompt portions in the
@@ -472,9 +479,9 @@ struct GqaPrepArgs {
 };
 cudaError_t gqa_prep(cudaStream_t s, const GqaPrepArgs& a);
 // cs[t][2i] = cos(a), cs[t][2i+1] = sin(a), a = positions[t] * freqs[i], i < half: the angle and its reduction to one turn in
-// double precision, sine and cosine of the remainder in fp32.  Once per step and per distinct frequency set, shared by every
+// double precision, sine and cosine of the remainder in fp32, both times mult.  Once per step and per distinct frequency set, shared by every
 // layer and head that rotates with it.
-cudaError_t stack_rope_table(cudaStream_t s, const int32_t* positions, const double* freqs, int half, float* cs, int T);
+cudaError_t stack_rope_table(cudaStream_t s, const int32_t* positions, const double* freqs, int half, float* cs, int T, float mult = 1.f);
 // out[t, h, :] = gate_h * sum_j p_j v_j over the keys position pos_t sees, p_j = exp(s_j) / (sum_i exp(s_i) + sink),
 // s_j = scale * q[t, h] . k_j (head h reads kv head h / (H / G)).  Visible keys: mask 0 (window) pos - window < j <= pos;
 // 1 (chunk) j <= pos in the block of `window` positions that holds pos; 2 (causal) j <= pos.  sink = 1 when unit_sink
@@ -569,6 +576,7 @@ cudaError_t exp_gate_scan(cudaStream_t s, const GateScanArgs& a);
 // S_t = a_t S_(t-1) + b_t k_t v_t^T;  out_t = q_scale * S_t^T q_t (+ skip[h] v_t) per (entry, head); query / key head of
 // head h: h / (H / G); a_t = ab[t, h], b_t = ab[t, H + h].  With nq: the vector n_t = a_t n_(t-1) + b_t k_t ([H][Dk] at
 // n_off of the slot) is carried too and nq[t, h] = q_scale * n_t . q_t.  S: [H][Dk][Dv] fp32 at s_off of the slot.
+// head_decay (instead of ab): a_t = head_decay[h], b_t = 1.  silu: q, k and v pass z * sigmoid(z) on their way in.
 struct LinRecArgs {
   const float* q; long ldq; int q_off;
   const float* k; long ldk; int k_off;
@@ -581,6 +589,8 @@ struct LinRecArgs {
   float* state; long slot_stride; size_t s_off, n_off;
   const int32_t* cu; const int32_t* first_pos; const int32_t* slots;
   int B, H, G, Dk, Dv;
+  const float* head_decay = nullptr;
+  int silu = 0;
 };
 cudaError_t lin_recurrence(cudaStream_t s, const LinRecArgs& a);
 // Matrix memory read-out: o = num[t, h, :] / (max(|nq[t, h]|, ab[t, 2H + h]) + 1e-6); out[t, col0 + h Dv + i] =
@@ -589,9 +599,10 @@ cudaError_t memory_readout(cudaStream_t s, const float* num, long ldnum, const f
                            const float* g, long ldg, const void* w, bool f32, float eps, float scale, float* out, bf16* out_b16,
                            long ldout, int col0, int T, int H, int Dv);
 // State-space read-out: u = y[t, :] * silu(z[t, :]) over n entries, divided by its root mean square in `parts` equal parts,
-// times w; out [T, n] (+ bf16 copy)
+// times w; out [T, n] (+ bf16 copy).  gate_last: u = y[t, :], and the normed row is multiplied by sigmoid(z[t, :]) instead
+// (linear attention with constant decays)
 cudaError_t gated_group_norm(cudaStream_t s, const float* y, long ldy, const float* z, long ldz, const void* w, bool f32, float eps,
-                             int parts, float* out, bf16* out_b16, int T, int n);
+                             int parts, float* out, bf16* out_b16, int T, int n, bool gate_last = false);
 // out[t, col0 + e] = in[t, e] * sigmoid(g[t, e]) * scale, e < n (in: fp32, or bf16 when in_b16 is given instead)
 cudaError_t gate_scale_rows(cudaStream_t s, const float* in, const bf16* in_b16, long ldi, const float* g, long ldg, float scale,
                             float* out, bf16* out_b16, long ldout, int col0, int T, int n);
@@ -613,6 +624,24 @@ cudaError_t relu2_rows(cudaStream_t s, const float* in, long ldi, float* out, bf
 // the same on bf16 rows (tensor-core path)
 cudaError_t relu2_rows_b16(cudaStream_t s, const bf16* in, long ldi, bf16* out, int T, int n);
 
+// ---- residual step of pre-normed stacks with S copies of the stream (stack_streams.cu).  x [rows][S][W]; either the start of a
+//      stack (x0: every copy becomes x0[r]) or the end of a sublayer: y[r] (+ bias), or a mixture's rows sum_k wts[r, k] *
+//      rows[row_of[r, k]] (bf16, in order of k), joins the copies, x_t <- sum_s mix[s][t] x_s + out[t] y (all from the old ones;
+//      mix / out null with S == 1: ones).  Then u = sum_t in[t] x_t (in null: ones), h[r] = u / rms(u) * w (w null: u itself) as
+//      fp32 and / or bf16.  last: nothing reads the copies again, they are not written back.
+constexpr int kMaxStreams = 16;
+struct StreamStep {
+  float* x; const float* x0; const float* y; const void* bias;
+  const void* mix; const void* out; const void* in; const void* w;
+  float* h; bf16* h16;
+  const bf16* rows; const int32_t* row_of; const float* wts; int top_k;
+  int S, W;
+  bool f32, last;
+  float eps;
+};
+cudaError_t stack_streams_init();
+cudaError_t stream_step(cudaStream_t s, const StreamStep& a, int rows);
+
 // ---- gated feed-forward units and mixtures of experts (stack_moe.cu).
 cudaError_t stack_moe_init();
 enum GluAct : int { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED = 2, GLU_NONE_GELU = 3 };  // GLU_NONE_GELU: ungated, gelu_erf(up)
@@ -622,9 +651,9 @@ enum GluAct : int { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED = 2, GLU_NONE_G
 // neighbours, a group scores the sum of its two largest corrected scores and only the `keep` best groups are eligible.
 // The weights are the chosen outputs' uncorrected scores, divided by their sum (+ 1e-20) when renorm, times scale.  bias: the
 // correction row is added to the logits instead of the scores.  chosen: the largest (biased) logits are chosen and the weights
-// are the softmax over the chosen ones.
+// are the softmax over the chosen ones.  group_max: a group scores its largest corrected score.  A null correction row is zeros.
 struct RouteOpts {
-  int sigmoid = 0, groups = 0, keep = 0, renorm = 0, chosen = 0, bias = 0;
+  int sigmoid = 0, groups = 0, keep = 0, renorm = 0, chosen = 0, bias = 0, group_max = 0;
   float scale = 1.f;
 };
 // out[t, j] = act(gu[t, j]) * gu[t, F + j]   (row stride ldg; out may be null when only the bf16 copy is wanted)

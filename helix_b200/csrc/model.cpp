@@ -165,6 +165,40 @@ static size_t carve(Model* m, const hb_model_desc& d, uint8_t* base) {
 }
 
 // ------------------------------------------------------------------ layer-list decoders
+std::string unroll_stack(hb_stack_desc& d, std::vector<hb_layer_desc>& layers, std::vector<int>& id) {
+  const int n = (int)layers.size();
+  id.resize(n);
+  for (int i = 0; i < n; ++i) id[i] = i;
+  const int a = d.loop_start, b = d.loop_stop, times = d.loop_times;
+  if (times < 0) return "negative loop_times";
+  d.loop_start = d.loop_stop = d.loop_times = 0;
+  if (times <= 1) return "";
+  if (a < 0 || b <= a || b > n) return "loop_start .. loop_stop must be a range of layers";
+  if ((long)(b - a) * times > 65536) return "loop unrolls to more than 65536 layer runs";
+  const int extra = (b - a) * (times - 1);  // runs between the first pass and the layers behind the loop
+  // a layer named by another one (its tensors, its cache rows) sits at: its first run; for a cache source inside the loop, read
+  // from inside the loop, the run of the same pass
+  auto first_run = [&](int j) { return j < b ? j : j + extra; };
+  std::vector<hb_layer_desc> out;
+  std::vector<int> oid;
+  auto push = [&](int i, int pass) {
+    hb_layer_desc l = layers[i];
+    if (l.weights_of > 0 && l.weights_of <= n) l.weights_of = first_run(l.weights_of - 1) + 1;
+    else if (pass > 0) l.weights_of = first_run(i) + 1;
+    if (l.kv_from >= 0 && l.kv_from < n) l.kv_from = l.kv_from >= a && l.kv_from < b && i >= a && i < b ? l.kv_from + pass * (b - a) : first_run(l.kv_from);
+    out.push_back(l);
+    oid.push_back(i);
+  };
+  for (int i = 0; i < a; ++i) push(i, 0);
+  for (int p = 0; p < times; ++p)
+    for (int i = a; i < b; ++i) push(i, p);
+  for (int i = b; i < n; ++i) push(i, 0);
+  layers.swap(out);
+  id.swap(oid);
+  d.n_layers = (int)layers.size();
+  return "";
+}
+
 std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
   if (!L) return "no layer list";
   if (d.width <= 0 || d.vocab <= 0 || d.n_layers <= 0) return "non-positive dimension";
@@ -181,7 +215,8 @@ std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
       if (l.mask != HB_MASK_WINDOW && l.mask != HB_MASK_CAUSAL) return "latent attention masks: window or causal" + at;
       if (l.mask == HB_MASK_WINDOW && l.window <= 0) return "window size must be positive" + at;
       if (l.rope_pairing != 0 && l.rope_pairing != 1) return "unknown rope_pairing" + at;
-      if (l.attn_flags & ~(HB_ATTN_NO_SINK | HB_ATTN_HEAD_GATE)) return "unsupported latent attention option" + at;
+      if (l.attn_flags & ~(HB_ATTN_NO_SINK | HB_ATTN_HEAD_GATE | HB_ATTN_NO_GATE)) return "unsupported latent attention option" + at;
+      if ((l.attn_flags & HB_ATTN_HEAD_GATE) && (l.attn_flags & HB_ATTN_NO_GATE)) return "a gate per head and no gate" + at;
       if (l.rope_dims < 0 || l.rope_dims % 2 || l.rope_dims > l.rot_dim) return "rope_dims must be even and <= rot_dim" + at;
       if (l.rope_dims > 0 && !(l.rope_base > 0.f)) return "rope_base must be positive" + at;
       if (latent_attn_smem(l.kv_rank, l.rot_dim, l.mask == HB_MASK_CAUSAL ? 1 << 30 : l.window) > 200 * 1024) return "latent row exceeds the attention kernel's shared memory" + at;
@@ -222,6 +257,11 @@ std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
     } else if (l.mixer == HB_MIXER_MLSTM) {
       if (l.dim > 256) return "matrix-memory key channels per head > 256 unsupported" + at;
       if (!(l.gate_cap > 0.f)) return "gate_cap must be positive" + at;
+    } else if (l.mixer == HB_MIXER_LIGHTNING) {
+      if (l.dim > 256) return "linear-attention key channels per head > 256 unsupported" + at;
+      if (!l.head_decay) return "linear attention needs its decays (head_decay)" + at;
+      for (int h = 0; h < l.heads; ++h)
+        if (!(l.head_decay[h] >= 0.f && l.head_decay[h] <= 1.f)) return "decays must be in 0..1" + at;
     } else {
       return "unknown mixer" + at;
     }
@@ -239,14 +279,21 @@ std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
       if (!(l.side_gate_cap > 0.f)) return "side_gate_cap must be positive" + at;
       if (l.attn_flags & HB_ATTN_HEAD_GATE) return "a second mixer with a per-head gate on the first is unsupported" + at;
     }
+    if (l.mixer == HB_MIXER_LATENT || l.mixer == HB_MIXER_GQA) {
+      if (l.rope_yarn_factor > 0.f && (l.rope_original <= 0 || !(l.rope_yarn_fast > 0.f) || !(l.rope_yarn_slow > 0.f) || !(l.rope_base > 1.f)))
+        return "YaRN scaling needs original, fast, slow > 0 and a base above 1" + at;
+      if (l.rope_yarn_factor > 0.f && (l.rope_factor > 0.f || l.rope_linear > 0.f)) return "two scalings of the rotation" + at;
+    }
     if (l.weights_of < 0 || l.weights_of > d.n_layers || l.weights_of == i + 1) return "weights_of must name another layer" + at;
     if (l.weights_of > 0) {
       hb_layer_desc a = l, b = L[l.weights_of - 1];
       if (b.weights_of > 0) return "weights_of must name a layer with tensors of its own" + at;
       a.weights_of = b.weights_of = 0;
+      if ((a.kv_from >= 0) != (b.kv_from >= 0)) return "a layer that uses another layer's tensors must read cache rows the same way" + at;
+      a.kv_from = b.kv_from = -1;
+      if (a.head_decay && b.head_decay && memcmp(a.head_decay, b.head_decay, (size_t)a.heads * sizeof(float)) == 0) a.head_decay = b.head_decay = nullptr;
       if (memcmp(&a, &b, sizeof a) != 0) return "a layer that uses another layer's tensors must have its description" + at;
       if (l.attn_flags & HB_ATTN_V_BLEND) return "shared tensors with blended values are unsupported" + at;
-      if (l.mixer == HB_MIXER_LATENT) return "shared tensors for latent attention are unsupported" + at;
     }
     if (l.ff < 0) return "negative ff" + at;
     if (l.ff > 0) {
@@ -262,6 +309,7 @@ std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
           if (l.route_keep <= 0 || l.route_keep > l.route_groups) return "groups kept must be 1..groups" + at;
           if (l.route_keep * (R / l.route_groups) < l.top_k) return "the kept groups hold fewer outputs than top_k" + at;
         }
+        if (l.route_plain && l.route_bias) return "router logit biases and no correction tensor" + at;
         if (l.shared_ff < 0) return "negative shared_ff" + at;
       } else if (l.ff_kind != HB_FF_CLAMPED && l.ff_kind != HB_FF_GELU_TANH && l.ff_kind != HB_FF_SILU && l.ff_kind != HB_FF_RELU2) {
         return "unknown feed-forward kind" + at;
@@ -269,8 +317,18 @@ std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* L) {
     }
   }
   if (d.norm_place != HB_NORM_OF_SUM && d.norm_place != HB_NORM_OF_OUTPUT && d.norm_place != HB_NORM_BOTH_SIDES &&
-      d.norm_place != HB_NORM_PARALLEL)
+      d.norm_place != HB_NORM_PARALLEL && d.norm_place != HB_NORM_PRE)
     return "unknown norm_place";
+  if (d.norm_place == HB_NORM_PRE) {
+    if (d.norm_kind != HB_NORM_RMS || !d.plain_gains) return "pre-norms are RMS norms with plain gains";
+    if (d.streams < 0 || d.streams > kMaxStreams) return "more than 16 stream copies unsupported";
+    for (int i = 0; i < d.n_layers; ++i)
+      if (L[i].side_heads > 0) return "pre-norms with a second mixer are unsupported";
+  } else if (d.streams != 0) {
+    return "stream copies need pre-norms";
+  }
+  if (d.bigram_buckets < 0 || (d.bigram_buckets > 0 && (d.bigram_mul_prev < 0 || d.bigram_mul_cur < 0))) return "bigram embedding sizes";
+  if (d.loop_times > 1) return "loop not unrolled";
   if (d.norm_place == HB_NORM_PARALLEL) {
     if (d.norm_kind != HB_NORM_RMS) return "parallel sublayers need RMS norms";
     for (int i = 0; i < d.n_layers; ++i)
@@ -302,6 +360,15 @@ std::vector<double> stack_rope_freqs(const hb_layer_desc& l) {
   for (int i = 0; i < half; ++i) f[i] = pow((double)l.rope_base, -2.0 * i / (double)l.rope_dims);
   if (l.rope_linear > 0.f)
     for (int i = 0; i < half; ++i) f[i] /= (double)l.rope_linear;
+  if (l.rope_yarn_factor > 0.f) {
+    const double base = l.rope_base, dims = l.rope_dims, factor = l.rope_yarn_factor;
+    auto at = [&](double turns) { return dims * log((double)l.rope_original / (2.0 * M_PI * turns)) / (2.0 * log(base)); };
+    const double lo = std::max(floor(at(l.rope_yarn_fast)), 0.0), hi = std::min(ceil(at(l.rope_yarn_slow)), dims - 1.0);
+    for (int i = 0; i < half; ++i) {
+      const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+      f[i] = f[i] / factor * ramp + f[i] * (1.0 - ramp);
+    }
+  }
   if (l.rope_factor > 0.f) {
     const double factor = l.rope_factor, lo = l.rope_low, hi = l.rope_high, orig = l.rope_original;
     for (int i = 0; i < half; ++i) {
@@ -316,6 +383,10 @@ std::vector<double> stack_rope_freqs(const hb_layer_desc& l) {
     }
   }
   return f;
+}
+
+float stack_rope_mult(const hb_layer_desc& l) {
+  return l.rope_yarn_factor > 0.f ? (float)(0.1 * log((double)l.rope_yarn_factor) + 1.0) : 1.f;
 }
 
 static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc* L, uint8_t* base) {
@@ -359,6 +430,11 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
   uint8_t* embed = take(V * W);
   put("embed", embed, 0, V, W);
   uint8_t* embed_norm = d.embed_norm ? norm_block("embed.norm") : nullptr;
+  if (d.bigram_buckets > 0) {
+    uint8_t* bg = take(((size_t)d.bigram_buckets + 1) * W);
+    put("bigram", bg, 0, (size_t)d.bigram_buckets + 1, W);
+    if (m) m->s_bigram = bg;
+  }
   if (m) {
     m->s_embed = embed;
     m->s_embed_norm = embed_norm;
@@ -371,7 +447,7 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
   int planes = 0;
   for (int i = 0; i < d.n_layers; ++i) {
     const hb_layer_desc& l = L[i];
-    const std::string p = "l" + std::to_string(i) + ".";
+    const std::string p = "l" + std::to_string(m && !m->layer_id.empty() ? m->layer_id[i] : i) + ".";
     StackLayerW w;
     const size_t H = l.heads, Dk = l.dim, Dv = l.vdim;
     const bool shared_w = l.weights_of > 0;
@@ -388,6 +464,20 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
         put(p + "ls2", s2, 0, W, 1, true, 1.f);
         w.ls2 = s2;
       }
+    }
+    if (d.norm_place == HB_NORM_PRE && d.streams > 0) {
+      const size_t S = d.streams;
+      auto hyper = [&](const std::string& name, HyperW& hw) {
+        uint8_t* in = take(S);
+        uint8_t* out = take(S);
+        uint8_t* mix = take(S * S);
+        put(name + ".in", in, 0, S, 1, true, 1.f / (float)S);  // random init: the mean of the copies in, every copy gains y
+        put(name + ".out", out, 0, S, 1, true, 1.f);
+        put(name + ".mix", mix, 0, S, S, true, 1.f / (float)S);
+        hw.in = in; hw.out = out; hw.mix = mix;
+      };
+      hyper(p + "hc1", w.hc1);
+      if (l.ff > 0) hyper(p + "hc2", w.hc2);
     }
     // a matrix memory: rows [q | k | v | g | i | f] from row `row0` of the fused projection `in`, gate biases in `bias`
     auto carve_mlstm = [&](const std::string& pm, uint8_t* in, uint8_t* bias, size_t row0, size_t Hm, size_t Dm, size_t Dvm, float cap) {
@@ -458,6 +548,28 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
       uint8_t* o = take(W * H * Dv);
       put(p + "mix.o", o, 0, W, H * Dv);
       w.wo = o; w.o_cols = (int)(H * Dv);
+    } else if (l.mixer == HB_MIXER_LIGHTNING) {
+      w.off_q = 0;
+      w.off_k = (int)(H * Dk);
+      w.off_v = (int)(2 * H * Dk);
+      w.off_g = (int)(2 * H * Dk + H * Dv);
+      w.n_in = (int)(2 * H * Dk + 2 * H * Dv);
+      uint8_t* in = take((size_t)w.n_in * W);
+      w.w_in = in;
+      put(p + "mix.q", in, w.off_q, H * Dk, W);
+      put(p + "mix.k", in, w.off_k, H * Dk, W);
+      put(p + "mix.v", in, w.off_v, H * Dv, W);
+      put(p + "mix.g", in, w.off_g, H * Dv, W);
+      uint8_t* hn = take(H * Dv);
+      uint8_t* o = take(W * H * Dv);
+      put(p + "mix.norm", hn, 0, H * Dv, 1, true, 1.f);
+      put(p + "mix.o", o, 0, W, H * Dv);
+      w.hnorm = hn; w.wo = o;
+      if (m) {
+        w.state_off = m->state_floats;
+        m->state_floats += H * Dk * Dv;
+        m->state_floats = (m->state_floats + 3) & ~size_t(3);
+      }
     } else if (l.mixer == HB_MIXER_DELTA) {
       const size_t G = l.kv_heads, C = 2 * G * Dk + H * Dv, taps = l.conv_taps;
       w.off_q = 0;
@@ -610,7 +722,7 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
       const size_t Q = l.q_rank, R = l.kv_rank, Dr = l.rot_dim;
       const bool own = l.kv_from < 0;
       const size_t q_rows = Q > 0 ? Q : H * (Dk + Dr);  // the query latent, or the queries themselves
-      const size_t g_rows = (l.attn_flags & HB_ATTN_HEAD_GATE) ? H : H * Dv;
+      const size_t g_rows = (l.attn_flags & HB_ATTN_NO_GATE) ? 0 : (l.attn_flags & HB_ATTN_HEAD_GATE) ? H : H * Dv;
       w.off_dq = w.off_q = 0;
       w.off_dkv = own ? (int)q_rows : -1;
       w.off_g = (int)(q_rows + (own ? R + Dr : 0));
@@ -619,7 +731,7 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
       w.w_in = in;
       put(p + (Q > 0 ? "mix.dq" : "mix.q"), in, 0, q_rows, W);
       if (own) put(p + "mix.dkv", in, q_rows, R + Dr, W);
-      put(p + "mix.g", in, w.off_g, g_rows, W);
+      if (g_rows) put(p + "mix.g", in, w.off_g, g_rows, W);
       uint8_t* dqn = Q > 0 ? take(Q) : nullptr;
       uint8_t* uq = Q > 0 ? take(H * (Dk + Dr) * Q) : nullptr;
       uint8_t* dkvn = own ? take(R) : nullptr;
@@ -654,11 +766,11 @@ static size_t carve_stack(Model* m, const hb_stack_desc& d, const hb_layer_desc*
       uint8_t* n2 = d.one_norm ? nullptr : norm_block(p + "norm2");
       if (both) w.norm2b = norm_block(p + "norm2b");
       uint8_t* router = take(std::max<size_t>(R, 64) * W);  // at least one MMA tile of rows; the arena is zeroed at load
-      uint8_t* corr = take(R);
+      uint8_t* corr = l.route_plain ? nullptr : take(R);
       uint8_t* gu = take(E * (gated ? 2 : 1) * Fn * W);
       uint8_t* dn = take(E * W * Fn);
       put(p + "mlp.router", router, 0, R, W);
-      put(p + (l.route_bias ? "mlp.router.b" : "mlp.correction"), corr, 0, R, 1, false, 1.f, true);
+      if (!l.route_plain) put(p + (l.route_bias ? "mlp.router.b" : "mlp.correction"), corr, 0, R, 1, false, 1.f, true);
       if (l.shared_ff > 0) {
         const size_t Fs = l.shared_ff;
         uint8_t* sg = take(2 * Fs * W);

@@ -37,6 +37,11 @@ struct MlstmW {
   size_t state_off = 0, n_off = 0, m_off = 0;
 };
 
+// How one sublayer reads and writes S copies of the residual stream: in [S], out [S], mix [S][S] (from, to), weight type
+struct HyperW {
+  void *in = nullptr, *out = nullptr, *mix = nullptr;
+};
+
 struct StackLayerW {
   void *norm1 = nullptr, *norm2 = nullptr;
   void *norm1b = nullptr, *norm2b = nullptr;  // HB_NORM_BOTH_SIDES: the norms of the sublayers' outputs (norm1 / norm2: of their inputs)
@@ -59,6 +64,9 @@ struct StackLayerW {
   // [A_log (heads) | dt_bias (heads) | D (heads)]; hnorm [heads vdim]; state_off: S [heads][dim][vdim], tail_off: the convolution's
   // last inputs.  GQA with convolved projections: conv_w [q | k | v channels][taps], tail_off.
   void* conv_b = nullptr;
+  // LIGHTNING: rows [q | k | v | g] of w_in; hnorm [heads vdim]; state_off: S [heads][dim][vdim]; decay [heads] fp32 (device)
+  const float* decay = nullptr;
+  HyperW hc1, hc2;           // HB_NORM_PRE with stream copies: weights of the mixer's and the feed-forward's read and write
   MlstmW ml;                 // MLSTM as the only mixer, or the second mixer of the layer
   void* o_bias = nullptr;    // GQA: bias of the output projection [width]
   int o_cols = 0;            // columns of wo: the first mixer's heads * vdim (+ the second's, stored behind them in every row)
@@ -104,6 +112,9 @@ struct Model {
   hb_stack_desc sd{};
   std::vector<hb_layer_desc> sl;
   std::vector<StackLayerW> sw;
+  std::vector<int> layer_id;                   // layer run -> index of the layer its tensors are named after
+  std::vector<std::vector<float>> head_decay;  // layer run -> constant decays (LIGHTNING)
+  void* s_bigram = nullptr;
   void *s_embed = nullptr, *s_embed_norm = nullptr, *s_final_norm = nullptr, *s_head = nullptr;
   size_t state_floats = 0;              // fp32 state of one sequence over all GLA layers
   std::vector<int> plane_row;           // cache pool planes: elements per cached position (kv_rank + rot_dim; kv_heads * dim)
@@ -118,6 +129,9 @@ struct Model {
 std::string validate_desc(const hb_model_desc& d);
 // Layer-list decoders: validation, arena size, layout (fills m.sw, m.placements, m.state_floats, m.plane_row).
 std::string validate_stack(const hb_stack_desc& d, const hb_layer_desc* layers);
+// The layers in the order they run: the loop of `d` unrolled (later passes use the first one's tensors), d.n_layers = runs and no
+// loop left in d.  id[run] = the layer's index in the description.  Returns "" or why the loop is not possible.
+std::string unroll_stack(hb_stack_desc& d, std::vector<hb_layer_desc>& layers, std::vector<int>& id);
 size_t arena_bytes_for_stack(const hb_stack_desc& d, const hb_layer_desc* layers);
 void layout_stack(Model& m);
 // Arena size in bytes for a description (also used by hb_memory_estimate).
@@ -129,5 +143,7 @@ std::vector<float> rope_inv_freq(const hb_model_desc& d);
 // Rotation frequencies of a layer-list attention layer: base^(-2i/dims), i < dims/2, with the wavelength-dependent scaling
 // of hb_layer_desc (rope_factor <= 0: none), in double precision.
 std::vector<double> stack_rope_freqs(const hb_layer_desc& l);
+// ... and the factor of cos and sin that goes with them (YaRN scaling; 1 otherwise)
+float stack_rope_mult(const hb_layer_desc& l);
 
 }  // namespace hb

@@ -631,7 +631,7 @@ __global__ void head_gate_kernel(const bf16* __restrict__ o, long ldo, const flo
 }
 
 __global__ void rope_table_kernel(const int32_t* __restrict__ positions, const double* __restrict__ freqs, int half,
-                                  float* __restrict__ cs, int T) {
+                                  float* __restrict__ cs, int T, float mult) {
   const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (long)T * half) return;
   const int t = (int)(idx / half), i = (int)(idx % half);
@@ -639,14 +639,14 @@ __global__ void rope_table_kernel(const int32_t* __restrict__ positions, const d
   const double red = fma(-6.283185307179586476925, rint(ang * 0.15915494309189533577), ang);
   float s, c;
   sincosf((float)red, &s, &c);
-  *reinterpret_cast<float2*>(cs + 2 * idx) = make_float2(c, s);
+  *reinterpret_cast<float2*>(cs + 2 * idx) = make_float2(c * mult, s * mult);
 }
 
 }  // namespace
 
-cudaError_t stack_rope_table(cudaStream_t s, const int32_t* positions, const double* freqs, int half, float* cs, int T) {
+cudaError_t stack_rope_table(cudaStream_t s, const int32_t* positions, const double* freqs, int half, float* cs, int T, float mult) {
   if (T <= 0 || half <= 0) return cudaSuccess;
-  rope_table_kernel<<<(unsigned)(((long)T * half + 255) / 256), 256, 0, s>>>(positions, freqs, half, cs, T);
+  rope_table_kernel<<<(unsigned)(((long)T * half + 255) / 256), 256, 0, s>>>(positions, freqs, half, cs, T, mult);
   return cudaGetLastError();
 }
 

@@ -74,18 +74,18 @@ __device__ __forceinline__ void route_one(const float* zr, const WT* __restrict_
     if (ro.chosen) return zr[i] + (ro.bias ? ldf<WT>(corr, i) : 0.f);
     return ro.sigmoid ? sigmoidf_(zr[i]) : expf(zr[i] - mx) * inv;
   };
-  for (int i = l; i < R; i += 32) pick[i] = ro.bias ? score(i) : score(i) + ldf<WT>(corr, i);
+  for (int i = l; i < R; i += 32) pick[i] = ro.bias || !corr ? score(i) : score(i) + ldf<WT>(corr, i);
   __syncwarp();
   if (ro.groups > 1 && ro.keep < ro.groups) {
     float* gs = pick + R;
     const int per = R / ro.groups;
-    for (int g = l; g < ro.groups; g += 32) {  // a group scores the sum of its two largest choice scores
+    for (int g = l; g < ro.groups; g += 32) {  // a group scores the sum of its two largest choice scores, or its largest
       float a = -INFINITY, b = -INFINITY;
       for (int i = g * per; i < (g + 1) * per; ++i) {
         const float v = pick[i];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      gs[g] = per > 1 ? a + b : a;
+      gs[g] = per > 1 && !ro.group_max ? a + b : a;
     }
     __syncwarp();
     for (int k = 0; k < ro.keep; ++k) {  // the kept groups are marked with -inf (a real score is finite)

@@ -66,11 +66,18 @@ __global__ void __launch_bounds__(256) gemm_rt_kernel(const float* __restrict__ 
 // ------------------------------------------------------------------ row kernels
 template <typename WT>
 __global__ void embed_rows_kernel(const int32_t* __restrict__ tokens, const WT* __restrict__ table, float* __restrict__ x,
-                                  bf16* __restrict__ xb, int W, float scale) {
+                                  bf16* __restrict__ xb, int W, float scale, BigramArgs bg) {
   const int t = blockIdx.x;
   const WT* src = table + (size_t)tokens[t] * W;
+  const WT* pair = nullptr;
+  if (bg.table) {
+    const int prev = bg.prev[t];
+    const long long row = prev < 0 ? bg.buckets : ((long long)prev * bg.mul_prev + (long long)tokens[t] * bg.mul_cur) % bg.buckets;
+    pair = (const WT*)bg.table + (size_t)row * W;
+  }
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < W; i += gridDim.y * blockDim.x) {
-    const float v = ldf<WT>(src, i) * scale;
+    float v = ldf<WT>(src, i) * scale;
+    if (pair) v += ldf<WT>(pair, i);
     x[(size_t)t * W + i] = v;
     if (xb) xb[(size_t)t * W + i] = __float2bfloat16(v);
   }
@@ -268,7 +275,7 @@ __global__ void latent_gate_kernel(const float* __restrict__ o, long o_ts, long 
   if (j >= N) return;
   const int h = j / Dv, i = j - h * Dv;
   const float* src = o + (size_t)t * o_ts + (size_t)h * o_hs + i;
-  const float* gs = g + (size_t)t * ldg + (per_head ? h : j);
+  const float* gs = g ? g + (size_t)t * ldg + (per_head ? h : j) : nullptr;
   float v[VEC];
   if (VEC == 4) {
     const float4 x = *reinterpret_cast<const float4*>(src);
@@ -277,7 +284,8 @@ __global__ void latent_gate_kernel(const float* __restrict__ o, long o_ts, long 
     v[0] = src[0];
   }
 #pragma unroll
-  for (int e = 0; e < VEC; ++e) v[e] *= sigmoidf_(gs[per_head ? 0 : e]);
+  for (int e = 0; e < VEC; ++e)
+    if (gs) v[e] *= sigmoidf_(gs[per_head ? 0 : e]);
   if (VEC == 4) {
     if (out) *reinterpret_cast<float4*>(out + (size_t)t * N + j) = make_float4(v[0], v[1 % VEC], v[2 % VEC], v[VEC - 1]);
     if (outb) {
@@ -902,11 +910,12 @@ cudaError_t tanh_norm_step(cudaStream_t s, const float* x, const int32_t* row_in
   return cudaGetLastError();
 }
 
-cudaError_t embed_rows_f32(cudaStream_t s, const int32_t* tokens, const void* table, bool f32, float* x, bf16* xb, int T, int W, float scale) {
+cudaError_t embed_rows_f32(cudaStream_t s, const int32_t* tokens, const void* table, bool f32, float* x, bf16* xb, int T, int W, float scale,
+                           const BigramArgs& bg) {
   if (T <= 0) return cudaSuccess;
   const dim3 grid(T, T <= 256 ? (W + 127) / 128 : 1);
-  if (f32) embed_rows_kernel<float><<<grid, 128, 0, s>>>(tokens, (const float*)table, x, xb, W, scale);
-  else embed_rows_kernel<bf16><<<grid, 128, 0, s>>>(tokens, (const bf16*)table, x, xb, W, scale);
+  if (f32) embed_rows_kernel<float><<<grid, 128, 0, s>>>(tokens, (const float*)table, x, xb, W, scale, bg);
+  else embed_rows_kernel<bf16><<<grid, 128, 0, s>>>(tokens, (const bf16*)table, x, xb, W, scale, bg);
   return KERR();
 }
 

@@ -235,6 +235,8 @@ __global__ void __launch_bounds__(DKP * 2, 512 / DKP) lin_recurrence_kernel(LinR
   float* slot = a.state + (size_t)a.slots[b] * a.slot_stride;
   float* st = slot + a.s_off + (size_t)h * Dk * a.Dv;
   const bool fresh = a.first_pos[b] == 0;
+  const bool hd = a.head_decay != nullptr;
+  const float2 hab = make_float2(hd ? a.head_decay[h] : 0.f, 1.f);
   const bool do_n = a.nq != nullptr && blockIdx.z == 0;
   const int nch = i0 + (lane & 15);
   float* nst = slot + a.n_off + (size_t)h * Dk + nch;
@@ -275,6 +277,7 @@ __global__ void __launch_bounds__(DKP * 2, 512 / DKP) lin_recurrence_kernel(LinR
         for (int e = 0; e < NC; ++e)
           if (c0 + lane + 32 * e < a.Dv) cpa4(dst + 2 * DKP + lane + 32 * e, sv + lane + 32 * e);
       }
+      if (hd) continue;
       if (lane == 8 * NC) cpa4(dst + 2 * DKP + BC, a.ab + row * a.ldab + h);
       if (lane == 8 * NC + 1) cpa4(dst + 2 * DKP + BC + 1, a.ab + row * a.ldab + a.H + h);
     }
@@ -293,9 +296,18 @@ __global__ void __launch_bounds__(DKP * 2, 512 / DKP) lin_recurrence_kernel(LinR
     }
     __syncthreads();
     const float* base = sm + stage * stage_floats;
+    if (a.silu) {  // activations of the staged q | k | v, once per stage
+      float* raw = sm + stage * stage_floats;
+      for (int e = threadIdx.x; e < nt * (2 * DKP + BC); e += blockDim.x) {
+        const int at = e / (2 * DKP + BC) * per_tok + e % (2 * DKP + BC);
+        const float z = raw[at];
+        raw[at] = z * sigmoidf_(z);
+      }
+      __syncthreads();
+    }
     for (int tt = 0; tt < nt; ++tt) {
       const float* tk = base + tt * per_tok;
-      const float2 dab = *reinterpret_cast<const float2*>(tk + 2 * DKP + BC);
+      const float2 dab = hd ? hab : *reinterpret_cast<const float2*>(tk + 2 * DKP + BC);
       const float da = dab.x, db = dab.y;
       const float2 da2 = make_float2(da, da);
       float2 bv2[NC], oa[NC];
@@ -401,7 +413,7 @@ __global__ void memory_readout_kernel(const float* __restrict__ num, long ldnum,
 template <typename WT>
 __global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* __restrict__ y, long ldy, const float* __restrict__ z, long ldz,
                                                                const WT* __restrict__ w, float eps, int parts, float* __restrict__ out,
-                                                               bf16* __restrict__ outb, int n) {
+                                                               bf16* __restrict__ outb, int n, int gate_last) {
   __shared__ float red[32];
   const int t = blockIdx.y, part = blockIdx.x, len = n / parts, c0 = part * len;
   const float* ys = y + (size_t)t * ldy + c0;
@@ -415,12 +427,12 @@ __global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* __re
     keep[r] = 0.f;
     if (i < len) {
       const float zv = zs[i];
-      keep[r] = ys[i] * (zv * sigmoidf_(zv));
+      keep[r] = gate_last ? ys[i] : ys[i] * (zv * sigmoidf_(zv));
     }
     ss = fmaf(keep[r], keep[r], ss);
   }
   for (int i = threadIdx.x + kKeep * 256; i < len; i += blockDim.x) {
-    const float zv = zs[i], u = ys[i] * (zv * sigmoidf_(zv));
+    const float zv = zs[i], u = gate_last ? ys[i] : ys[i] * (zv * sigmoidf_(zv));
     ss = fmaf(u, u, ss);
   }
   ss = block_sum(ss, red);
@@ -429,14 +441,14 @@ __global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* __re
   for (int r = 0; r < kKeep; ++r) {
     const int i = threadIdx.x + r * 256;
     if (i >= len) break;
-    const float v = keep[r] * rs * ldf<WT>(w, c0 + i);
+    const float v = keep[r] * rs * ldf<WT>(w, c0 + i) * (gate_last ? sigmoidf_(zs[i]) : 1.f);
     const size_t d = (size_t)t * n + c0 + i;
     if (out) out[d] = v;
     if (outb) outb[d] = __float2bfloat16(v);
   }
   for (int i = threadIdx.x + kKeep * 256; i < len; i += blockDim.x) {
-    const float zv = zs[i], u = ys[i] * (zv * sigmoidf_(zv));
-    const float v = u * rs * ldf<WT>(w, c0 + i);
+    const float zv = zs[i], sg = sigmoidf_(zv), u = gate_last ? ys[i] : ys[i] * (zv * sg);
+    const float v = u * rs * ldf<WT>(w, c0 + i) * (gate_last ? sg : 1.f);
     const size_t d = (size_t)t * n + c0 + i;
     if (out) out[d] = v;
     if (outb) outb[d] = __float2bfloat16(v);
@@ -686,12 +698,12 @@ cudaError_t memory_readout(cudaStream_t s, const float* num, long ldnum, const f
 }
 
 cudaError_t gated_group_norm(cudaStream_t s, const float* y, long ldy, const float* z, long ldz, const void* w, bool f32, float eps, int parts,
-                             float* out, bf16* outb, int T, int n) {
+                             float* out, bf16* outb, int T, int n, bool gate_last) {
   if (T <= 0) return cudaSuccess;
   if (parts < 1 || n % parts) return cudaErrorInvalidValue;
   dim3 grid(parts, T);
-  if (f32) gated_group_norm_kernel<float><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const float*)w, eps, parts, out, outb, n);
-  else gated_group_norm_kernel<bf16><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const bf16*)w, eps, parts, out, outb, n);
+  if (f32) gated_group_norm_kernel<float><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const float*)w, eps, parts, out, outb, n, gate_last);
+  else gated_group_norm_kernel<bf16><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const bf16*)w, eps, parts, out, outb, n, gate_last);
   return cudaGetLastError();
 }
 

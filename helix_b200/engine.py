@@ -81,15 +81,16 @@ MIXER_GQA = 2
 MIXER_DELTA = 3
 MIXER_MAMBA2 = 4
 MIXER_MLSTM = 5
+MIXER_LIGHTNING = 6
 MASK_WINDOW, MASK_CHUNK, MASK_CAUSAL = 0, 1, 2
 FF_CLAMPED, FF_GELU_TANH, FF_MOE, FF_SILU, FF_RELU2 = 0, 1, 2, 3, 4
-NORM_OF_SUM, NORM_OF_OUTPUT, NORM_BOTH_SIDES, NORM_PARALLEL = 0, 1, 2, 3
+NORM_OF_SUM, NORM_OF_OUTPUT, NORM_BOTH_SIDES, NORM_PARALLEL, NORM_PRE = 0, 1, 2, 3, 4
 NORM_RMS, NORM_TANH = 0, 1
 ROUTER_SOFTMAX, ROUTER_SIGMOID, ROUTER_CHOSEN = 0, 1, 2
 EXPERT_SILU, EXPERT_CLAMPED, EXPERT_GELU = 0, 1, 2
 ATTN_QK_UNIT_NORM, ATTN_V_IS_K, ATTN_UNIT_SINK, ATTN_HEAD_GATE = 1, 2, 4, 8
 ATTN_QKV_BIAS, ATTN_QK_PROJ_NORM, ATTN_LEARNED_SINK, ATTN_V_BLEND = 16, 32, 64, 128
-ATTN_QKV_CONV, ATTN_OUT_GATE, ATTN_OUT_BIAS, ATTN_NO_SINK = 256, 512, 1024, 2048
+ATTN_QKV_CONV, ATTN_OUT_GATE, ATTN_OUT_BIAS, ATTN_NO_SINK, ATTN_NO_GATE = 256, 512, 1024, 2048, 4096
 
 
 @dataclass
@@ -145,8 +146,16 @@ class LayerDesc:
     mix_scale: float = 0.0     # weights of the two mixers' outputs; 0 = 1
     side_scale: float = 0.0
     route_bias: int = 0        # FF_MOE: 1: mlp.router.b joins the logits (no correction tensor)
+    route_group_max: int = 0   # FF_MOE: 1: a group scores its largest score, 0: the sum of its two largest
+    route_plain: int = 0       # FF_MOE: 1: no correction tensor
+    rope_yarn_factor: float = 0.0  # <= 0: no YaRN scaling of the rotation; original length: rope_original
+    rope_yarn_fast: float = 32.0
+    rope_yarn_slow: float = 1.0
+    head_decay: tuple = ()     # LIGHTNING: one constant decay per head
 
     def to_c(self):
+        # (the structure keeps the decay array alive; so does an array of structures built from it)
+        decay = (C.c_float * len(self.head_decay))(*self.head_decay) if len(self.head_decay) else None
         return LayerDescC(self.mixer, self.heads, self.dim, self.vdim, self.tau, self.decay_rank, self.q_rank, self.kv_rank,
                           self.rot_dim, self.rope_dims, self.window, self.kv_from, self.rope_base, self.scale, self.ff, self.ff_limit,
                           self.kv_heads, self.mask, self.attn_flags, self.rope_pairing, self.rope_factor, self.rope_low,
@@ -154,7 +163,9 @@ class LayerDesc:
                           self.score_cap, self.conv_taps, self.router_kind, self.route_groups, self.route_keep, self.route_renorm,
                           self.route_scale, self.expert_kind, self.shared_ff, self.shared_limit, self.weights_of, self.rope_linear,
                           self.norm_groups, self.gate_cap, self.side_mixer, self.side_heads, self.side_dim, self.side_vdim,
-                          self.side_gate_cap, self.mix_scale, self.side_scale, self.route_bias)
+                          self.side_gate_cap, self.mix_scale, self.side_scale, self.route_bias, self.route_group_max,
+                          self.route_plain, self.rope_yarn_factor, self.rope_yarn_fast, self.rope_yarn_slow,
+                          head_decay=C.cast(decay, C.POINTER(C.c_float)) if decay else None)
 
 
 @dataclass
@@ -177,6 +188,13 @@ class StackDesc:
     one_norm: int = 0          # NORM_PARALLEL: both sublayers read norm1(x)
     layer_scale: int = 0       # NORM_PARALLEL: per-entry gains ls1 / ls2 on the sublayers' outputs
     resid_mult: float = 0.0    # NORM_PARALLEL: factor of the sublayers' sum; 0 = 1
+    streams: int = 0           # NORM_PRE: copies of the residual stream; 0: one stream without read / write weights
+    bigram_buckets: int = 0    # 0: no bigram embedding
+    bigram_mul_prev: int = 0
+    bigram_mul_cur: int = 0
+    loop_start: int = 0        # layers loop_start .. loop_stop - 1 run loop_times times in a row (<= 1: no loop)
+    loop_stop: int = 0
+    loop_times: int = 0
     arch: int = 2
     unused_tensors: frozenset = frozenset()  # checkpoint tensors the design names but this stack has no use for (skipped at load)
 
@@ -192,7 +210,8 @@ class StackDesc:
         arr = (LayerDescC * len(self.layers))(*[l.to_c() for l in self.layers])
         return StackDescC(self.width, self.vocab, len(self.layers), self.compute_f32, self.norm_eps, self.resid_alpha,
                           self.logit_softcap, self.norm_place, self.embed_norm, self.plain_gains, self.norm_kind, self.embed_scale,
-                          self.logit_scale, self.tie_head, self.one_norm, self.layer_scale, self.resid_mult), arr
+                          self.logit_scale, self.tie_head, self.one_norm, self.layer_scale, self.resid_mult, self.streams, self.bigram_buckets,
+                          self.bigram_mul_prev, self.bigram_mul_cur, self.loop_start, self.loop_stop, self.loop_times), arr
 
 
 @dataclass

@@ -12,7 +12,7 @@ import struct
 import numpy as np
 
 from . import engine as _e
-from .engine import LayerDesc, ModelDesc, StackDesc, bf16_bits, MIXER_GLA, MIXER_LATENT, MIXER_GQA, MIXER_DELTA, MIXER_MAMBA2, MIXER_MLSTM
+from .engine import LayerDesc, ModelDesc, StackDesc, bf16_bits, MIXER_GLA, MIXER_LATENT, MIXER_GQA, MIXER_DELTA, MIXER_MAMBA2, MIXER_MLSTM, MIXER_LIGHTNING
 
 _DT = {"BF16": (np.uint16, 2), "F16": (np.float16, 2), "F32": (np.float32, 4)}
 _IGNORED = ("pooler.", "embeddings.position_ids", "rotary_emb.inv_freq", "cls.", "visual.")  # visual.: the VL tower (not served)
@@ -318,9 +318,90 @@ def kamivik_desc(cfg, shapes=None, compute_f32=False):
                      plain_gains=1, one_norm=1, layer_scale=1, resid_mult=mult)
 
 
+def pupalix_desc(cfg, shapes=None, compute_f32=False):
+    """config.json of a Pupalix checkpoint -> StackDesc: a scaled embedding (also the output matrix) plus rows picked by token
+    pairs, several copies of the stream with learned read / write weights per sublayer, pre-norms; latent attention (directly
+    projected queries, interleaved YaRN-scaled rotation, ordinary softmax, no gate), grouped-query attention inside blocks of
+    positions (values = keys, whole-projection q / k norm, capped scores, no rotation) and linear attention with constant decays;
+    tanh-GELU units or mixtures of SiLU experts (softmax scores, groups ranked by their largest, not renormalised); a run of
+    layers that is passed through several times.  Every size and every constant that may differ between checkpoints comes from
+    the configuration."""
+    def nonzero(v, what):
+        if v == 0.0:
+            raise ValueError(f"{what} of zero is not representable (0 means 1)")
+        return v
+
+    layers = []
+    for i, ly in enumerate(cfg["layers"]):
+        m = ly["mixer"]
+        d = LayerDesc(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]))
+        if ly["type"] == "latent_attention":
+            d.mixer, d.mask, d.attn_flags, d.rope_pairing = MIXER_LATENT, _e.MASK_CAUSAL, _e.ATTN_NO_SINK | _e.ATTN_NO_GATE, 1
+            d.kv_rank, d.rot_dim, d.scale = int(m["kv_rank"]), int(m["rot_dim"]), float(m["scale"])
+            rot = m.get("rot")
+            if rot and rot.get("dims"):
+                d.rope_dims, d.rope_base = int(rot["dims"]), float(rot["base"])
+                sc = rot.get("scaling")
+                if sc:
+                    d.rope_yarn_factor, d.rope_original = float(sc["factor"]), int(sc["original"])
+                    d.rope_yarn_fast, d.rope_yarn_slow = float(sc["fast"]), float(sc["slow"])
+        elif ly["type"] == "attention":
+            d.mixer, d.kv_heads, d.scale = MIXER_GQA, int(m["kv_heads"]), float(m["scale"])
+            d.attn_flags = _e.ATTN_V_IS_K | _e.ATTN_QK_PROJ_NORM
+            d.score_cap = float(m.get("softcap") or 0.0)
+            mask = m.get("mask")
+            if mask and mask.get("size"):
+                d.mask, d.window = _e.MASK_CHUNK, int(mask["size"])
+            else:
+                d.mask, d.window = _e.MASK_CAUSAL, 0
+        elif ly["type"] == "lightning":
+            d.mixer = MIXER_LIGHTNING
+            decay = m["decay"]
+            d.head_decay = tuple(float(a) for a in (decay if isinstance(decay, (list, tuple)) else [decay] * d.heads))
+            if len(d.head_decay) != d.heads:
+                raise ValueError(f"layer {i}: one decay per head")
+        else:
+            raise ValueError(f"layer {i}: unknown layer type {ly['type']!r}")
+        mlp = ly.get("mlp")
+        if mlp is not None:
+            kind = mlp.get("kind")
+            if kind == "dense":
+                d.ff_kind, d.ff = _e.FF_GELU_TANH, int(mlp["ff"])
+            elif kind == "moe":
+                r = mlp["router"]
+                d.ff_kind, d.ff, d.experts, d.top_k = _e.FF_MOE, int(mlp["expert"]["ff"]), int(r["experts"]), int(r["top"])
+                d.router_kind, d.expert_kind, d.route_plain = _e.ROUTER_SOFTMAX, _e.EXPERT_SILU, 1
+                g = r.get("groups")
+                if g:
+                    d.route_groups, d.route_keep, d.route_group_max = int(g["count"]), int(g["keep"]), 1
+            else:
+                raise ValueError(f"layer {i}: unsupported feed-forward kind {kind!r}")
+        layers.append(d)
+    # a checkpoint may carry the norm and the stream weights of a feed-forward that a layer does not have
+    unused = frozenset(f"l{i}.{n}" for i, d in enumerate(layers) if d.ff == 0 for n in ("norm2", "hc2.in", "hc2.out", "hc2.mix"))
+    streams = int(cfg.get("streams") or 0)
+    if streams == 1 and shapes is not None and not any(".hc1." in n for n in shapes):
+        streams = 0  # one plain residual stream
+    emb = cfg.get("embedding") or {}
+    out = StackDesc(unused_tensors=unused, width=int(cfg["width"]), vocab=int(cfg["vocab"]), layers=layers, compute_f32=int(bool(compute_f32)),
+                    norm_eps=float(cfg["norm"]["eps"]), resid_alpha=1.0, norm_place=_e.NORM_PRE, plain_gains=1, tie_head=1, streams=streams,
+                    embed_scale=nonzero(float(emb.get("scale", 1.0)), "an embedding scale"),
+                    logit_scale=nonzero(float(cfg.get("logit_scale", 1.0)), "a logit scale"), logit_softcap=float(cfg.get("logit_softcap") or 0.0))
+    big = emb.get("bigram")
+    if big:
+        out.bigram_buckets = int(big["buckets"])  # the row is a sum modulo the buckets, so the multipliers may be reduced first
+        out.bigram_mul_prev, out.bigram_mul_cur = int(big["mul_prev"]) % out.bigram_buckets, int(big["mul_cur"]) % out.bigram_buckets
+    loop = cfg.get("loop")
+    if loop:
+        out.loop_start, out.loop_stop, out.loop_times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+        if out.loop_times < 1:
+            raise ValueError("a loop runs at least once")
+    return out
+
+
 # layer-list decoders by config.json "architecture"
 STACK_READERS = {"Risepel": risepel_desc, "Lurepel": lurepel_desc, "Latanex": latanex_desc, "Funudra": funudra_desc,
-                 "Kamivik": kamivik_desc}
+                 "Kamivik": kamivik_desc, "Pupalix": pupalix_desc}
 
 
 def desc_from_hf_config(cfg, shapes=None, compute_f32=False):

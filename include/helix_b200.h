@@ -46,7 +46,7 @@
 extern "C" {
 #endif
 
-#define HB_ABI_VERSION 7
+#define HB_ABI_VERSION 8
 
 typedef enum hb_status {
   HB_OK = 0,
@@ -129,7 +129,8 @@ typedef struct hb_model_desc {
  *                         Options: q_rank == 0: queries are projected straight from the layer input (mix.q, no query latent);
  *                         mask HB_MASK_CAUSAL: every earlier position is seen; rope_pairing; attn_flags HB_ATTN_NO_SINK (an
  *                         ordinary softmax, no mix.sink) and HB_ATTN_HEAD_GATE (mix.g has one row per head, head h's output
- *                         times sigmoid of row h, instead of one row per output entry).
+ *                         times sigmoid of row h, instead of one row per output entry) or HB_ATTN_NO_GATE (no gate, no mix.g);
+ *                         rope_yarn_factor > 0 (frequencies interpolated per dimension, cos and sin scaled).
  *        HB_MIXER_GQA     grouped-query attention over cached per-head keys and values (kv_heads of them; query head h reads
  *                         head h / (heads / kv_heads)).  rope_dims leading entries of q and k rotate (rope_pairing, optional
  *                         wavelength-dependent frequency scaling rope_factor / rope_low / rope_high / rope_original); the
@@ -162,6 +163,10 @@ typedef struct hb_model_desc {
  *                         S <- exp(f + m - m') S + exp(i - m') k v^T, n likewise with k alone;
  *                         o = S^T q / (max(|n . q|, exp(-m')) + 1e-6); per-head unit RMS, gain mix.norm over all heads'
  *                         entries, sigmoid(mix.g x), mix.o.  State slot: S [heads][dim][vdim], n [heads][dim], m [heads].
+ *        HB_MIXER_LIGHTNING linear attention with one constant decay per head (head_decay): q = silu(mix.q x), k = silu(mix.k x)
+ *                         (heads x dim), v = silu(mix.v x) (heads x vdim), S <- decay_h S + k v^T, o = S^T q; the concatenated
+ *                         heads divided by their root mean square, times mix.norm (heads * vdim entries) and
+ *                         sigmoid(mix.g x), then mix.o.  State slot: S [heads][dim][vdim].
  *      side_heads > 0: a second mixer of kind side_mixer (HB_MIXER_MLSTM; side_heads / side_dim / side_vdim / side_gate_cap)
  *      reads the same input beside the first; the layer's mixer output is mix_scale * first + side_scale * second (0 = 1).
  *      The first mixer's tensors are then mix.left.*, the second's mix.right.*.
@@ -171,12 +176,17 @@ typedef struct hb_model_desc {
  *      HB_ATTN_OUT_BIAS (mix.o.b), rope_linear > 0 (every rotation frequency divided by it).
  *      weights_of = j + 1 > 0: the layer has no tensors of its own and uses those of layer j (another layer of equal
  *      description that has its own); its cache planes and its part of the state slot are its own.
+ *      Loop (hb_stack_desc.loop_times > 1): layers loop_start .. loop_stop - 1 are run loop_times times in a row with the same
+ *      tensors, then the rest; every pass has cache planes and a part of the state slot of its own.
  *      Residual step (hb_stack_desc.norm_place): HB_NORM_OF_SUM x <- norm(alpha x + f(x)), HB_NORM_OF_OUTPUT
  *      x <- x + norm(f(x)), HB_NORM_BOTH_SIDES x <- x + norm_b(f(norm_a(x))) (norm1 / norm1b around the mixer, norm2 /
  *      norm2b around the feed-forward), or HB_NORM_PARALLEL x <- x + mixer(norm1(x)) + ff(norm2(x)): both sublayers read
  *      the same x (RMS norms; HB_FF_RELU2, the gated units and mixtures of experts); with one_norm both read norm1(x) and there
  *      is no norm2.  layer_scale: the mixer's output is multiplied entry by entry by ls1, the feed-forward's by ls2, and
- *      resid_mult (0 = 1) multiplies their sum (HB_NORM_PARALLEL).  norm_kind: HB_NORM_RMS, or HB_NORM_TANH = tanh(alpha x) * w + b with a scalar
+ *      resid_mult (0 = 1) multiplies their sum (HB_NORM_PARALLEL).  HB_NORM_PRE: x <- x + mixer(norm1(x)), x <- x + ff(norm2(x))
+ *      (RMS norms); with streams = S > 0 there are S copies x_1 .. x_S of the stream (all equal to the embedding at the start,
+ *      their sum at the end) and sublayer q (1: mixer, 2: feed-forward) reads u = sum_s in[s] x_s, y = f(norm_q(u)), and
+ *      leaves x_t <- sum_s mix[s][t] x_s + out[t] y, with l<i>.hc<q>.{in,out,mix}.  norm_kind: HB_NORM_RMS, or HB_NORM_TANH = tanh(alpha x) * w + b with a scalar
  *      alpha and a vector b stored beside the gain as <name>.alpha and <name>.b (no statistic of the row; eps unused).
  *      f = mixer and, when ff > 0, the feed-forward (ff_kind):
  *        HB_FF_CLAMPED    g = min(gate, limit), u = clamp(up, +-limit), y = down(g sigmoid(1.702 g) (u + 1)), with biases
@@ -187,7 +197,8 @@ typedef struct hb_model_desc {
  *                         Options: router_kind HB_ROUTER_SIGMOID (scores = sigmoid of the logits); route_groups > 1: the
  *                         experts form that many equal groups of neighbours, a group scores the sum of its two largest
  *                         corrected scores and only experts of the route_keep best groups can be chosen; route_renorm: the
- *                         chosen scores are divided by their sum (+ 1e-20); route_scale (0 = 1) multiplies the weights;
+ *                         chosen scores are divided by their sum (+ 1e-20); route_group_max: a group scores its largest
+ *                         score instead; route_plain: there is no correction tensor; route_scale (0 = 1) multiplies the weights;
  *                         expert_kind HB_EXPERT_CLAMPED: experts are clamped units (as HB_FF_CLAMPED without biases, limit
  *                         ff_limit), HB_EXPERT_GELU: experts are ungated units down(gelu_erf(up h)) (no e<j>.gate);
  *                         router_kind HB_ROUTER_CHOSEN: the top_k largest logits are chosen and weighted by the softmax over
@@ -196,16 +207,18 @@ typedef struct hb_model_desc {
  *                         mlp.shared.*) runs for every token and is added.
  *        HB_FF_SILU       y = down(silu(gate) * up), no biases
  *        HB_FF_RELU2      y = down(relu(up)^2): mlp.up, mlp.down, no gate, no biases
+ *      bigram_buckets = B > 0: the row (previous token * bigram_mul_prev + token * bigram_mul_cur) mod B of the tensor `bigram`
+ *      ([B + 1][width]) is added to the (scaled) embedding; row B for the first token of a sequence.
  *      Norm gains are stored as offsets from 1 unless plain_gains.  embed_norm: the embedding row is normed (embed.norm) before
  *      the first layer.  tie_head: the logits come from the embedding table (no head tensor).  Logits are soft-capped: cap * tanh(z / cap) (cap <= 0: off).  Tensor names: embed[.norm], final.norm,
- *      head, l<i>.norm1/2[b], l<i>.ls1/2, l<i>.mix.{q,k,v,g,o,norm,a1,a2,a2.b | dq,dq.norm,uq (or q),dkv,dkv.norm,uk,uv,[sink,]g,o | q,k,[v,]g,o |
- *      q,k,v,{q,k,v}.conv,b,a,A_log,dt_bias,norm,g,o | in,conv,conv.b,dt_bias,A_log,D,norm,o | q,k,v,g,i,i.b,f,f.b,norm,o},
+ *      head, bigram, l<i>.norm1/2[b], l<i>.ls1/2, l<i>.hc1/2.{in,out,mix}, l<i>.mix.{q,k,v,g,o,norm,a1,a2,a2.b | dq,dq.norm,uq (or q),dkv,dkv.norm,uk,uv,[sink,]g,o | q,k,[v,]g,o |
+ *      q,k,v,{q,k,v}.conv,b,a,A_log,dt_bias,norm,g,o | in,conv,conv.b,dt_bias,A_log,D,norm,o | q,k,v,g,i,i.b,f,f.b,norm,o | q,k,v,g,norm,o},
  *      l<i>.mlp.{gate,up,down}[.b] or
  *      l<i>.mlp.{router,correction | router.b,[e<j>.gate,]e<j>.up,e<j>.down[,shared.gate,shared.up,shared.down]}. ---- */
-typedef enum hb_mixer { HB_MIXER_GLA = 0, HB_MIXER_LATENT = 1, HB_MIXER_GQA = 2, HB_MIXER_DELTA = 3, HB_MIXER_MAMBA2 = 4, HB_MIXER_MLSTM = 5 } hb_mixer;
+typedef enum hb_mixer { HB_MIXER_GLA = 0, HB_MIXER_LATENT = 1, HB_MIXER_GQA = 2, HB_MIXER_DELTA = 3, HB_MIXER_MAMBA2 = 4, HB_MIXER_MLSTM = 5, HB_MIXER_LIGHTNING = 6 } hb_mixer;
 typedef enum hb_mask { HB_MASK_WINDOW = 0, HB_MASK_CHUNK = 1, HB_MASK_CAUSAL = 2 } hb_mask;
 typedef enum hb_ff_kind { HB_FF_CLAMPED = 0, HB_FF_GELU_TANH = 1, HB_FF_MOE = 2, HB_FF_SILU = 3, HB_FF_RELU2 = 4 } hb_ff_kind;
-typedef enum hb_norm_place { HB_NORM_OF_SUM = 0, HB_NORM_OF_OUTPUT = 1, HB_NORM_BOTH_SIDES = 2, HB_NORM_PARALLEL = 3 } hb_norm_place;
+typedef enum hb_norm_place { HB_NORM_OF_SUM = 0, HB_NORM_OF_OUTPUT = 1, HB_NORM_BOTH_SIDES = 2, HB_NORM_PARALLEL = 3, HB_NORM_PRE = 4 } hb_norm_place;
 typedef enum hb_norm_kind { HB_NORM_RMS = 0, HB_NORM_TANH = 1 } hb_norm_kind;
 typedef enum hb_router_kind { HB_ROUTER_SOFTMAX = 0, HB_ROUTER_SIGMOID = 1, HB_ROUTER_CHOSEN = 2 } hb_router_kind;
 typedef enum hb_expert_kind { HB_EXPERT_SILU = 0, HB_EXPERT_CLAMPED = 1, HB_EXPERT_GELU = 2 } hb_expert_kind;
@@ -221,7 +234,8 @@ enum {
   HB_ATTN_QKV_CONV = 256,    /* q, k, v (after their biases) pass a causal convolution over conv_taps tokens per channel */
   HB_ATTN_OUT_GATE = 512,    /* the concatenated heads times sigmoid(mix.g x) entry by entry (mix.g has heads * vdim rows) */
   HB_ATTN_OUT_BIAS = 1024,   /* the output projection has a bias (mix.o.b) */
-  HB_ATTN_NO_SINK = 2048     /* LATENT: no learned sink in the softmax denominator */
+  HB_ATTN_NO_SINK = 2048,    /* LATENT: no learned sink in the softmax denominator */
+  HB_ATTN_NO_GATE = 4096     /* LATENT: the heads leave ungated (no mix.g) */
 };
 typedef struct hb_layer_desc {
   int32_t mixer;       /* hb_mixer */
@@ -237,7 +251,7 @@ typedef struct hb_layer_desc {
   float ff_limit;
   int32_t kv_heads;    /* GQA */
   int32_t mask;        /* hb_mask (GQA; LATENT: HB_MASK_WINDOW or HB_MASK_CAUSAL) */
-  int32_t attn_flags;  /* HB_ATTN_* (GQA; LATENT: HB_ATTN_NO_SINK, HB_ATTN_HEAD_GATE) */
+  int32_t attn_flags;  /* HB_ATTN_* (GQA; LATENT: HB_ATTN_NO_SINK, HB_ATTN_HEAD_GATE, HB_ATTN_NO_GATE) */
   int32_t rope_pairing;  /* 0: entry i pairs with i + rope_dims/2; 1: entry 2i pairs with 2i+1 (GQA, LATENT) */
   float rope_factor, rope_low, rope_high; /* GQA: frequency scaling, rope_factor <= 0: off.  With wavelength l = 2 pi / f: f stays */
   int32_t rope_original;                  /* where l < original/high, becomes f/factor where l > original/low, blends between */
@@ -261,7 +275,14 @@ typedef struct hb_layer_desc {
   float side_gate_cap;
   float mix_scale, side_scale;      /* weights of the two mixers' outputs; 0 = 1 */
   int32_t route_bias;               /* HB_FF_MOE: 1: mlp.router.b joins the logits, no correction tensor */
-  int32_t reserved[4];
+  int32_t route_group_max;          /* HB_FF_MOE: 1: a group of experts scores its largest score, 0: the sum of its two largest */
+  int32_t route_plain;              /* HB_FF_MOE: 1: no correction tensor */
+  /* YaRN scaling of the rotation (rope_yarn_factor <= 0: off).  With d(t) = dims ln(original / (2 pi t)) / (2 ln base),
+   * lo = max(floor d(fast), 0), hi = min(ceil d(slow), dims - 1): frequency i becomes f (r / factor + 1 - r),
+   * r = clamp((i - lo) / max(hi - lo, 0.001), 0, 1); cos and sin are multiplied by 0.1 ln(factor) + 1; original: rope_original */
+  float rope_yarn_factor, rope_yarn_fast, rope_yarn_slow;
+  int32_t reserved[3];
+  const float* head_decay;          /* LIGHTNING: [heads], read during hb_model_load_begin_stack / _random_stack */
 } hb_layer_desc;
 typedef struct hb_stack_desc {
   int32_t width, vocab, n_layers;
@@ -277,7 +298,10 @@ typedef struct hb_stack_desc {
   int32_t one_norm;    /* HB_NORM_PARALLEL: 1: both sublayers read norm1(x), no norm2 */
   int32_t layer_scale; /* HB_NORM_PARALLEL: 1: gains ls1 / ls2 on the sublayers' outputs */
   float resid_mult;    /* HB_NORM_PARALLEL: factor of the sublayers' sum; 0 = 1 */
-  int32_t reserved[1];
+  int32_t streams;     /* HB_NORM_PRE: copies of the residual stream; 0: one stream without read / write weights */
+  int32_t bigram_buckets, bigram_mul_prev, bigram_mul_cur; /* 0 buckets: no bigram embedding; multipliers >= 0 */
+  int32_t loop_start, loop_stop, loop_times;               /* loop_times <= 1: no loop */
+  int32_t reserved[2];
 } hb_stack_desc;
 
 typedef struct hb_sampling {
