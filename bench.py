@@ -16,7 +16,7 @@ cache.  tokens = sessions * (seq + decode).
                  oracle port on all host threads (pinned with threadpoolctl), bounded sample; --cpu-impl hf switches to
                  HF transformers on torch CPU, which measured 30x slower on the GPU box (profiles/r02c_reference_hf.json)
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference] [--workload llama8b|bge|pack|risepel|lurepel|latanex|funudra|kamivik]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference] [--workload llama8b|bge|pack|risepel|lurepel|latanex|funudra|kamivik|pupalix]
 """
 import argparse
 import json
@@ -408,11 +408,16 @@ def bench_kamivik(args):
     return bench_stack(args, "kamivik")
 
 
+def bench_pupalix(args):
+    return bench_stack(args, "pupalix")
+
+
 def bench_stack(args, family):
-    """--workload risepel | lurepel | latanex | funudra | kamivik: prefill and decode throughput of layer-list decoder stacks of that design
-    (helix_b200.configs.risepel_stack / lurepel_stack / latanex_stack / funudra_stack / kamivik_stack; the Funudra run also times
+    """--workload risepel | lurepel | latanex | funudra | kamivik | pupalix: prefill and decode throughput of layer-list decoder stacks of that design
+    (helix_b200.configs.risepel_stack / lurepel_stack / latanex_stack / funudra_stack / kamivik_stack / pupalix_stack; the Funudra run also times
     the Latanex stack, the closest design with recurrent layers, the Kamivik run the Risepel and Lurepel stacks, the closest with
-    latent attention and with a mixture of experts, at the same sizes; random weights, bf16 serving mode) at a few layer sizes, beside a Llama-family model of equal width / depth / feed-forward size
+    latent attention and with a mixture of experts, the Pupalix run the Funudra, Kamivik and Lurepel stacks, the closest with a recurrence, with
+    latent attention and with grouped-query attention in blocks, at the same sizes; random weights, bf16 serving mode) at a few layer sizes, beside a Llama-family model of equal width / depth / feed-forward size
     through the same engine API.  Per size: `sessions` prompts of `seq` tokens + `decode` generated tokens each; tokens/s =
     tokens / device time of the forward passes of each phase; `families` = CUDA-event spans of one profiled pass by kernel
     family with achieved FLOP/s or B/s."""
@@ -428,12 +433,15 @@ def bench_stack(args, family):
         ff = 4 * width
         row = {"width": width, "layers": layers, "ff": ff}
         build = {"risepel": configs.risepel_stack, "lurepel": configs.lurepel_stack, "latanex": configs.latanex_stack,
-                 "funudra": configs.funudra_stack, "kamivik": configs.kamivik_stack}[family]
+                 "funudra": configs.funudra_stack, "kamivik": configs.kamivik_stack, "pupalix": configs.pupalix_stack}[family]
         arms = [(family, build(width, layers, ff=ff)), ("llama", configs.llama_like(width, layers, ff))]
         if family == "funudra":
             arms.append(("latanex", configs.latanex_stack(width, layers, ff=ff)))
         if family == "kamivik":
             arms += [("risepel", configs.risepel_stack(width, layers, ff=ff)), ("lurepel", configs.lurepel_stack(width, layers, ff=ff))]
+        if family == "pupalix":
+            arms += [("funudra", configs.funudra_stack(width, layers, ff=ff)), ("kamivik", configs.kamivik_stack(width, layers, ff=ff)),
+                     ("lurepel", configs.lurepel_stack(width, layers, ff=ff))]
         if args.arms:
             arms = [a for a in arms if a[0] in args.arms.split(",")]
             if not any(a[0] == family for a in arms):
@@ -609,9 +617,9 @@ def main():
     ap.add_argument("--mixed-step-tokens", type=int, default=512)
     ap.add_argument("--fixed-total-sessions", type=int, default=256)
     ap.add_argument("--layers", type=int, default=0, help="debug: truncate the model (INVALID as a bench number)")
-    ap.add_argument("--workload", default="llama8b", choices=["llama8b", "bge", "pack", "risepel", "lurepel", "latanex", "funudra", "kamivik"])
+    ap.add_argument("--workload", default="llama8b", choices=["llama8b", "bge", "pack", "risepel", "lurepel", "latanex", "funudra", "kamivik", "pupalix"])
     ap.add_argument("--arms", default="", help="layer-list workloads: comma list of the models to time (default: all of the workload's)")
-    ap.add_argument("--risepel-sizes", nargs="*", default=[], help="risepel / lurepel / latanex / funudra / kamivik workloads: WIDTHxLAYERS ... (default 1024x12 2048x12 4096x6)")
+    ap.add_argument("--risepel-sizes", nargs="*", default=[], help="risepel / lurepel / latanex / funudra / kamivik / pupalix workloads: WIDTHxLAYERS ... (default 1024x12 2048x12 4096x6)")
     ap.add_argument("--chunks", type=int, default=100000)
     ap.add_argument("--ragged", action="store_true", help="bge workload: chunk lengths U[64,512] instead of 512")
     ap.add_argument("--pack-seconds", type=float, default=8.0)
@@ -625,10 +633,10 @@ def main():
     if args.impl == "reference":
         reference_arm(args, rank, world)
         return
-    if args.workload in ("bge", "pack", "risepel", "lurepel", "latanex", "funudra", "kamivik"):
+    if args.workload in ("bge", "pack", "risepel", "lurepel", "latanex", "funudra", "kamivik", "pupalix"):
         if rank == 0:
             {"bge": bench_bge, "pack": bench_pack, "risepel": bench_risepel, "lurepel": bench_lurepel, "latanex": bench_latanex,
-             "funudra": bench_funudra, "kamivik": bench_kamivik}[args.workload](args)
+             "funudra": bench_funudra, "kamivik": bench_kamivik, "pupalix": bench_pupalix}[args.workload](args)
         return
 
     import torch

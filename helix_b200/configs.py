@@ -180,6 +180,44 @@ def kamivik_stack(width, layers, ff=None, window=1024, experts=16, top=4, kv_ran
                        norm_place=E.NORM_PARALLEL, plain_gains=1, one_norm=1, layer_scale=1, resid_mult=0.5)
 
 
+def pupalix_stack(width, layers, ff=None, chunk=1024, streams=2, experts=16, top=4, groups=(4, 2), kv_rank=512, loop=None, vocab=32768,
+                  compute_f32=False):
+    """A Pupalix-design stack at sizes that resemble a served model's layers (random-init benchmarks): of every four layers two are
+    linear attention with constant decays (heads of 128 x 128), one is latent attention (heads of 128 unrotated and 64 rotated query /
+    key channels and 128 value channels over a latent of kv_rank entries, YaRN-scaled rotation), one grouped-query attention (heads
+    of 128, four query heads per key / value head) in blocks of `chunk` positions with capped scores.  Even layers have a dense gated
+    unit of size ff, odd ones a mixture of `experts` gated experts of which a token uses `top`, sized so that a token spends the
+    products of the dense unit.  `streams` copies of the residual stream; loop = (start, stop, times): layers start .. stop - 1 run
+    times times in a row."""
+    from . import engine as E
+    heads = max(1, width // 128)
+    ff = ff or (width * 4)
+    out = []
+    for i in range(layers):
+        if i % 4 == 2:
+            l = E.LayerDesc(mixer=E.MIXER_LATENT, heads=heads, dim=128, vdim=128, kv_rank=kv_rank, rot_dim=64, rope_dims=64, rope_pairing=1,
+                            rope_base=10000.0, scale=(128 + 64) ** -0.5, mask=E.MASK_CAUSAL, attn_flags=E.ATTN_NO_SINK | E.ATTN_NO_GATE,
+                            rope_yarn_factor=4.0, rope_original=4096)
+        elif i % 4 == 3:
+            l = E.LayerDesc(mixer=E.MIXER_GQA, heads=heads, kv_heads=max(1, heads // 4), dim=128, vdim=128, scale=128 ** -0.5, score_cap=30.0,
+                            mask=E.MASK_CHUNK, window=chunk, attn_flags=E.ATTN_V_IS_K | E.ATTN_QK_PROJ_NORM)
+        else:
+            l = E.LayerDesc(mixer=E.MIXER_LIGHTNING, heads=heads, dim=128, vdim=128,
+                            head_decay=tuple(1.0 - 2.0 ** (-1.0 - 8.0 * h / heads) for h in range(heads)))
+        if i % 2 == 0:
+            l.ff_kind, l.ff = E.FF_GELU_TANH, ff
+        else:
+            l.ff_kind, l.ff, l.experts, l.top_k = E.FF_MOE, max(64, ff // top), experts, top
+            l.route_plain, l.route_groups, l.route_keep, l.route_group_max = 1, groups[0], groups[1], 1
+        out.append(l)
+    d = E.StackDesc(width=width, vocab=vocab, layers=out, compute_f32=int(compute_f32), norm_eps=1e-5, resid_alpha=1.0,
+                    norm_place=E.NORM_PRE, plain_gains=1, tie_head=1, streams=streams, embed_scale=width ** 0.5, logit_scale=0.5,
+                    logit_softcap=30.0, bigram_buckets=vocab - 1, bigram_mul_prev=31, bigram_mul_cur=7)
+    if loop:
+        d.loop_start, d.loop_stop, d.loop_times = loop
+    return d
+
+
 def llama_like(width, layers, ff, vocab=32768):
     """The closest existing decoder at equal width / depth / feed-forward size (comparison arm of the layer-list benchmarks)."""
     heads = max(1, width // 128)

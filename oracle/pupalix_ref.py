@@ -280,3 +280,164 @@ class PupalixOracle:
         st["prev"] = int(tokens[-1])
         z = rms_norm(xs.sum(0), sd["final.norm"], self.eps) @ sd["embed"].T * cfg.get("logit_scale", 1.0)
         return cap(z, cfg.get("logit_softcap"))
+
+
+# ------------------------------------------------------------------ random checkpoints for tests
+def latent_cfg(heads=3, dim=16, rot_dim=8, vdim=24, kv_rank=40, base=1000.0, scaling=(4.0, 60, 8.0, 1.0), scale=None):
+    """scaling: (factor, original, fast, slow) or None"""
+    rot = dict(dims=rot_dim, base=float(base))
+    if scaling:
+        rot["scaling"] = dict(factor=float(scaling[0]), original=int(scaling[1]), fast=float(scaling[2]), slow=float(scaling[3]))
+    return dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, rot=rot, scale=float(scale if scale is not None else (dim + rot_dim) ** -0.5))
+
+
+def gqa_cfg(heads=4, kv_heads=2, dim=24, block=37, softcap=20.0, scale=None):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=float(scale if scale is not None else 2.0 * dim ** -0.5))
+    if softcap:
+        m["softcap"] = float(softcap)
+    if block:
+        m["mask"] = dict(size=block)
+    return m
+
+
+def light_cfg(heads=3, dim=24, vdim=40, decay=(0.5, 0.93, 0.998)):
+    return dict(heads=heads, dim=dim, vdim=vdim, decay=[float(decay[h % len(decay)]) for h in range(heads)])
+
+
+def moe_cfg(experts=6, top=3, ff=40, groups=(3, 2)):
+    r = dict(experts=experts, top=top)
+    if groups:
+        r["groups"] = dict(count=groups[0], keep=groups[1])
+    return dict(kind="moe", expert=dict(ff=ff), router=r)
+
+
+def dense_cfg(ff=72):
+    return dict(kind="dense", ff=ff)
+
+
+DEFAULT_ORDER = ((LIGHT, "dense"), (LATENT, "moe"), (GQA, "dense"), (LIGHT, "moe"))
+
+
+def random_config(width=96, vocab=120, order=DEFAULT_ORDER, latent=None, gqa=None, light=None, moe=None, ff=72, streams=3, loop=(1, 3, 2), buckets=97,
+                  mul=(31, 5), embed_scale=2.5, logit_scale=0.5, logit_cap=12.0, eps=1e-5, per_layer=None, per_mlp=None):
+    """order: (type, "dense" | "moe" | None) per layer; per_layer / per_mlp {i: dict}: that layer's mixer / feed-forward."""
+    layers = []
+    for i, (kind, f) in enumerate(order):
+        mixer = {LATENT: latent or latent_cfg(), GQA: gqa or gqa_cfg(), LIGHT: light or light_cfg()}[kind]
+        mlp = dense_cfg(ff) if f == "dense" else (moe or moe_cfg()) if f == "moe" else None
+        layers.append(dict(type=kind, mixer=(per_layer or {}).get(i, mixer), mlp=(per_mlp or {}).get(i, mlp)))
+    cfg = dict(architecture="Pupalix", width=width, vocab=vocab, layers=layers, norm=dict(eps=eps), streams=streams, logit_scale=float(logit_scale),
+               embedding=dict(scale=float(embed_scale), bigram=dict(buckets=buckets, mul_prev=mul[0], mul_cur=mul[1])))
+    if logit_cap:
+        cfg["logit_softcap"] = float(logit_cap)
+    if loop:
+        cfg["loop"] = dict(start=loop[0], stop=loop[1], times=loop[2])
+    return cfg
+
+
+def reserved(cfg):
+    """leading stream entries that no sublayer writes: one per expert, then two for planted features"""
+    return max([ly["mlp"]["router"]["experts"] for ly in cfg["layers"] if ly["mlp"] and ly["mlp"]["kind"] == "moe"] + [0]) + 2
+
+
+def random_state_dict(cfg, seed=0):
+    """Router choices are made by the leading stream entries, which hold a shuffled grid of values per token and keep its order
+    through every mix of the copies, so that no choice is a close call; everything else is random."""
+    from .weights import _rng, _t, to_bf16_f32
+    W, V, S = cfg["width"], cfg["vocab"], cfg["streams"]
+    s = lambda n: 1.0 / math.sqrt(n)
+    n_res = reserved(cfg)
+    E0 = n_res - 2
+    step = min(0.5, 4.0 / max(E0, 1))
+    table = _t(seed, "embed", (V, W), 0.4)
+    g = _rng(seed, "grid")
+    for v in range(V):
+        table[v, :E0] = (g.permutation(E0) - (E0 - 1) / 2.0) * step
+    table[:, E0:n_res] = 0.0
+    big = _t(seed, "bigram", (cfg["embedding"]["bigram"]["buckets"] + 1, W), 0.6)
+    big[:, :n_res] = 0.0
+    sd = {"embed": to_bf16_f32(table), "bigram": to_bf16_f32(big), "final.norm": _t(seed, "fn", (W,), 0.1, 1.0)}
+    for i, ly in enumerate(cfg["layers"]):
+        m, p = ly["mixer"], f"l{i}."
+        H, Dk, Dv = m["heads"], m["dim"], m["vdim"]
+        o_rows = _t(seed, p + "o", (W, H * Dv), 1.5 * s(H * Dv))
+        o_rows[:n_res] = 0.0
+        sd[p + "mix.o"] = o_rows
+        for q in (1, 2):
+            if q == 2 and not ly["mlp"]:
+                continue
+            sd[p + f"norm{q}"] = _t(seed, p + f"n{q}", (W,), 0.1, 1.0)
+            sd[p + f"norm{q}"][:n_res] = 1.0
+            sd[p + f"hc{q}.in"] = to_bf16_f32(np.abs(_t(seed, p + f"hi{q}", (S,), 0.3, 1.0 / S)) + 0.05)
+            sd[p + f"hc{q}.out"] = _t(seed, p + f"ho{q}", (S,), 0.5, 0.7)
+            sd[p + f"hc{q}.mix"] = to_bf16_f32(np.abs(_t(seed, p + f"hm{q}", (S, S), 0.15)) + 0.75 * np.eye(S))
+        if ly["type"] == LATENT:
+            Dr, R = m["rot_dim"], m["kv_rank"]
+            sd[p + "mix.q"] = _t(seed, p + "q", (H * (Dk + Dr), W), 1.5 * s(W))
+            sd[p + "mix.dkv"] = _t(seed, p + "dkv", (R + Dr, W), 1.5 * s(W))
+            sd[p + "mix.dkv.norm"] = _t(seed, p + "dkvn", (R,), 0.1, 1.0)
+            sd[p + "mix.uk"] = _t(seed, p + "uk", (H * Dk, R), 1.5 * s(R))
+            sd[p + "mix.uv"] = _t(seed, p + "uv", (H * Dv, R), 1.5 * s(R))
+        elif ly["type"] == GQA:
+            G = m["kv_heads"]
+            sd[p + "mix.q"] = _t(seed, p + "q", (H * Dk, W), 1.5 * s(W))
+            sd[p + "mix.k"] = _t(seed, p + "k", (G * Dk, W), 1.5 * s(W))
+            sd[p + "mix.q.norm"] = _t(seed, p + "qn", (H * Dk,), 0.2, 1.0)
+            sd[p + "mix.k.norm"] = _t(seed, p + "kn", (G * Dk,), 0.2, 1.0)
+        else:
+            for n, rows in (("q", H * Dk), ("k", H * Dk), ("v", H * Dv), ("g", H * Dv)):
+                sd[p + "mix." + n] = _t(seed, p + n, (rows, W), 1.5 * s(W))
+            sd[p + "mix.norm"] = _t(seed, p + "ln", (H * Dv,), 0.2, 1.0)
+        if not ly["mlp"]:
+            continue
+        if ly["mlp"]["kind"] == "dense":
+            units, Fn = [""], ly["mlp"]["ff"]
+        else:
+            E, Fn = ly["mlp"]["router"]["experts"], ly["mlp"]["expert"]["ff"]
+            units = [f"e{e}." for e in range(E)]
+            router = _t(seed, p + "router", (E, W), 0.05 * s(W))
+            router[:, :n_res] = 0.0
+            for e in range(E):
+                router[e, e] = 4.0 / step / cfg["embedding"]["scale"]
+            sd[p + "mlp.router"] = to_bf16_f32(router)
+        for u in units:
+            sd[p + f"mlp.{u}gate"] = _t(seed, p + f"{u}g", (Fn, W), 1.5 * s(W))
+            sd[p + f"mlp.{u}up"] = _t(seed, p + f"{u}u", (Fn, W), 1.5 * s(W))
+            down = _t(seed, p + f"{u}d", (W, Fn), (2.0 if u else 1.0) * s(Fn))
+            down[:n_res] = 0.0
+            sd[p + f"mlp.{u}down"] = down
+    return sd
+
+
+def plant_marker(cfg, sd, layers, strength=14.0):
+    """Token vocab - 1 becomes a marker: in the named attention layers every head's score for it stands out wherever it is seen, and
+    its value is unlike any other token's, so whether a position sees it shows in the logits."""
+    from .weights import to_bf16_f32
+    sd = {k: v.copy() for k, v in sd.items()}
+    const, mark = reserved(cfg) - 2, reserved(cfg) - 1
+    sd["embed"][:, const], sd["embed"][:, mark] = 1.0, 0.0
+    sd["embed"][-1, mark] = 4.0
+    for i in layers:
+        m, p = cfg["layers"][i]["mixer"], f"l{i}."
+        H, Dk = m["heads"], m["dim"]
+        if cfg["layers"][i]["type"] == LATENT:
+            Dr, R = m["rot_dim"], m["kv_rank"]
+            sd[p + "mix.dkv.norm"][0] = 1.0
+            sd[p + "mix.dkv"][0] = 0.0
+            sd[p + "mix.dkv"][0, mark] = 16.0
+            for h in range(H):
+                q = sd[p + "mix.q"][h * (Dk + Dr):(h + 1) * (Dk + Dr)]
+                q *= 0.25
+                q[0] = 0.0
+                q[0, const] = strength / (0.5 * math.sqrt(R) * m["scale"])
+                uk = sd[p + "mix.uk"][h * Dk:(h + 1) * Dk]
+                uk[0] = 0.0
+                uk[0, 0] = 1.0
+        else:  # the norms over the whole projections leave entry 0 of every head near sqrt(dim) in marked keys and in all queries
+            for n, rows, col, big in (("q", H, const, 40.0), ("k", m["kv_heads"], mark, 16.0)):
+                w = sd[p + "mix." + n]
+                for h in range(rows):
+                    w[h * Dk] = 0.0
+                    w[h * Dk, col] = big
+                    sd[p + f"mix.{n}.norm"][h * Dk] = 1.0
+    return {k: to_bf16_f32(v) for k, v in sd.items()}
