@@ -455,6 +455,52 @@ __global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* __re
   }
 }
 
+// The same with a part in registers as float4 (parts of a multiple of 4 entries, up to 4 * 256 * CH)
+template <typename WT, int CH>
+__global__ void __launch_bounds__(256) gated_group_norm_vec_kernel(const float* __restrict__ y, long ldy, const float* __restrict__ z, long ldz,
+                                                                   const WT* __restrict__ w, float eps, int parts, float* __restrict__ out,
+                                                                   bf16* __restrict__ outb, int n, int gate_last) {
+  __shared__ float red[32];
+  const int t = blockIdx.y, part = blockIdx.x, len = n / parts, c0 = part * len;
+  const float* ys = y + (size_t)t * ldy + c0;
+  const float* zs = z + (size_t)t * ldz + c0;
+  float4 u[CH], g[CH];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = (threadIdx.x + c * 256) * 4;
+    u[c] = g[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= len) continue;
+    u[c] = *reinterpret_cast<const float4*>(ys + i);
+    g[c] = *reinterpret_cast<const float4*>(zs + i);
+  }
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const float4 s = make_float4(sigmoidf_(g[c].x), sigmoidf_(g[c].y), sigmoidf_(g[c].z), sigmoidf_(g[c].w));
+    if (!gate_last) u[c] = make_float4(u[c].x * (g[c].x * s.x), u[c].y * (g[c].y * s.y), u[c].z * (g[c].z * s.z), u[c].w * (g[c].w * s.w));
+    g[c] = gate_last ? s : make_float4(1.f, 1.f, 1.f, 1.f);
+    ss += u[c].x * u[c].x + u[c].y * u[c].y + u[c].z * u[c].z + u[c].w * u[c].w;
+  }
+  const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)len + eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = (threadIdx.x + c * 256) * 4;
+    if (i >= len) continue;
+    const size_t d = (size_t)t * n + c0 + i;
+    float4 v;
+    v.x = u[c].x * rs * ldf<WT>(w, c0 + i) * g[c].x; v.y = u[c].y * rs * ldf<WT>(w, c0 + i + 1) * g[c].y;
+    v.z = u[c].z * rs * ldf<WT>(w, c0 + i + 2) * g[c].z; v.w = u[c].w * rs * ldf<WT>(w, c0 + i + 3) * g[c].w;
+    if (out) *reinterpret_cast<float4*>(out + d) = v;
+    if (outb) {
+      __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+      uint2 pk;
+      pk.x = *reinterpret_cast<unsigned*>(&lo);
+      pk.y = *reinterpret_cast<unsigned*>(&hi);
+      *reinterpret_cast<uint2*>(outb + d) = pk;
+    }
+  }
+}
+
 __global__ void gate_scale_kernel(const float* __restrict__ in, const bf16* __restrict__ inb, long ldi, const float* __restrict__ g, long ldg,
                                   float scale, float* __restrict__ out, bf16* __restrict__ outb, long ldout, int col0, int n) {
   const int t = blockIdx.y, e = blockIdx.x * blockDim.x + threadIdx.x;
@@ -702,6 +748,18 @@ cudaError_t gated_group_norm(cudaStream_t s, const float* y, long ldy, const flo
   if (T <= 0) return cudaSuccess;
   if (parts < 1 || n % parts) return cudaErrorInvalidValue;
   dim3 grid(parts, T);
+  const int len = n / parts;
+  if (len % 4 == 0 && len <= 8192 && ((ldy | ldz) & 3) == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)out) & 15) == 0 && ((uintptr_t)outb & 7) == 0) {
+#define HB_GGN(WT, CH) gated_group_norm_vec_kernel<WT, CH><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const WT*)w, eps, parts, out, outb, n, gate_last)
+#define HB_GGN_T(CH) do { if (f32) HB_GGN(float, CH); else HB_GGN(bf16, CH); } while (0)
+    if (len <= 1024) HB_GGN_T(1);
+    else if (len <= 2048) HB_GGN_T(2);
+    else if (len <= 4096) HB_GGN_T(4);
+    else HB_GGN_T(8);
+#undef HB_GGN_T
+#undef HB_GGN
+    return cudaGetLastError();
+  }
   if (f32) gated_group_norm_kernel<float><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const float*)w, eps, parts, out, outb, n, gate_last);
   else gated_group_norm_kernel<bf16><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const bf16*)w, eps, parts, out, outb, n, gate_last);
   return cudaGetLastError();

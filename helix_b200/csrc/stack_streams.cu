@@ -62,34 +62,47 @@ __global__ void __launch_bounds__(256) stream_step_vec_kernel(StreamStep a) {
   float* xr = a.x + r * S * W;
   float4 u[CH];
   float ss = 0.f;
+  // all of a thread's loads go out before its first store when its share of the row fits in registers (the stores may alias
+  // later loads for all the compiler knows, so it cannot move them itself); a thread only reads what it writes itself
+  constexpr int B = S * CH <= 8 ? CH : 1;
+  float4 x[B][S], y[B];
+  auto load = [&](int c, float4(&xc)[S], float4& yc) {
+    const int i = (threadIdx.x + c * 256) * 4;
+    yc = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= W) return;
+#pragma unroll
+    for (int s = 0; s < S; ++s) xc[s] = a.x0 ? *reinterpret_cast<const float4*>(a.x0 + r * W + i) : *reinterpret_cast<const float4*>(xr + (size_t)s * W + i);
+    if (a.y) yc = *reinterpret_cast<const float4*>(a.y + r * W + i);
+#pragma unroll
+    for (int k = 0; k < kTop; ++k)
+      if (k < a.top_k) yc = fma4(wk[k], ld4<bf16>(a.rows + rk[k] + i), yc);
+    if (a.bias) yc = fma4(1.f, ld4<WT>((const WT*)a.bias + i), yc);
+  };
+  if constexpr (B > 1) {
+#pragma unroll
+    for (int c = 0; c < CH; ++c) load(c, x[c], y[c]);
+  }
 #pragma unroll
   for (int c = 0; c < CH; ++c) {
     const int i = (threadIdx.x + c * 256) * 4;
     if (i >= W) continue;
-    float4 x[S], v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if constexpr (B == 1) load(c, x[0], y[0]);
+    float4(&xc)[S] = x[B == 1 ? 0 : c];
+    const float4 yc = y[B == 1 ? 0 : c];
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (a.x0) {
-      const float4 e = *reinterpret_cast<const float4*>(a.x0 + r * W + i);
 #pragma unroll
       for (int s = 0; s < S; ++s) {
-        x[s] = e;
-        *reinterpret_cast<float4*>(xr + (size_t)s * W + i) = e;
-        v = fma4(in[s], e, v);
+        *reinterpret_cast<float4*>(xr + (size_t)s * W + i) = xc[s];
+        v = fma4(in[s], xc[s], v);
       }
-    } else {
-#pragma unroll
-      for (int s = 0; s < S; ++s) x[s] = *reinterpret_cast<const float4*>(xr + (size_t)s * W + i);
     }
     if (add) {
-      float4 y = a.y ? *reinterpret_cast<const float4*>(a.y + r * W + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-      for (int k = 0; k < kTop; ++k)
-        if (k < a.top_k) y = fma4(wk[k], ld4<bf16>(a.rows + rk[k] + i), y);
-      if (a.bias) y = fma4(1.f, ld4<WT>((const WT*)a.bias + i), y);
 #pragma unroll
       for (int t = 0; t < S; ++t) {
-        float4 n = make_float4(out[t] * y.x, out[t] * y.y, out[t] * y.z, out[t] * y.w);
+        float4 n = make_float4(out[t] * yc.x, out[t] * yc.y, out[t] * yc.z, out[t] * yc.w);
 #pragma unroll
-        for (int s = 0; s < S; ++s) n = fma4(mix[s][t], x[s], n);
+        for (int s = 0; s < S; ++s) n = fma4(mix[s][t], xc[s], n);
         if (!a.last) *reinterpret_cast<float4*>(xr + (size_t)t * W + i) = n;
         v = fma4(in[t], n, v);
       }
