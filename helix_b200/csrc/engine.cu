@@ -167,6 +167,7 @@ void Engine::free_all() {
   };
   frh(h_step_);
   frh(h_sampled_);
+  frh(kernel_error_);
   frh(h_lp_ids_);
   frh(h_lp_vals_);
   frh(h_logits_);
@@ -1371,6 +1372,10 @@ int Engine::run_prefill(std::vector<Request*>& batch) {
   CU(cudaEventRecord(fwd_b_, stream_));
   if (!step_driven_) CU(cudaMemcpyAsync(h_sampled_, sampled_, (size_t)B * 4, cudaMemcpyDeviceToHost, stream_));
   CU(cudaStreamSynchronize(stream_));
+  if (kernel_error_ && *kernel_error_) {
+    *kernel_error_ = 0;
+    return fail_cuda(cudaErrorLaunchTimeout, "a wait inside a kernel of this step ran out");
+  }
   {
     float ms = 0.f;
     if (cudaEventElapsedTime(&ms, fwd_a_, fwd_b_) == cudaSuccess) gpu_ms_prefill_ += ms;

@@ -268,6 +268,7 @@ class Engine {
   uint8_t* d_step_ = nullptr;  // per-step int/float inputs (layout())
   uint8_t* h_step_ = nullptr;  // pinned mirror
   int32_t* h_sampled_ = nullptr;
+  int* kernel_error_ = nullptr;  // pinned: a kernel of a layer-list step whose bounded wait ran out sets it
   size_t step_bytes_ = 0;
   float* all_logits_ = nullptr;  // lazily allocated [cap_rows][vocab] for HB_CAPTURE_PROMPT_LOGITS
   int all_logits_rows_ = 0;

@@ -260,6 +260,11 @@ static bool gqa_fused_ok(const Model& m, const hb_layer_desc& l, int max_ctx) {
   (void)max_ctx;
   return !off && !m.sd.compute_f32 && l.mixer == HB_MIXER_GQA && l.dim == l.vdim && (l.dim == 64 || l.dim == 128);
 }
+// Linear-attention layers whose prompt portions run chunk by chunk on the tensor cores: bf16 mode and head sizes of that kernel
+static bool light_chunk_ok(const Model& m, const hb_layer_desc& l) {
+  static const bool off = [] { const char* e = getenv("HB_STACK_LIN_CHUNK"); return e && atoi(e) == 0; }();
+  return !off && !m.sd.compute_f32 && l.mixer == HB_MIXER_LIGHTNING && lin_chunk_ok(l.dim, l.vdim) && l.heads * l.vdim <= 8192;
+}
 // experts run as grouped tcgen05 products when the mode and the shapes allow (16-byte TMA strides, at least one MMA tile)
 static bool moe_grouped_ok(const Model& m, const hb_layer_desc& l) {
   static const bool off = [] { const char* e = getenv("HB_STACK_MOE_GROUPED"); return e && atoi(e) == 0; }();
@@ -292,6 +297,7 @@ static StackDims stack_dims(const Model& m, int max_ctx, int tokens) {
     } else if (l.mixer == HB_MIXER_LIGHTNING) {
       d.cx = std::max(d.cx, l.heads * l.vdim);
       d.decays += l.heads;
+      if (light_chunk_ok(m, l)) d.gu = std::max(d.gu, m.sw[i].n_in);
     } else if (l.mixer == HB_MIXER_DELTA) {
       d.n2 = std::max(d.n2, 2 * l.kv_heads * l.dim + l.heads * l.vdim + 2 * l.heads + l.kv_heads);
       d.cx = std::max(d.cx, l.heads * l.vdim);
@@ -402,6 +408,7 @@ int Engine::alloc_runtime_stack() {
   CU(stack_delta_init());
   CU(stack_ssm_init());
   CU(stack_streams_init());
+  CU(stack_lightning_init());
   CU(attn_latent_init());
   if (!sd.compute_f32) {  // stream-K plans allocate on first use of a shape: make them now, not inside a graph capture
     SmLimitScope sm_scope(cfg_.sm_budget);
@@ -572,6 +579,8 @@ int Engine::alloc_runtime_stack() {
   CU(cudaMalloc(&d_step_, step_bytes_));
   CU(cudaMallocHost(&h_step_, step_bytes_));
   CU(cudaMallocHost(&h_sampled_, (size_t)b_cap_ * 4));
+  CU(cudaMallocHost(&kernel_error_, sizeof(int)));
+  *kernel_error_ = 0;
   CU(cudaMallocHost(&h_lp_ids_, (size_t)cfg_.max_seqs * HB_MAX_LOGPROBS * 4));
   CU(cudaMallocHost(&h_lp_vals_, (size_t)cfg_.max_seqs * HB_MAX_LOGPROBS * 4));
 
@@ -1014,8 +1023,18 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     // every projection that reads the stream, in one GEMM
     // (grouped-query layers keep the rows of this product dense: the buffer's stride is sized for the widest gated unit)
     const int ldin = l.mixer == HB_MIXER_GQA ? up8(w.n_in) : k.ld1;
-    int rc = stack_gemm(xin, x16, W, w.w_in, w.n_in, W, k.p1, ldin, T);
-    if (rc != HB_OK) return rc;
+    int rc = HB_OK, longest_entry = 0;
+    for (const StepEntry& en : step_entries_) longest_entry = std::max(longest_entry, en.n);
+    // linear attention over a long portion: bf16 rows, the activations of q | k | v on the accumulators' way out
+    const bool chunked = light_chunk_ok(model_, l) && T > 256 && longest_entry >= kAttDenseMin && k.gu16 && stack_tc(w.n_in, W, W, w.n_in);
+    if (chunked) {
+      GemmArgs g{x16, W, (const bf16*)w.w_in, W, k.gu16, w.n_in, nullptr, 0, nullptr, T, w.n_in, W, EPI_SILU_COLS, 0};
+      g.silu_cols = w.off_g;
+      SPAN(0, 2.0 * T * w.n_in * W, gemm_bf16_tn(stream_, g));
+    } else {
+      rc = stack_gemm(xin, x16, W, w.w_in, w.n_in, W, k.p1, ldin, T);
+      if (rc != HB_OK) return rc;
+    }
     // the norm that prepares the input of whatever follows a sublayer (norms on both sides)
     const void* pre_next = i + 1 < sd.n_layers ? model_.sw[i + 1].norm1 : nullptr;
     const int ocols = w.o_cols ? w.o_cols : H * Dv;  // columns of the output projection (both mixers' when there are two)
@@ -1048,6 +1067,18 @@ int Engine::forward_stack(int T, int B, const StepLayout& L, const int32_t* extr
     } else if (l.mixer == HB_MIXER_MLSTM) {
       rc = run_memory(w, k.ld1, 0, ocols, 1.f, mo_f32);
       if (rc != HB_OK) return rc;
+    } else if (chunked) {
+      LinChunkArgs la{};
+      la.q = k.gu16 + w.off_q; la.k = k.gu16 + w.off_k; la.v = k.gu16 + w.off_v; la.ld = w.n_in;
+      la.decay = w.decay;
+      la.out = k.ctx; la.ldo = k.ldctx;
+      la.state = state_ + w.state_off; la.slot_stride = (long)model_.state_floats;
+      la.cu = cu; la.first_pos = first; la.slots = sslot;
+      la.error = kernel_error_;
+      la.T = T; la.B = B; la.H = H; la.Dk = Dk; la.Dv = Dv;
+      SPAN(6, 4.0 * T * H * Dk * Dv, lin_chunk(stream_, la));
+      SPAN(3, 14.0 * T * H * Dv, gated_group_norm(stream_, k.ctx, k.ldctx, nullptr, w.n_in, w.hnorm, f32, sd.norm_eps, 1, mo_f32, mo16, T, H * Dv, true,
+                                                  k.gu16 + w.off_g));
     } else if (l.mixer == HB_MIXER_LIGHTNING) {
       LinRecArgs ra{};
       ra.q = k.p1; ra.ldq = k.ld1; ra.q_off = w.off_q;

@@ -98,7 +98,7 @@ __global__ void __launch_bounds__(kNumThreads, 1)
 gemm_tn_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                const __grid_constant__ CUtensorMap map_c, const __grid_constant__ CUtensorMap map_r,
                const bf16* __restrict__ bias, int M, int N, int K, int tile_grp, int tile_group_n,
-               const __grid_constant__ RopeEpi rope, const int32_t* __restrict__ m_tile_group, float glu_limit) {
+               const __grid_constant__ RopeEpi rope, const int32_t* __restrict__ m_tile_group, float glu_limit, int silu_cols) {
   using C = Cfg<BN, CG>;
   constexpr int TILE_M = BLOCK_M * CG;  // rows of one UMMA tile (per CTA: BLOCK_M)
   const uint32_t cta_rank = (CG == 2) ? cluster_ctarank() : 0u;
@@ -427,6 +427,11 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
               for (int j = 0; j < 32; j += 2) gelu_erf2(f[j], f[j + 1]);
             }
+            if constexpr (EPI == EPI_SILU_COLS) {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (n_out0 + col + j < silu_cols) f[j] = silu(f[j]);
+            }
             if constexpr (EPI == EPI_RELU2) {
 #pragma unroll
               for (int j = 0; j < 32; ++j) {
@@ -540,7 +545,7 @@ cudaError_t launch_cfg(cudaStream_t stream, const GemmArgs& g, int num_sms) {
   cfg.attrs = attr;
   cfg.numAttrs = (CG > 1) ? 1 : 0;
   static const int l2_hints = [] { const char* e = getenv("HB_GEMM_L2HINTS"); return e ? atoi(e) : 0; }();  // A/B knob
-  return cudaLaunchKernelEx(&cfg, kern, ma, mb, mc, mr, g.bias, g.M, g.N, g.K, grp, group_n | (l2_hints ? 2 : 0), g.rope, g.m_tile_group, g.glu_limit);
+  return cudaLaunchKernelEx(&cfg, kern, ma, mb, mc, mr, g.bias, g.M, g.N, g.K, grp, group_n | (l2_hints ? 2 : 0), g.rope, g.m_tile_group, g.glu_limit, g.silu_cols);
 }
 
 bool use_pair() {  // HB_GEMM_2CTA=0 falls back to single-CTA tiles (A/B measurements)
@@ -605,6 +610,7 @@ cudaError_t gemm_init() {
   if ((e = set_attr_epi<EPI_CLAMPGLU>()) != cudaSuccess) return e;
   if ((e = set_attr_epi<EPI_RELU2>()) != cudaSuccess) return e;
   if ((e = set_attr_epi<EPI_GELU>()) != cudaSuccess) return e;
+  if ((e = set_attr_epi<EPI_SILU_COLS>()) != cudaSuccess) return e;
   return set_attr_epi<EPI_SWIGLU>();
 }
 
@@ -653,6 +659,7 @@ cudaError_t gemm_bf16_tn(cudaStream_t stream, const GemmArgs& g) {
     case EPI_F32: return launch_epi<EPI_F32>(stream, g, sms);
     case EPI_RELU2: return launch_epi<EPI_RELU2>(stream, g, sms);
     case EPI_GELU: return launch_epi<EPI_GELU>(stream, g, sms);
+    case EPI_SILU_COLS: return launch_epi<EPI_SILU_COLS>(stream, g, sms);
     case EPI_ROPE: {
       const RopeEpi& r = g.rope;
       if ((g.N % 256) || !r.out || !r.cs || (r.D != 64 && r.D != 128) || g.N != (r.Hq + 2 * r.Hkv) * r.D || (r.ldc % 8)) return cudaErrorInvalidValue;

@@ -31,6 +31,7 @@ enum Epi : int {
                        // (limit = GemmArgs::glu_limit)
   EPI_RELU2 = 10,      // C = relu(acc)^2                      (bf16)
   EPI_GELU = 11,       // C = gelu_erf(acc)                    (bf16)
+  EPI_SILU_COLS = 12,  // C = silu(acc) in the columns below silu_cols, acc elsewhere (bf16)
   EPI_ROPE = 7,        // fused QKV projection of a decoder: C = bf16(acc [+ bias]) with the q and k heads rotated
                        // (RopeEpi) and the k / v rows also scattered into the paged KV cache
 };
@@ -65,6 +66,7 @@ struct GemmArgs {
   const int32_t* m_tile_group = nullptr;
   int groups = 1;
   float glu_limit = 0.f;  // EPI_CLAMPGLU
+  int silu_cols = 0;      // EPI_SILU_COLS
 };
 cudaError_t gemm_bf16_tn(cudaStream_t stream, const GemmArgs& a);
 // Debug/test-only CUDA-core GEMM (same contract, EPI_NONE/EPI_F32 only); used by tests as an on-device checker.
@@ -593,6 +595,21 @@ struct LinRecArgs {
   int silu = 0;
 };
 cudaError_t lin_recurrence(cudaStream_t s, const LinRecArgs& a);
+// S_t = decay_h S_(t-1) + k_t v_t^T, out_t = S_t^T q_t on the tensor cores, chunk by chunk (stack_lightning.cu): q, k [T, H * Dk] and
+// v [T, H * Dv] are bf16 columns (behind their activations) of rows of stride ld, out fp32, the state as for lin_recurrence.
+// error: a word that the host can read; set to 1 when a wait inside the kernel ran out (results are then void).
+struct LinChunkArgs {
+  const bf16* q; const bf16* k; const bf16* v; long ld;
+  const float* decay;
+  float* out; long ldo;
+  float* state; long slot_stride;  // state + slot * slot_stride -> this layer's [H][Dk][Dv]
+  const int32_t* cu; const int32_t* first_pos; const int32_t* slots;
+  int* error;
+  int T, B, H, Dk, Dv;
+};
+bool lin_chunk_ok(int Dk, int Dv);
+cudaError_t stack_lightning_init();
+cudaError_t lin_chunk(cudaStream_t s, const LinChunkArgs& a);
 // Matrix memory read-out: o = num[t, h, :] / (max(|nq[t, h]|, ab[t, 2H + h]) + 1e-6); out[t, col0 + h Dv + i] =
 // o_i / rms(o) * w[h Dv + i] * sigmoid(g[t, h Dv + i]) * scale (+ bf16 copy at the same place of out_b16)
 cudaError_t memory_readout(cudaStream_t s, const float* num, long ldnum, const float* nq, long ldn, const float* ab, long ldab,
@@ -600,9 +617,9 @@ cudaError_t memory_readout(cudaStream_t s, const float* num, long ldnum, const f
                            long ldout, int col0, int T, int H, int Dv);
 // State-space read-out: u = y[t, :] * silu(z[t, :]) over n entries, divided by its root mean square in `parts` equal parts,
 // times w; out [T, n] (+ bf16 copy).  gate_last: u = y[t, :], and the normed row is multiplied by sigmoid(z[t, :]) instead
-// (linear attention with constant decays)
+// (linear attention with constant decays).  z_b16: z as bf16 instead (then n / parts is a multiple of 4, at most 8192)
 cudaError_t gated_group_norm(cudaStream_t s, const float* y, long ldy, const float* z, long ldz, const void* w, bool f32, float eps,
-                             int parts, float* out, bf16* out_b16, int T, int n, bool gate_last = false);
+                             int parts, float* out, bf16* out_b16, int T, int n, bool gate_last = false, const bf16* z_b16 = nullptr);
 // out[t, col0 + e] = in[t, e] * sigmoid(g[t, e]) * scale, e < n (in: fp32, or bf16 when in_b16 is given instead)
 cudaError_t gate_scale_rows(cudaStream_t s, const float* in, const bf16* in_b16, long ldi, const float* g, long ldg, float scale,
                             float* out, bf16* out_b16, long ldout, int col0, int T, int n);

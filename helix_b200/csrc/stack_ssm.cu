@@ -409,6 +409,13 @@ __global__ void memory_readout_kernel(const float* __restrict__ num, long ldnum,
   }
 }
 
+template <typename WT>
+__device__ __forceinline__ float4 ldf4(const WT* p) {
+  if constexpr (sizeof(WT) == 4) return *reinterpret_cast<const float4*>(p);
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
 // one block per (part, token)
 template <typename WT>
 __global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* __restrict__ y, long ldy, const float* __restrict__ z, long ldz,
@@ -457,13 +464,14 @@ __global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* __re
 
 // The same with a part in registers as float4 (parts of a multiple of 4 entries, up to 4 * 256 * CH)
 template <typename WT, int CH>
-__global__ void __launch_bounds__(256) gated_group_norm_vec_kernel(const float* __restrict__ y, long ldy, const float* __restrict__ z, long ldz,
+__global__ void __launch_bounds__(256) gated_group_norm_vec_kernel(const float* __restrict__ y, long ldy, const float* __restrict__ z, const bf16* __restrict__ zb, long ldz,
                                                                    const WT* __restrict__ w, float eps, int parts, float* __restrict__ out,
                                                                    bf16* __restrict__ outb, int n, int gate_last) {
   __shared__ float red[32];
   const int t = blockIdx.y, part = blockIdx.x, len = n / parts, c0 = part * len;
   const float* ys = y + (size_t)t * ldy + c0;
-  const float* zs = z + (size_t)t * ldz + c0;
+  const float* zs = z ? z + (size_t)t * ldz + c0 : nullptr;
+  const bf16* zbs = zb ? zb + (size_t)t * ldz + c0 : nullptr;
   float4 u[CH], g[CH];
   float ss = 0.f;
 #pragma unroll
@@ -472,7 +480,7 @@ __global__ void __launch_bounds__(256) gated_group_norm_vec_kernel(const float* 
     u[c] = g[c] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i >= len) continue;
     u[c] = *reinterpret_cast<const float4*>(ys + i);
-    g[c] = *reinterpret_cast<const float4*>(zs + i);
+    g[c] = zs ? *reinterpret_cast<const float4*>(zs + i) : ldf4<bf16>(zbs + i);
   }
 #pragma unroll
   for (int c = 0; c < CH; ++c) {
@@ -561,13 +569,6 @@ __global__ void __launch_bounds__(256) parallel_step_kernel(const float* x, cons
 // The same step with the row in registers as float4 (W a multiple of 4, W <= 4 * 256 * kParChunks)
 constexpr int kParChunks = 8;
 constexpr int kParTop = 8;  // expert rows per token that the in-register form takes
-template <typename WT>
-__device__ __forceinline__ float4 ldf4(const WT* p) {
-  if constexpr (sizeof(WT) == 4) return *reinterpret_cast<const float4*>(p);
-  const uint2 u = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
 __device__ __forceinline__ float4 fma4(float a, float4 b, float4 c) {
   return make_float4(fmaf(a, b.x, c.x), fmaf(a, b.y, c.y), fmaf(a, b.z, c.z), fmaf(a, b.w, c.w));
 }
@@ -744,13 +745,13 @@ cudaError_t memory_readout(cudaStream_t s, const float* num, long ldnum, const f
 }
 
 cudaError_t gated_group_norm(cudaStream_t s, const float* y, long ldy, const float* z, long ldz, const void* w, bool f32, float eps, int parts,
-                             float* out, bf16* outb, int T, int n, bool gate_last) {
+                             float* out, bf16* outb, int T, int n, bool gate_last, const bf16* zb) {
   if (T <= 0) return cudaSuccess;
   if (parts < 1 || n % parts) return cudaErrorInvalidValue;
   dim3 grid(parts, T);
   const int len = n / parts;
-  if (len % 4 == 0 && len <= 8192 && ((ldy | ldz) & 3) == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)out) & 15) == 0 && ((uintptr_t)outb & 7) == 0) {
-#define HB_GGN(WT, CH) gated_group_norm_vec_kernel<WT, CH><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const WT*)w, eps, parts, out, outb, n, gate_last)
+  if (len % 4 == 0 && len <= 8192 && ((ldy | ldz) & 3) == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)out) & 15) == 0 && (((uintptr_t)outb | (uintptr_t)zb) & 7) == 0) {
+#define HB_GGN(WT, CH) gated_group_norm_vec_kernel<WT, CH><<<grid, 256, 0, s>>>(y, ldy, z, zb, ldz, (const WT*)w, eps, parts, out, outb, n, gate_last)
 #define HB_GGN_T(CH) do { if (f32) HB_GGN(float, CH); else HB_GGN(bf16, CH); } while (0)
     if (len <= 1024) HB_GGN_T(1);
     else if (len <= 2048) HB_GGN_T(2);
@@ -760,6 +761,7 @@ cudaError_t gated_group_norm(cudaStream_t s, const float* y, long ldy, const flo
 #undef HB_GGN
     return cudaGetLastError();
   }
+  if (zb) return cudaErrorInvalidValue;
   if (f32) gated_group_norm_kernel<float><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const float*)w, eps, parts, out, outb, n, gate_last);
   else gated_group_norm_kernel<bf16><<<grid, 256, 0, s>>>(y, ldy, z, ldz, (const bf16*)w, eps, parts, out, outb, n, gate_last);
   return cudaGetLastError();

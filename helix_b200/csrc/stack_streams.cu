@@ -38,7 +38,7 @@ __device__ __forceinline__ void st_both(float* f, bf16* b, float4 v) {
 }
 
 // One block per row, S copies of four neighbouring entries per thread and chunk (W a multiple of 4)
-template <typename WT, int S, int CH>
+template <typename WT, int S, int CH, bool ROWS>
 __global__ void __launch_bounds__(256) stream_step_vec_kernel(StreamStep a) {
   __shared__ float red[32];
   const size_t r = blockIdx.x;
@@ -51,14 +51,16 @@ __global__ void __launch_bounds__(256) stream_step_vec_kernel(StreamStep a) {
 #pragma unroll
     for (int t = 0; t < S; ++t) mix[s][t] = a.mix ? ldf<WT>((const WT*)a.mix, s * S + t) : (s == t ? 1.f : 0.f);
   }
-  float wk[kTop];
-  size_t rk[kTop];
+  float wk[ROWS ? kTop : 1];
+  int rk[ROWS ? kTop : 1];
+  if constexpr (ROWS) {
 #pragma unroll
-  for (int k = 0; k < kTop; ++k) {
-    wk[k] = k < a.top_k ? a.wts[r * a.top_k + k] : 0.f;
-    rk[k] = k < a.top_k ? (size_t)a.row_of[r * a.top_k + k] * W : 0;
+    for (int k = 0; k < kTop; ++k) {
+      wk[k] = k < a.top_k ? a.wts[r * a.top_k + k] : 0.f;
+      rk[k] = k < a.top_k ? a.row_of[r * a.top_k + k] : 0;
+    }
   }
-  const bool add = a.y || a.top_k > 0;
+  const bool add = ROWS || a.y;
   float* xr = a.x + r * S * W;
   float4 u[CH];
   float ss = 0.f;
@@ -73,9 +75,11 @@ __global__ void __launch_bounds__(256) stream_step_vec_kernel(StreamStep a) {
 #pragma unroll
     for (int s = 0; s < S; ++s) xc[s] = a.x0 ? *reinterpret_cast<const float4*>(a.x0 + r * W + i) : *reinterpret_cast<const float4*>(xr + (size_t)s * W + i);
     if (a.y) yc = *reinterpret_cast<const float4*>(a.y + r * W + i);
+    if constexpr (ROWS) {
 #pragma unroll
-    for (int k = 0; k < kTop; ++k)
-      if (k < a.top_k) yc = fma4(wk[k], ld4<bf16>(a.rows + rk[k] + i), yc);
+      for (int k = 0; k < kTop; ++k)
+        if (k < a.top_k) yc = fma4(wk[k], ld4<bf16>(a.rows + (size_t)rk[k] * W + i), yc);
+    }
     if (a.bias) yc = fma4(1.f, ld4<WT>((const WT*)a.bias + i), yc);
   };
   if constexpr (B > 1) {
@@ -173,12 +177,17 @@ __global__ void __launch_bounds__(256) stream_step_kernel(StreamStep a) {
   }
 }
 
+template <typename WT, int S, bool ROWS>
+void launch_rows(cudaStream_t s, const StreamStep& a, int rows) {
+  if (a.W <= 1024) stream_step_vec_kernel<WT, S, 1, ROWS><<<rows, 256, 0, s>>>(a);
+  else if (a.W <= 2048) stream_step_vec_kernel<WT, S, 2, ROWS><<<rows, 256, 0, s>>>(a);
+  else if (a.W <= 4096) stream_step_vec_kernel<WT, S, 4, ROWS><<<rows, 256, 0, s>>>(a);
+  else stream_step_vec_kernel<WT, S, 8, ROWS><<<rows, 256, 0, s>>>(a);
+}
 template <typename WT, int S>
 void launch_vec(cudaStream_t s, const StreamStep& a, int rows) {
-  if (a.W <= 1024) stream_step_vec_kernel<WT, S, 1><<<rows, 256, 0, s>>>(a);
-  else if (a.W <= 2048) stream_step_vec_kernel<WT, S, 2><<<rows, 256, 0, s>>>(a);
-  else if (a.W <= 4096) stream_step_vec_kernel<WT, S, 4><<<rows, 256, 0, s>>>(a);
-  else stream_step_vec_kernel<WT, S, 8><<<rows, 256, 0, s>>>(a);
+  if (a.top_k > 0) launch_rows<WT, S, true>(s, a, rows);
+  else launch_rows<WT, S, false>(s, a, rows);
 }
 
 }  // namespace
